@@ -244,6 +244,11 @@ int64_t llmopt_cuda_f16_argmax(const void* halves, size_t count);
 int llmopt_cuda_sample_f16(const void* halves, size_t count, double temperature, int top_k, double top_p,
                            double min_p, uint64_t seed, int64_t* token);
 
+/* The same sampler over fp32 logits (an addition of this library: the models whose output
+ * projection writes fp32 sample from it without a rounding to half). */
+int llmopt_cuda_sample_f32(const void* floats, size_t count, double temperature, int top_k, double top_p,
+                           double min_p, uint64_t seed, int64_t* token);
+
 /* caml_llmopt_metal_measure_hardware (:477-611, bound at bin/hardware_probe.ml:11): device
  * name, the largest thread block, the median launch-to-completion time of an empty kernel
  * (host clock, seconds) and the median bandwidth of a device-to-device copy of `bytes`

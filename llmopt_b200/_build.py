@@ -5,11 +5,18 @@ from __future__ import annotations
 import os
 import subprocess
 import sys
+from typing import Optional
 
 PACKAGE_DIR = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(PACKAGE_DIR, "csrc")
 LIBRARY = os.path.join(PACKAGE_DIR, "libllmopt_cuda.so")
 OBJECTS = os.path.join(PACKAGE_DIR, "build")
+
+# Kernel families that are enough to serve one kind of model: a host that needs no others can build
+# and load libllmopt_cuda_<family>.so (the runtime registers only the names that were linked in).
+FAMILIES = {
+    "mixers": ("runtime", "sampling", "dense_linear", "dense_gemm_tc", "sequence_glue", "row_attention", "matrix_state"),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -17,25 +24,40 @@ NVCC_FLAGS = [
 ]
 
 
-def sources() -> list[str]:
-    return sorted(os.path.join(CSRC, name) for name in os.listdir(CSRC) if name.endswith(".cu"))
+def library_path(family: Optional[str] = None) -> str:
+    return LIBRARY if family is None else os.path.join(PACKAGE_DIR, f"libllmopt_cuda_{family}.so")
+
+
+def sources(family: Optional[str] = None) -> list[str]:
+    names = sorted(name[:-3] for name in os.listdir(CSRC) if name.endswith(".cu"))
+    return [os.path.join(CSRC, name + ".cu") for name in names if family is None or name in FAMILIES[family]]
+
+
+def headers() -> list[str]:
+    found = [os.path.join(CSRC, name) for name in os.listdir(CSRC) if name.endswith((".cuh", ".h"))]
+    return found + [os.path.join(PACKAGE_DIR, "..", "include", "llmopt_cuda.h")]
+
+
+def current(family: Optional[str] = None) -> bool:
+    """Whether the library exists and is no older than its sources."""
+    library = library_path(family)
+    return os.path.exists(library) and not any(_newer(path, library) for path in sources(family) + headers())
 
 
 def _newer(path: str, than: str) -> bool:
     return (not os.path.exists(than)) or os.path.getmtime(path) > os.path.getmtime(than)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    """Compile changed translation units and link the shared library."""
+def build(force: bool = False, verbose: bool = False, family: Optional[str] = None) -> str:
+    """Compile changed translation units and link the shared library (of one family of kernels)."""
     nvcc = os.environ.get("NVCC", "nvcc")
     os.makedirs(OBJECTS, exist_ok=True)
-    headers = [os.path.join(CSRC, name) for name in os.listdir(CSRC) if name.endswith((".cuh", ".h"))]
-    headers.append(os.path.join(PACKAGE_DIR, "..", "include", "llmopt_cuda.h"))
+    library = library_path(family)
     objects, jobs = [], []
-    for source in sources():
+    for source in sources(family):
         obj = os.path.join(OBJECTS, os.path.basename(source)[:-3] + ".o")
         objects.append(obj)
-        stale = force or _newer(source, obj) or any(_newer(h, obj) for h in headers if os.path.exists(h))
+        stale = force or _newer(source, obj) or any(_newer(h, obj) for h in headers() if os.path.exists(h))
         if stale:
             command = [nvcc, *NVCC_FLAGS, "-c", source, "-o", obj]
             if verbose:
@@ -51,12 +73,13 @@ def build(force: bool = False, verbose: bool = False) -> str:
             sys.stderr.write(output)
     if failed:
         raise RuntimeError("libllmopt_cuda.so: compilation failed")
-    if jobs or not os.path.exists(LIBRARY):
+    if jobs or not os.path.exists(library) or any(_newer(obj, library) for obj in objects):
         subprocess.check_call(
-            [nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-o", LIBRARY, *objects, "-lcudart"]
+            [nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-o", library, *objects, "-lcudart"]
         )
-    return LIBRARY
+    return library
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
+    chosen = [name for name in FAMILIES if f"--{name}" in sys.argv]
+    print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv, family=chosen[0] if chosen else None))

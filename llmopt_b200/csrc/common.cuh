@@ -49,6 +49,10 @@ struct KernelArgs {
 };
 
 typedef int (*Launcher)(const KernelArgs&);
+struct NamedLauncher {
+  const char* name;
+  Launcher launcher;
+};
 
 // Scratch owned by the context; grows on demand outside graph capture.
 void* context_scratch(Context* ctx, size_t bytes, std::string* error);

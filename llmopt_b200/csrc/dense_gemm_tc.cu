@@ -1,0 +1,265 @@
+// Prompt rows of the dense bfloat16 linear layer on the 5th-generation tensor cores:
+//   y[m, n] = x[m, k] . w[n, k]^T, fp32 accumulation in tensor memory.
+//
+// A persistent CTA walks over 128 x BN output tiles.  Warp 0 brings the x tile [128 x 64] and the w
+// tile [BN x 64] of every k-block into a shared-memory ring by TMA (128-byte swizzle); one thread of
+// warp 1 issues four tcgen05.mma (K = 16) per k-block into one of two accumulators in tensor memory;
+// warps 2-5 read the finished accumulator (each its quarter of the lanes = output rows), apply bias
+// and activation and store, while the next tile accumulates in the other one.  Rows, columns and k
+// beyond the matrices are zero-filled by TMA.
+//
+// Every wait on an mbarrier is bounded; a wait that runs out raises the context's device error word,
+// and the CTA lets its copies land, frees its tensor memory and returns.
+#include <cuda.h>
+
+#include "dense_linear.cuh"
+#include "w4a16_tc_device.cuh"
+
+namespace llmopt {
+using namespace tc;
+
+uint32_t* context_device_error(Context* ctx);
+
+namespace {
+
+constexpr uint32_t kRows = 128, kDepth = 64;
+constexpr uint32_t kThreads = 192;  // TMA, MMA, four epilogue warps
+constexpr uint32_t kXTileBytes = kRows * kDepth * 2;
+
+template <uint32_t BN>
+struct Shape {
+  static constexpr uint32_t kWTileBytes = BN * kDepth * 2;
+  static constexpr uint32_t kStageBytes = kXTileBytes + kWTileBytes;
+  static constexpr uint32_t kStages = BN == 256 ? 4 : (BN == 128 ? 6 : 8);
+  static constexpr uint32_t kTmemColumns = 2 * BN;
+  static constexpr uint32_t kBarriers = kStages * kStageBytes;
+  static constexpr uint32_t kHolder = kBarriers + (2 * kStages + 4) * 8;
+  static constexpr uint32_t kAbort = kHolder + 4;
+  static constexpr uint32_t kSharedBytes = kAbort + 4 + 1024;  // slack: 1024-byte alignment of the tiles
+};
+
+// kind::f16 with bfloat16 A and B (format 1), fp32 accumulator, both K-major.
+__host__ __device__ constexpr uint32_t bf16_instruction(uint32_t m, uint32_t n) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((m >> 4) << 24);
+}
+
+template <uint32_t BN>
+__global__ void __launch_bounds__(kThreads, 1)
+dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
+                     const DenseProblem p, uint32_t* error_word) {
+  using S = Shape<BN>;
+  extern __shared__ unsigned char shared_raw[];
+  grid_chain_prologue();
+  const uint32_t base = (smem_u32(shared_raw) + 1023u) & ~1023u;
+  unsigned char* base_pointer = shared_raw + (base - smem_u32(shared_raw));
+  const uint32_t full = base + S::kBarriers, empty = full + S::kStages * 8;
+  const uint32_t sums_full = empty + S::kStages * 8, sums_empty = sums_full + 16;
+  volatile uint32_t* holder = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kHolder);
+  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kAbort);
+  const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
+  const uint32_t m_tiles = (p.m + kRows - 1u) / kRows, n_tiles = (p.n + BN - 1u) / BN, tiles = m_tiles * n_tiles;
+  const uint32_t k_blocks = (p.k + kDepth - 1u) / kDepth;
+
+  if (threadIdx.x == 0) {
+    for (uint32_t s = 0; s < S::kStages; ++s) {
+      barrier_init(full + s * 8, 1);   // the producer's expect_tx arrival; completes by byte count
+      barrier_init(empty + s * 8, 1);  // one tcgen05.commit
+    }
+    for (uint32_t s = 0; s < 2; ++s) {
+      barrier_init(sums_full + s * 8, 1);   // one tcgen05.commit
+      barrier_init(sums_empty + s * 8, 4);  // one arrival per epilogue warp
+    }
+    *abort_flag = 0u;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(base + S::kHolder),
+                 "r"(S::kTmemColumns)
+                 : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+  const uint32_t tmem_base = *holder;
+  auto give_up = [&]() {
+    *abort_flag = 1u;
+    if (error_word) atomicExch(error_word, 1u);
+  };
+
+  if (warp == 0) {
+    if (lane == 0) {
+      uint32_t issued = 0;  // k-blocks over all tiles of this CTA
+      bool ok = true;
+      for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
+        const uint32_t m0 = (tile % m_tiles) * kRows, n0 = (tile / m_tiles) * BN;
+        for (uint32_t kb = 0; kb < k_blocks; ++kb, ++issued) {
+          const uint32_t s = issued % S::kStages;
+          ok = !*abort_flag && barrier_wait(empty + s * 8, ((issued / S::kStages) & 1u) ^ 1u);
+          if (!ok) {
+            give_up();
+            break;
+          }
+          barrier_expect_tx(full + s * 8, S::kStageBytes);
+          const uint32_t stage = base + s * S::kStageBytes;
+          tma_load_2d(stage, &map_x, (int32_t)(kb * kDepth), (int32_t)m0, full + s * 8);
+          tma_load_2d(stage + kXTileBytes, &map_w, (int32_t)(kb * kDepth), (int32_t)n0, full + s * 8);
+        }
+      }
+      // on the way out after a failure the copies already started must land first
+      if (!ok || *abort_flag)
+        for (uint32_t i = issued > S::kStages ? issued - S::kStages : 0u; i < issued; ++i)
+          barrier_wait(full + (i % S::kStages) * 8, (i / S::kStages) & 1u);
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      uint32_t consumed = 0, turn = 0;
+      bool ok = true;
+      for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++turn) {
+        const uint32_t half = turn & 1u, sums = tmem_base + half * BN;
+        ok = !*abort_flag && barrier_wait(sums_empty + half * 8, ((turn >> 1) & 1u) ^ 1u);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        for (uint32_t kb = 0; kb < k_blocks && ok; ++kb, ++consumed) {
+          const uint32_t s = consumed % S::kStages;
+          ok = !*abort_flag && barrier_wait(full + s * 8, (consumed / S::kStages) & 1u);
+          if (!ok) break;
+          asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+          const uint32_t x_tile = base + s * S::kStageBytes, w_tile = x_tile + kXTileBytes;
+#pragma unroll
+          for (uint32_t j = 0; j < kDepth / 16; ++j)
+            mma_f16(sums, operand_descriptor(x_tile + j * 32), operand_descriptor(w_tile + j * 32),
+                    (kb > 0 || j > 0) ? 1u : 0u, bf16_instruction(kRows, BN));
+          mma_commit(empty + s * 8);
+        }
+        if (ok) mma_commit(sums_full + half * 8);
+      }
+      if (!ok) give_up();
+    }
+  } else {
+    const uint32_t quarter = warp & 3u;
+    uint32_t turn = 0;
+    bool ok = true;
+    for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++turn) {
+      const uint32_t half = turn & 1u;
+      ok = !*abort_flag && barrier_wait(sums_full + half * 8, (turn >> 1) & 1u);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) {
+        give_up();
+        break;
+      }
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const uint32_t row = (tile % m_tiles) * kRows + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
+      const uint32_t address = tmem_base + half * BN + ((quarter * 32u) << 16);
+#pragma unroll 1
+      for (uint32_t piece = 0; piece < BN / 32u; ++piece) {
+        uint32_t raw[32];
+        tmem_load_32(address + piece * 32u, raw);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        const uint32_t column = n0 + piece * 32u;
+        const size_t at = (size_t)row * p.split + column;
+        const size_t at32 = (size_t)row * (p.n - p.split) + (column - p.split);
+        if (row >= p.m || column >= p.n) {
+          // absent
+        } else if (column + 32u <= p.split && (at & 7u) == 0) {
+          uint4* target = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + at);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            uint32_t packed[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const int e = i * 8 + j * 2;
+              const __nv_bfloat162 pair =
+                  __floats2bfloat162_rn(dense_finish<bf16>(p, row, column + e, __uint_as_float(raw[e])),
+                                        dense_finish<bf16>(p, row, column + e + 1, __uint_as_float(raw[e + 1])));
+              packed[j] = *reinterpret_cast<const uint32_t*>(&pair);
+            }
+            target[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+          }
+        } else if (column >= p.split && column + 32u <= p.n && (at32 & 3u) == 0) {
+          float4* target = reinterpret_cast<float4*>(p.out32 + at32);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            float v[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              v[j] = dense_finish<bf16>(p, row, column + i * 4 + j, __uint_as_float(raw[i * 4 + j]));
+            target[i] = make_float4(v[0], v[1], v[2], v[3]);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+        }
+        __syncwarp();  // tcgen05.ld needs the whole warp
+      }
+      asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      __syncwarp();
+      if (lane == 0) barrier_arrive(sums_empty + half * 8);
+    }
+  }
+
+  __syncthreads();
+  if (warp == 1) {
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(S::kTmemColumns)
+                 : "memory");
+  }
+}
+
+// cuTensorMapEncodeTiled, resolved through the runtime so that the library does not link libcuda.
+typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
+                                const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
+                                CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// Row-major bf16 matrix [outer, inner] read in boxes of 64 x `box_rows` with the 128-byte swizzle.
+bool make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint32_t box_rows) {
+  static EncodeTiled encode = []() -> EncodeTiled {
+    void* pointer = nullptr;
+    cudaDriverEntryPointQueryResult result;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &pointer, cudaEnableDefault, &result) != cudaSuccess ||
+        result != cudaDriverEntryPointSuccess)
+      return nullptr;
+    return reinterpret_cast<EncodeTiled>(pointer);
+  }();
+  if (encode == nullptr) return false;
+  const cuuint64_t dims[2] = {inner, outer}, strides[1] = {inner * 2};
+  const cuuint32_t box[2] = {kDepth, box_rows}, element_strides[2] = {1, 1};
+  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, element_strides,
+                CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <uint32_t BN>
+int run(const KernelArgs& args, const DenseProblem& p, uint32_t sms) {
+  using S = Shape<BN>;
+  CUtensorMap map_x, map_w;
+  if (!make_map(&map_x, p.x, p.k, p.m, kRows) || !make_map(&map_w, p.w, p.k, p.n, BN)) return -1;
+  auto kernel = dense_gemm_tc_kernel<BN>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSharedBytes) != cudaSuccess) {
+    cudaGetLastError();
+    return -1;
+  }
+  const uint32_t tiles = ((p.m + kRows - 1u) / kRows) * ((p.n + BN - 1u) / BN);
+  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, p,
+                context_device_error(args.ctx));
+  return check_launch(args);
+}
+
+}  // namespace
+
+int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& p) {
+  if (args.ctx == nullptr || p.k % 8u != 0 || ((uintptr_t)p.x & 15u) != 0 || ((uintptr_t)p.w & 15u) != 0) return -1;
+  const uint32_t sms = (uint32_t)context_sm_count(args.ctx);
+  // waves times the cost of one MMA (an MMA of up to 128 columns costs about two thirds of one of 256)
+  const uint32_t m_tiles = (p.m + kRows - 1u) / kRows;
+  auto cost = [&](uint32_t columns, uint32_t mma) {
+    const uint32_t tiles = m_tiles * ((p.n + columns - 1u) / columns);
+    return (tiles + sms - 1u) / sms * mma;
+  };
+  const uint32_t wide = cost(256, 128), middle = cost(128, 85), narrow = cost(64, 80);
+  if (narrow < middle && narrow < wide) return run<64>(args, p, sms);
+  if (middle < wide) return run<128>(args, p, sms);
+  return run<256>(args, p, sms);
+}
+
+}  // namespace llmopt

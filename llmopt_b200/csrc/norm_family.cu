@@ -459,10 +459,6 @@ int launch_unary(const KernelArgs& args) {
 }
 
 // name -> launcher table of this file, appended to the registry by the runtime
-struct NamedLauncher {
-  const char* name;
-  Launcher launcher;
-};
 const NamedLauncher* norm_family_launchers(size_t* count) {
   static const NamedLauncher table[] = {
       {"llmopt_rms_norm_f32_f16_wf32_simd", launch_rms_norm_f32_wf32},

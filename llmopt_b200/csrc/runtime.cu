@@ -27,68 +27,72 @@
 namespace llmopt {
 
 // ---- launchers defined in the kernel translation units --------------------------
-int launch_w4a16_linear(const KernelArgs&);
-int launch_w4a16_linear_affine(const KernelArgs&);
-int launch_w4a16_qkv_linear(const KernelArgs&);
-int launch_w4a16_swiglu_rms_f16(const KernelArgs&);
-int launch_w4a16_swiglu_rms_f32(const KernelArgs&);
-int launch_w4a16_dual_swiglu(const KernelArgs&);
-int launch_w4a16_down_add(const KernelArgs&);
-template <int TAG> int launch_w4a16_linear_tagged(const KernelArgs&);
-template <bool F32, bool EXTRA> int launch_w4a16_lm_head_argmax(const KernelArgs&);
-template <bool F32, bool EXTRA> int launch_w4a16_lm_head_stage1(const KernelArgs&);
-int launch_w4a16_lm_head_reduce(const KernelArgs&);
-int launch_w4a16_linear_partial_f32(const KernelArgs&);
-int launch_tp_exchange_sum(const KernelArgs&);
-int launch_tp_exchange_argmax(const KernelArgs&);
-int launch_tp_exchange_sum_norm(const KernelArgs&);
-int launch_tp_exchange_reduce_rows(const KernelArgs&);
-int launch_tp_exchange_gather_rows(const KernelArgs&);
-int launch_attention_dense(const KernelArgs&);
-int launch_q4_0_linear(const KernelArgs&);
-int launch_q4_0_gated_linear(const KernelArgs&);
-int launch_tile32_affine4_linear(const KernelArgs&);
-int launch_cache_pack_tile32_affine8_fwht(const KernelArgs&);
-int launch_cache_unpack_tile32_affine8_fwht(const KernelArgs&);
-int launch_cache_pack_tile32_affine4_fwht(const KernelArgs&);
-int launch_cache_unpack_tile32_affine4_fwht(const KernelArgs&);
-int launch_tile32_affine8_linear(const KernelArgs&);
-int launch_q4_0_qkv_linear(const KernelArgs&);
-int launch_q4_0_dequant(const KernelArgs&);
-int launch_cache_pack_attention_q8(const KernelArgs&);
-int launch_cache_pack_attention_q8_pair(const KernelArgs&);
-int launch_cache_unpack_attention_q8(const KernelArgs&);
-int launch_cache_pack_checkpoint_q8(const KernelArgs&);
-int launch_cache_unpack_checkpoint_q8(const KernelArgs&);
-int launch_attention_q8_paged(const KernelArgs&);
-template <bool WEIGHT_F32> int launch_short_conv(const KernelArgs&);
-template <bool WEIGHT_F32> int launch_short_conv_silu_tm(const KernelArgs&);
-int launch_short_conv_step(const KernelArgs&);
-int launch_short_conv_prefill(const KernelArgs&);
-template <bool INPUT_F32> int launch_rms_norm(const KernelArgs&);
-int launch_rotary_qk(const KernelArgs&);
-int launch_rotary_pack_fused(const KernelArgs& rotary, const KernelArgs& pack);
-bool paged_attention_takes_rotary_pack(const KernelArgs& attention, const RotaryPackFusion& fusion);
-int launch_embedding_f16(const KernelArgs&);
-int launch_chain_token_id(const KernelArgs&);
-int launch_chain_token_ids(const KernelArgs&);
-void launch_argmax_f16(const __half* values, uint32_t count, int* result, cudaStream_t stream);
-struct NamedLauncher {
-  const char* name;
-  Launcher launcher;
-};
-const NamedLauncher* norm_family_launchers(size_t* count);
+// Weak: a library linked from some of the kernel families only (llmopt_b200/_build.py) has null here for
+// the others, registers no names for them and reports a missing kernel function when one is asked for.
+#define LLMOPT_FAMILY __attribute__((weak, visibility("default")))
+LLMOPT_FAMILY int launch_w4a16_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_linear_affine(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_qkv_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_swiglu_rms_f16(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_swiglu_rms_f32(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_dual_swiglu(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_down_add(const KernelArgs&);
+template <int TAG> LLMOPT_FAMILY int launch_w4a16_linear_tagged(const KernelArgs&);
+template <bool F32, bool EXTRA> LLMOPT_FAMILY int launch_w4a16_lm_head_argmax(const KernelArgs&);
+template <bool F32, bool EXTRA> LLMOPT_FAMILY int launch_w4a16_lm_head_stage1(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_lm_head_reduce(const KernelArgs&);
+LLMOPT_FAMILY int launch_w4a16_linear_partial_f32(const KernelArgs&);
+LLMOPT_FAMILY int launch_tp_exchange_sum(const KernelArgs&);
+LLMOPT_FAMILY int launch_tp_exchange_argmax(const KernelArgs&);
+LLMOPT_FAMILY int launch_tp_exchange_sum_norm(const KernelArgs&);
+LLMOPT_FAMILY int launch_tp_exchange_reduce_rows(const KernelArgs&);
+LLMOPT_FAMILY int launch_tp_exchange_gather_rows(const KernelArgs&);
+LLMOPT_FAMILY int launch_attention_dense(const KernelArgs&);
+LLMOPT_FAMILY int launch_q4_0_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_q4_0_gated_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_tile32_affine4_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_pack_tile32_affine8_fwht(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_unpack_tile32_affine8_fwht(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_pack_tile32_affine4_fwht(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_unpack_tile32_affine4_fwht(const KernelArgs&);
+LLMOPT_FAMILY int launch_tile32_affine8_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_q4_0_qkv_linear(const KernelArgs&);
+LLMOPT_FAMILY int launch_q4_0_dequant(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_pack_attention_q8(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_pack_attention_q8_pair(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_unpack_attention_q8(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_pack_checkpoint_q8(const KernelArgs&);
+LLMOPT_FAMILY int launch_cache_unpack_checkpoint_q8(const KernelArgs&);
+LLMOPT_FAMILY int launch_attention_q8_paged(const KernelArgs&);
+template <bool WEIGHT_F32> LLMOPT_FAMILY int launch_short_conv(const KernelArgs&);
+template <bool WEIGHT_F32> LLMOPT_FAMILY int launch_short_conv_silu_tm(const KernelArgs&);
+LLMOPT_FAMILY int launch_short_conv_step(const KernelArgs&);
+LLMOPT_FAMILY int launch_short_conv_prefill(const KernelArgs&);
+template <bool INPUT_F32> LLMOPT_FAMILY int launch_rms_norm(const KernelArgs&);
+LLMOPT_FAMILY int launch_rotary_qk(const KernelArgs&);
+LLMOPT_FAMILY int launch_rotary_pack_fused(const KernelArgs& rotary, const KernelArgs& pack);
+LLMOPT_FAMILY bool make_rotary_pack_fusion(const KernelArgs& rotary, const KernelArgs& pack, RotaryPackFusion* fusion);
+LLMOPT_FAMILY bool paged_attention_takes_rotary_pack(const KernelArgs& attention, const RotaryPackFusion& fusion);
+LLMOPT_FAMILY int launch_embedding_f16(const KernelArgs&);
+LLMOPT_FAMILY int launch_chain_token_id(const KernelArgs&);
+LLMOPT_FAMILY int launch_chain_token_ids(const KernelArgs&);
+LLMOPT_FAMILY void launch_argmax_f16(const __half* values, uint32_t count, int* result, cudaStream_t stream);
+LLMOPT_FAMILY const NamedLauncher* norm_family_launchers(size_t* count);
+LLMOPT_FAMILY const NamedLauncher* dense_linear_launchers(size_t* count);
+LLMOPT_FAMILY const NamedLauncher* sequence_glue_launchers(size_t* count);
+LLMOPT_FAMILY const NamedLauncher* row_attention_launchers(size_t* count);
+LLMOPT_FAMILY const NamedLauncher* matrix_state_launchers(size_t* count);
 struct ExprProgram {
   uint8_t code[192];
   uint32_t length;
   uint32_t operands;
 };
-const char* validate_expr_program(const uint8_t* code, size_t length, int operand_count);
-int launch_w4a16_linear_expr(const KernelArgs&);
-int launch_q4_0_linear_expr(const KernelArgs&);
-int launch_gated_delta_f32(const KernelArgs&);
-int launch_gated_delta_tm_f16(const KernelArgs&);
-int launch_triangular_recurrence(const KernelArgs&);
+LLMOPT_FAMILY const char* validate_expr_program(const uint8_t* code, size_t length, int operand_count);
+LLMOPT_FAMILY int launch_w4a16_linear_expr(const KernelArgs&);
+LLMOPT_FAMILY int launch_q4_0_linear_expr(const KernelArgs&);
+LLMOPT_FAMILY int launch_gated_delta_f32(const KernelArgs&);
+LLMOPT_FAMILY int launch_gated_delta_tm_f16(const KernelArgs&);
+LLMOPT_FAMILY int launch_triangular_recurrence(const KernelArgs&);
 
 // ---- objects -----------------------------------------------------------------------
 
@@ -229,6 +233,7 @@ uint32_t* context_device_error(Context* context) { return context->device_error;
 
 static void register_kernels(llmopt_cuda_library* library) {
   auto add = [&](const char* name, Launcher launcher) {
+    if (launcher == nullptr) return;  // a family this library was linked without
     library->launchers[name] = launcher;
     library->names.push_back(name);
   };
@@ -375,10 +380,16 @@ static void register_kernels(llmopt_cuda_library* library) {
   for (const char* name : kGatedDeltaF32) add(name, launch_gated_delta_f32);
   for (const char* name : kGatedDeltaF16) add(name, launch_gated_delta_tm_f16);
   add("llmopt_triangular_recurrence_f32", launch_triangular_recurrence);
-  // norm variants, fused norm + rotary, casts, pointwise (norm_family.cu)
-  size_t extra = 0;
-  const NamedLauncher* table = norm_family_launchers(&extra);
-  for (size_t i = 0; i < extra; ++i) add(table[i].name, table[i].launcher);
+  // families that list their own names: norm variants, fused norm + rotary, casts, pointwise (norm_family.cu);
+  // the sequence-mixer kernels
+  const NamedLauncher* (*const families[])(size_t*) = {norm_family_launchers, dense_linear_launchers,
+                                                       sequence_glue_launchers, row_attention_launchers,
+                                                       matrix_state_launchers};
+  for (auto family : families) {
+    size_t count = 0;
+    const NamedLauncher* table = family != nullptr ? family(&count) : nullptr;
+    for (size_t i = 0; i < count; ++i) add(table[i].name, table[i].launcher);
+  }
 }
 
 static bool is_paged_attention_name(const char* name) {
@@ -831,6 +842,8 @@ int llmopt_cuda_register_expr_epilogue(llmopt_cuda_library* library, const char*
     return set_error(LLMOPT_CUDA_INVALID_ARGUMENT, "expression epilogue needs a name and a program");
   if (library->launchers.count(name))
     return set_error(LLMOPT_CUDA_INVALID_ARGUMENT, std::string("kernel name is already taken: ") + name);
+  if (validate_expr_program == nullptr)
+    return set_error(LLMOPT_CUDA_FAILURE, "this library was linked without the expression epilogues");
   if (const char* problem = validate_expr_program((const uint8_t*)program, program_bytes, operand_count))
     return set_error(LLMOPT_CUDA_INVALID_ARGUMENT, problem);
   ExprProgram stored = {};
@@ -1001,6 +1014,7 @@ int llmopt_cuda_buffer_argmax_f16(llmopt_cuda_buffer* buffer, int64_t vocabulary
   Context* context = buffer->allocation->context;
   const size_t rows = buffer->length / ((size_t)vocabulary * 2);
   const __half* last_row = (const __half*)buffer->pointer() + (rows - 1) * (size_t)vocabulary;
+  if (launch_argmax_f16 == nullptr) return set_error(LLMOPT_CUDA_FAILURE, "this library was linked without the fp16 argmax");
   launch_argmax_f16(last_row, (uint32_t)vocabulary, context->argmax_result, context->stream);
   int result = 0;
   CUDA_TRY(cudaMemcpyAsync(&result, context->argmax_result, sizeof(int), cudaMemcpyDeviceToHost, context->stream),
@@ -1548,6 +1562,8 @@ int llmopt_cuda_w4a16_linear(llmopt_cuda_context* context, const void* input, co
   args.name = "llmopt_w4a16_linear_f16_g64";
   std::string message;
   args.error = &message;
+  if (launch_w4a16_linear == nullptr)
+    return set_error(LLMOPT_CUDA_FAILURE, "this library was linked without the W4A16 kernels");
   if (launch_w4a16_linear(args) != 0) return set_error(LLMOPT_CUDA_FAILURE, message);
   return LLMOPT_CUDA_OK;
 }

@@ -96,21 +96,20 @@ double median_of(std::vector<double>& samples) {
 
 using namespace llmopt;
 
-extern "C" int llmopt_cuda_sample_f16(const void* halves, size_t count, double temperature, int top_k, double top_p,
-                                      double min_p, uint64_t seed, int64_t* token) {
-  if (token == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f16: null result pointer");
-  *token = 0;
-  if (count == 0) return LLMOPT_CUDA_OK;
-  if (halves == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f16: null logits");
-  const __half* logits = static_cast<const __half*>(halves);
+namespace {
+
+// `logit(i)`: logit i of the row as fp32.
+template <typename Logit>
+int sample_logits(Logit logit, size_t count, double temperature, int top_k, double top_p, double min_p, uint64_t seed,
+                  int64_t* token) {
   const float temp = (float)temperature, nucleus = (float)top_p, floor_p = (float)min_p;
 
   // greedy: first maximum of the row, compared as halves
   if (temp <= 0.0001f || top_k == 1) {
-    float best = __half2float(logits[0]);
+    float best = logit(0);
     size_t best_index = 0;
     for (size_t i = 1; i < count; ++i) {
-      const float value = __half2float(logits[i]);
+      const float value = logit(i);
       if (value > best) {
         best = value;
         best_index = i;
@@ -126,7 +125,7 @@ extern "C" int llmopt_cuda_sample_f16(const void* halves, size_t count, double t
   else if (top_k > 256) keep = 256;
   CandidateHeap heap;
   for (size_t i = 0; i < count; ++i) {
-    const float value = __half2float(logits[i]);
+    const float value = logit(i);
     if (heap.size < keep) {
       heap.item[heap.size] = {(uint32_t)i, value};
       heap.settle_up(heap.size);
@@ -203,6 +202,29 @@ extern "C" int llmopt_cuda_sample_f16(const void* halves, size_t count, double t
   }
   *token = (int64_t)chosen;
   return LLMOPT_CUDA_OK;
+}
+
+}  // namespace
+
+extern "C" int llmopt_cuda_sample_f16(const void* halves, size_t count, double temperature, int top_k, double top_p,
+                                      double min_p, uint64_t seed, int64_t* token) {
+  if (token == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f16: null result pointer");
+  *token = 0;
+  if (count == 0) return LLMOPT_CUDA_OK;
+  if (halves == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f16: null logits");
+  const __half* logits = static_cast<const __half*>(halves);
+  return sample_logits([=](size_t i) { return __half2float(logits[i]); }, count, temperature, top_k, top_p, min_p, seed,
+                       token);
+}
+
+extern "C" int llmopt_cuda_sample_f32(const void* floats, size_t count, double temperature, int top_k, double top_p,
+                                      double min_p, uint64_t seed, int64_t* token) {
+  if (token == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f32: null result pointer");
+  *token = 0;
+  if (count == 0) return LLMOPT_CUDA_OK;
+  if (floats == nullptr) return sampler_fail(LLMOPT_CUDA_INVALID_ARGUMENT, "sample_f32: null logits");
+  const float* logits = static_cast<const float*>(floats);
+  return sample_logits([=](size_t i) { return logits[i]; }, count, temperature, top_k, top_p, min_p, seed, token);
 }
 
 extern "C" int llmopt_cuda_measure_hardware(int device, int warmup, int repeats, int64_t bytes, char* name,

@@ -1,0 +1,463 @@
+// Row-wise kernels of decoders whose residual stream is kept in fp32 and whose sublayers read it
+// directly (T: bfloat16 or float, the element of activations and weights):
+//   llmopt_embedding_residual_{bf16,f32}   x = table[token], with a T copy for the next product
+//   llmopt_residual_norm_{bf16,f32}        x += norm(y), or of the mean of two normed branches
+//   llmopt_gather_norm_{bf16,f32}          norm of chosen rows (input of the output projection)
+//   llmopt_row_attention_prepare_{bf16,f32} head norm + rotary of q and k, k and v into the cache
+//   llmopt_head_norm_gate_{bf16,f32}       per-head norm of a mixer's read-out times its gate
+//   llmopt_argmax_f32, llmopt_advance_tokens   greedy pick and the step's bookkeeping on the device
+#include "element.cuh"
+
+namespace llmopt {
+namespace {
+
+// ---- embedding ---------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) embedding_residual_kernel(const long long* ids, const T* __restrict__ table,
+                                                                 float* x, T* x_copy, uint32_t rows, uint32_t vocabulary,
+                                                                 uint32_t width) {
+  grid_chain_prologue();
+  const uint32_t row = blockIdx.x;
+  const size_t token = min((unsigned long long)ids[row], (unsigned long long)(vocabulary - 1u));
+  for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) {
+    const T value = table[token * width + c];
+    x[(size_t)row * width + c] = as_float(value);
+    if (sizeof(T) != 4) x_copy[(size_t)row * width + c] = value;
+  }
+}
+
+template <typename T>
+int launch_embedding_residual(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == 12,
+                 "expects buffers [ids, table, x, x copy] and 12 parameter bytes {rows, vocabulary, width}");
+  const uint32_t rows = param_u32(args, 0), vocabulary = param_u32(args, 1), width = param_u32(args, 2);
+  LLMOPT_REQUIRE(vocabulary > 0 && width > 0, "needs a vocabulary and a width");
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)rows * 8 && args.lengths[1] >= (size_t)vocabulary * width * sizeof(T) &&
+                     args.lengths[2] >= (size_t)rows * width * 4 && args.lengths[3] >= (size_t)rows * width * sizeof(T),
+                 "buffer is too short");
+  if (rows == 0) return 0;
+  launch_kernel(args, embedding_residual_kernel<T>, dim3(rows), dim3(256), 0, (const long long*)args.buffers[0],
+                (const T*)args.buffers[1], (float*)args.buffers[2], (T*)args.buffers[3], rows, vocabulary, width);
+  return check_launch(args);
+}
+
+// ---- residual + norm ---------------------------------------------------------------------------
+struct ResidualNormParams {
+  uint32_t rows, width;
+  float epsilon, weight_offset;  // the norm multiplies by weight_offset + weight
+  uint32_t pair;                 // 1: y is the mean of two branches, each RMS-normed with its own weight
+};
+
+// One CTA per row; a thread keeps up to V float4 of the row in registers between the passes.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) residual_norm_kernel(const float* x_in, const float* y, const float* __restrict__ w,
+                                                            const float* y2, const float* __restrict__ w_left,
+                                                            const float* __restrict__ w_right, float* x_out, T* x_copy,
+                                                            ResidualNormParams p) {
+  grid_chain_prologue();
+  __shared__ float scratch[8];
+  const size_t base = (size_t)blockIdx.x * p.width;
+  const uint32_t vectors = p.width / 4u;
+  float4 value[V];
+  auto square = [](const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+  float sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const uint32_t at = threadIdx.x + i * 256u;
+    value[i] = at < vectors ? reinterpret_cast<const float4*>(y + base)[at] : make_float4(0.f, 0.f, 0.f, 0.f);
+    sum += square(value[i]);
+  }
+  if (p.pair) {
+    float4 other[V];
+    float other_sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const uint32_t at = threadIdx.x + i * 256u;
+      other[i] = at < vectors ? reinterpret_cast<const float4*>(y2 + base)[at] : make_float4(0.f, 0.f, 0.f, 0.f);
+      other_sum += square(other[i]);
+    }
+    const float left = 0.5f / sqrtf(block_sum(sum, scratch) / (float)p.width + p.epsilon);
+    const float right = 0.5f / sqrtf(block_sum(other_sum, scratch) / (float)p.width + p.epsilon);
+    sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const uint32_t at = threadIdx.x + i * 256u;
+      if (at < vectors) {
+        const float4 wl = reinterpret_cast<const float4*>(w_left)[at], wr = reinterpret_cast<const float4*>(w_right)[at];
+        value[i].x = value[i].x * left * wl.x + other[i].x * right * wr.x;
+        value[i].y = value[i].y * left * wl.y + other[i].y * right * wr.y;
+        value[i].z = value[i].z * left * wl.z + other[i].z * right * wr.z;
+        value[i].w = value[i].w * left * wl.w + other[i].w * right * wr.w;
+      }
+      sum += square(value[i]);
+    }
+  }
+  const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)p.width + p.epsilon);
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const uint32_t at = threadIdx.x + i * 256u;
+    if (at >= vectors) continue;
+    const float4 weight = reinterpret_cast<const float4*>(w)[at];
+    float4 x = reinterpret_cast<const float4*>(x_in + base)[at];
+    x.x += value[i].x * scale * (p.weight_offset + weight.x);
+    x.y += value[i].y * scale * (p.weight_offset + weight.y);
+    x.z += value[i].z * scale * (p.weight_offset + weight.z);
+    x.w += value[i].w * scale * (p.weight_offset + weight.w);
+    reinterpret_cast<float4*>(x_out + base)[at] = x;
+    if (sizeof(T) != 4) {
+      const __nv_bfloat162 low = __floats2bfloat162_rn(x.x, x.y), high = __floats2bfloat162_rn(x.z, x.w);
+      uint2 packed = make_uint2(*reinterpret_cast<const uint32_t*>(&low), *reinterpret_cast<const uint32_t*>(&high));
+      reinterpret_cast<uint2*>(x_copy + base)[at] = packed;
+    }
+  }
+}
+
+// Any width: the row is read again in every pass.
+template <typename T>
+__global__ void __launch_bounds__(256) residual_norm_any_kernel(const float* x_in, const float* y,
+                                                                const float* __restrict__ w, const float* y2,
+                                                                const float* __restrict__ w_left,
+                                                                const float* __restrict__ w_right, float* x_out, T* x_copy,
+                                                                ResidualNormParams p) {
+  grid_chain_prologue();
+  __shared__ float scratch[8];
+  const size_t base = (size_t)blockIdx.x * p.width;
+  float left = 0.0f, right = 0.0f;
+  auto at = [&](uint32_t c) {
+    return p.pair ? y[base + c] * left * w_left[c] + y2[base + c] * right * w_right[c] : y[base + c];
+  };
+  if (p.pair) {
+    float a = 0.0f, b = 0.0f;
+    for (uint32_t c = threadIdx.x; c < p.width; c += 256u) {
+      a += y[base + c] * y[base + c];
+      b += y2[base + c] * y2[base + c];
+    }
+    left = 0.5f / sqrtf(block_sum(a, scratch) / (float)p.width + p.epsilon);
+    right = 0.5f / sqrtf(block_sum(b, scratch) / (float)p.width + p.epsilon);
+  }
+  float sum = 0.0f;
+  for (uint32_t c = threadIdx.x; c < p.width; c += 256u) {
+    const float v = at(c);
+    sum += v * v;
+  }
+  const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)p.width + p.epsilon);
+  for (uint32_t c = threadIdx.x; c < p.width; c += 256u) {
+    const float x = x_in[base + c] + at(c) * scale * (p.weight_offset + w[c]);
+    x_out[base + c] = x;
+    if (sizeof(T) != 4) x_copy[base + c] = from_float<T>(x);
+  }
+}
+
+// Buffers [x in, y, weight, y of the second branch, left weight, right weight, x out, x copy].
+template <typename T>
+int launch_residual_norm(const KernelArgs& args) {
+  ResidualNormParams p;
+  LLMOPT_REQUIRE(args.buffer_count == 8 && args.param_bytes == sizeof(p), "expects 8 buffers and 20 parameter bytes");
+  memcpy(&p, args.params, sizeof(p));
+  const size_t row_bytes = (size_t)p.rows * p.width * 4;
+  LLMOPT_REQUIRE(p.width > 0, "needs a width");
+  LLMOPT_REQUIRE(args.lengths[0] >= row_bytes && args.lengths[1] >= row_bytes && args.lengths[6] >= row_bytes &&
+                     args.lengths[7] >= row_bytes / 4 * sizeof(T) && args.lengths[2] >= (size_t)p.width * 4,
+                 "buffer is too short");
+  LLMOPT_REQUIRE(!p.pair || (args.lengths[3] >= row_bytes && args.lengths[4] >= (size_t)p.width * 4 &&
+                             args.lengths[5] >= (size_t)p.width * 4),
+                 "branch buffer is too short");
+  if (p.rows == 0) return 0;
+  auto run = [&](auto kernel) {
+    launch_kernel(args, kernel, dim3(p.rows), dim3(256), 0, (const float*)args.buffers[0], (const float*)args.buffers[1],
+                  (const float*)args.buffers[2], (const float*)args.buffers[3], (const float*)args.buffers[4],
+                  (const float*)args.buffers[5], (float*)args.buffers[6], (T*)args.buffers[7], p);
+  };
+  bool vectors = p.width % 4u == 0 && p.width <= 8192u;
+  for (int i = 0; i < 8; ++i)
+    if ((uintptr_t)args.buffers[i] & 15u) vectors = false;
+  if (!vectors) run(residual_norm_any_kernel<T>);
+  else if (p.width <= 1024u) run(residual_norm_kernel<T, 1>);
+  else if (p.width <= 2048u) run(residual_norm_kernel<T, 2>);
+  else if (p.width <= 4096u) run(residual_norm_kernel<T, 4>);
+  else run(residual_norm_kernel<T, 8>);
+  return check_launch(args);
+}
+
+// ---- norm of chosen rows -----------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) gather_norm_kernel(const float* x, const uint32_t* rows, const float* __restrict__ w,
+                                                          T* out, uint32_t source_rows, uint32_t width, float epsilon,
+                                                          float weight_offset) {
+  grid_chain_prologue();
+  __shared__ float scratch[8];
+  const float* source = x + (size_t)min(rows[blockIdx.x], source_rows - 1u) * width;
+  float sum = 0.0f;
+  for (uint32_t c = threadIdx.x; c < width; c += 256u) sum += source[c] * source[c];
+  const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + epsilon);
+  for (uint32_t c = threadIdx.x; c < width; c += 256u)
+    out[(size_t)blockIdx.x * width + c] = from_float<T>(source[c] * scale * (weight_offset + w[c]));
+}
+
+// Buffers [x, rows u32, weight, out]; params {count, source rows, width, epsilon, weight offset}.
+template <typename T>
+int launch_gather_norm(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == 20, "expects 4 buffers and 20 parameter bytes");
+  const uint32_t count = param_u32(args, 0), source_rows = param_u32(args, 1), width = param_u32(args, 2);
+  LLMOPT_REQUIRE(source_rows > 0 && width > 0, "needs source rows and a width");
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)source_rows * width * 4 && args.lengths[1] >= (size_t)count * 4 &&
+                     args.lengths[2] >= (size_t)width * 4 && args.lengths[3] >= (size_t)count * width * sizeof(T),
+                 "buffer is too short");
+  if (count == 0) return 0;
+  launch_kernel(args, gather_norm_kernel<T>, dim3(count), dim3(256), 0, (const float*)args.buffers[0],
+                (const uint32_t*)args.buffers[1], (const float*)args.buffers[2], (T*)args.buffers[3], source_rows, width,
+                param_f32(args, 3), param_f32(args, 4));
+  return check_launch(args);
+}
+
+// ---- attention inputs --------------------------------------------------------------------------
+struct AttentionPrepareParams {
+  uint32_t sequences, tokens, heads, kv_heads, dim, vdim;
+  uint32_t stride;                        // elements per row of the projections
+  uint32_t q_column, k_column, v_column;  // first column of each
+  uint32_t rotary_dims, trig_rows;
+  uint32_t token_stride, key_offset, value_offset;  // cache row, in elements
+  uint32_t table_stride, table_rows, pool_rows;
+  uint32_t head_norm;
+  float epsilon;
+};
+
+// One warp per (row, head): query heads are normed, rotated and stored; key heads too, into the
+// cache row of the token; value heads are copied there.  Dimensions 2i, 2i + 1 turn together; `trig`
+// holds [positions][dims / 2] pairs (cos, sin).
+template <typename T>
+__global__ void __launch_bounds__(128) attention_prepare_kernel(const T* projected, const float* __restrict__ q_weight,
+                                                                const float* __restrict__ k_weight,
+                                                                const float2* __restrict__ trig, T* q_out, T* pool,
+                                                                const uint32_t* slots, const uint32_t* past,
+                                                                const uint32_t* sequence_rows, AttentionPrepareParams p,
+                                                                uint32_t* error_word) {
+  grid_chain_prologue();
+  const uint32_t lane = threadIdx.x & 31u, item = blockIdx.x * 4u + (threadIdx.x >> 5);
+  const uint32_t per_row = p.heads + 2u * p.kv_heads;
+  if (item >= p.sequences * p.tokens * per_row) return;
+  const uint32_t row = item / per_row, head = item % per_row, sequence = row / p.tokens;
+  const uint32_t position = past[sequence] + row % p.tokens;
+  const T* source = projected + (size_t)row * p.stride;
+  if (head < p.heads) source += p.q_column + head * p.dim;
+  else if (head < p.heads + p.kv_heads) source += p.k_column + (head - p.heads) * p.dim;
+  else source += p.v_column + (head - p.heads - p.kv_heads) * p.vdim;
+
+  T* target;
+  if (head < p.heads) {
+    target = q_out + ((size_t)row * p.heads + head) * p.dim;
+  } else {
+    const uint32_t table_row = sequence_rows[sequence];
+    uint32_t slot = p.pool_rows;
+    if (table_row < p.table_rows && position < p.table_stride) slot = slots[(size_t)table_row * p.table_stride + position];
+    if (slot >= p.pool_rows) {  // never write outside the pool
+      if (error_word && lane == 0) atomicExch(error_word, 1u);
+      return;
+    }
+    target = pool + (size_t)slot * p.token_stride;
+    if (head >= p.heads + p.kv_heads) {
+      target += p.value_offset + (head - p.heads - p.kv_heads) * p.vdim;
+      for (uint32_t c = lane; c < p.vdim; c += 32u) target[c] = source[c];
+      return;
+    }
+    target += p.key_offset + (head - p.heads) * p.dim;
+  }
+  const float* weight = head < p.heads ? q_weight : k_weight;
+  float scale = 1.0f;
+  if (p.head_norm) {
+    float sum = 0.0f;
+    for (uint32_t c = lane; c < p.dim; c += 32u) {
+      const float v = as_float(source[c]);
+      sum += v * v;
+    }
+    scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
+  }
+  const uint32_t trig_row = min(position, p.trig_rows - 1u);
+  for (uint32_t pair = lane; pair * 2u < p.dim; pair += 32u) {
+    const uint32_t c = pair * 2u;
+    float u = as_float(source[c]) * scale, v = c + 1u < p.dim ? as_float(source[c + 1u]) * scale : 0.0f;
+    if (p.head_norm) {
+      u *= weight[c];
+      if (c + 1u < p.dim) v *= weight[c + 1u];
+    }
+    if (c + 1u < p.rotary_dims) {
+      const float2 turn = trig[(size_t)trig_row * (p.rotary_dims / 2u) + pair];
+      const float rotated = u * turn.x - v * turn.y;
+      v = v * turn.x + u * turn.y;
+      u = rotated;
+    }
+    target[c] = from_float<T>(u);
+    if (c + 1u < p.dim) target[c + 1u] = from_float<T>(v);
+  }
+}
+
+}  // namespace
+uint32_t* context_device_error(Context* ctx);
+namespace {
+
+// Buffers [projected, q weight, k weight, trig, q out, pool, slot table, past, sequence rows].
+template <typename T>
+int launch_attention_prepare(const KernelArgs& args) {
+  AttentionPrepareParams p;
+  LLMOPT_REQUIRE(args.buffer_count == 9 && args.param_bytes == sizeof(p), "expects 9 buffers and 80 parameter bytes");
+  memcpy(&p, args.params, sizeof(p));
+  const size_t rows = (size_t)p.sequences * p.tokens, e = sizeof(T);
+  LLMOPT_REQUIRE(p.heads > 0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.dim > 0 && p.vdim > 0,
+                 "needs whole groups of query heads");
+  LLMOPT_REQUIRE(p.rotary_dims <= p.dim && p.rotary_dims % 2u == 0, "rotated dimensions come in pairs inside the head");
+  LLMOPT_REQUIRE(p.q_column + p.heads * p.dim <= p.stride && p.k_column + p.kv_heads * p.dim <= p.stride &&
+                     p.v_column + p.kv_heads * p.vdim <= p.stride,
+                 "projection columns lie outside the row");
+  LLMOPT_REQUIRE(p.key_offset + p.kv_heads * p.dim <= p.token_stride && p.value_offset + p.kv_heads * p.vdim <= p.token_stride,
+                 "key or value segment lies outside the cache row");
+  LLMOPT_REQUIRE(args.lengths[0] >= rows * p.stride * e && args.lengths[4] >= rows * p.heads * p.dim * e, "buffer is too short");
+  LLMOPT_REQUIRE(!p.head_norm || (args.lengths[1] >= (size_t)p.dim * 4 && args.lengths[2] >= (size_t)p.dim * 4),
+                 "head norm weight is too short");
+  LLMOPT_REQUIRE(p.rotary_dims == 0 || (p.trig_rows > 0 && args.lengths[3] >= (size_t)p.trig_rows * p.rotary_dims * 4),
+                 "trig table is too short");
+  LLMOPT_REQUIRE(args.lengths[5] >= (size_t)p.pool_rows * p.token_stride * e &&
+                     args.lengths[6] >= (size_t)p.table_rows * p.table_stride * 4 &&
+                     args.lengths[7] >= (size_t)p.sequences * 4 && args.lengths[8] >= (size_t)p.sequences * 4,
+                 "cache buffer is too short");
+  if (rows == 0) return 0;
+  const size_t items = rows * (p.heads + 2u * p.kv_heads);
+  launch_kernel(args, attention_prepare_kernel<T>, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0,
+                (const T*)args.buffers[0], (const float*)args.buffers[1], (const float*)args.buffers[2],
+                (const float2*)args.buffers[3], (T*)args.buffers[4], (T*)args.buffers[5], (const uint32_t*)args.buffers[6],
+                (const uint32_t*)args.buffers[7], (const uint32_t*)args.buffers[8], p, context_device_error(args.ctx));
+  return check_launch(args);
+}
+
+// ---- per-head norm and gate of a mixer's read-out ---------------------------------------------
+struct HeadNormGateParams {
+  uint32_t rows, heads, dim;
+  uint32_t gate_stride, gate_column;
+  uint32_t weight_per_head;  // 1: weight [heads * dim]; 0: weight [dim] shared by the heads
+  uint32_t gate_sigmoid;     // 1: sigmoid, 0: silu
+  float epsilon;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* o, const T* gate, const float* __restrict__ weight,
+                                                             T* out, HeadNormGateParams p) {
+  grid_chain_prologue();
+  const uint32_t lane = threadIdx.x & 31u, item = blockIdx.x * 4u + (threadIdx.x >> 5);
+  if (item >= p.rows * p.heads) return;
+  const uint32_t row = item / p.heads, head = item % p.heads;
+  const float* source = o + (size_t)item * p.dim;
+  const T* gate_row = gate + (size_t)row * p.gate_stride + p.gate_column + head * p.dim;
+  float sum = 0.0f;
+  for (uint32_t c = lane; c < p.dim; c += 32u) sum += source[c] * source[c];
+  const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
+  for (uint32_t c = lane; c < p.dim; c += 32u) {
+    const float z = as_float(gate_row[c]);
+    const float w = weight[p.weight_per_head ? head * p.dim + c : c];
+    out[(size_t)item * p.dim + c] = from_float<T>(source[c] * scale * w * (p.gate_sigmoid ? sigmoid_f32(z) : silu_f32(z)));
+  }
+}
+
+// Buffers [o f32, gate, weight, out].
+template <typename T>
+int launch_head_norm_gate(const KernelArgs& args) {
+  HeadNormGateParams p;
+  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == sizeof(p), "expects 4 buffers and 32 parameter bytes");
+  memcpy(&p, args.params, sizeof(p));
+  const size_t items = (size_t)p.rows * p.heads;
+  LLMOPT_REQUIRE(p.gate_column + p.heads * p.dim <= p.gate_stride, "gate columns lie outside the row");
+  LLMOPT_REQUIRE(args.lengths[0] >= items * p.dim * 4 && args.lengths[1] >= (size_t)p.rows * p.gate_stride * sizeof(T) &&
+                     args.lengths[2] >= (size_t)p.dim * (p.weight_per_head ? p.heads : 1u) * 4 &&
+                     args.lengths[3] >= items * p.dim * sizeof(T),
+                 "buffer is too short");
+  if (items == 0) return 0;
+  launch_kernel(args, head_norm_gate_kernel<T>, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0,
+                (const float*)args.buffers[0], (const T*)args.buffers[1], (const float*)args.buffers[2],
+                (T*)args.buffers[3], p);
+  return check_launch(args);
+}
+
+// ---- greedy pick and bookkeeping ----------------------------------------------------------------
+// Larger logits first, then smaller columns, as one unsigned integer.
+__device__ __forceinline__ unsigned long long ranked(float value, uint32_t column) {
+  uint32_t bits = __float_as_uint(value);
+  bits = (bits & 0x80000000u) ? ~bits : bits | 0x80000000u;
+  return ((unsigned long long)bits << 32) | (0xffffffffu - column);
+}
+
+__global__ void __launch_bounds__(256) argmax_kernel(const float* logits, unsigned long long* best, uint32_t columns,
+                                                     uint32_t parts) {
+  grid_chain_prologue();
+  __shared__ unsigned long long warp_best[8];
+  const float* row = logits + (size_t)blockIdx.y * columns;
+  unsigned long long top = 0;
+  for (uint32_t c = blockIdx.x * 256u + threadIdx.x; c < columns; c += parts * 256u) top = max(top, ranked(row[c], c));
+  for (int offset = 16; offset > 0; offset >>= 1) top = max(top, __shfl_xor_sync(0xffffffffu, top, offset));
+  if ((threadIdx.x & 31u) == 0u) warp_best[threadIdx.x >> 5] = top;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    for (int w = 1; w < 8; ++w) top = max(top, warp_best[w]);
+    best[(size_t)blockIdx.y * parts + blockIdx.x] = top;
+  }
+}
+
+// Buffers [logits f32, candidates u64 [rows, parts]]; params {rows, columns, parts}.
+int launch_argmax_f32(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 2 && args.param_bytes == 12, "expects 2 buffers and 12 parameter bytes");
+  const uint32_t rows = param_u32(args, 0), columns = param_u32(args, 1), parts = param_u32(args, 2);
+  LLMOPT_REQUIRE(columns > 0 && parts > 0 && rows <= 65535u, "needs columns, parts and at most 65535 rows");
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)rows * columns * 4 && args.lengths[1] >= (size_t)rows * parts * 8,
+                 "buffer is too short");
+  if (rows == 0) return 0;
+  launch_kernel(args, argmax_kernel, dim3(parts, rows), dim3(256), 0, (const float*)args.buffers[0],
+                (unsigned long long*)args.buffers[1], columns, parts);
+  return check_launch(args);
+}
+
+__global__ void __launch_bounds__(32) advance_kernel(const unsigned long long* best, int* picked, long long* ids,
+                                                     uint32_t* past, uint32_t parts, uint32_t step) {
+  grid_chain_prologue();
+  unsigned long long top = 0;
+  for (uint32_t i = threadIdx.x; i < parts; i += 32u) top = max(top, best[(size_t)blockIdx.x * parts + i]);
+  for (int offset = 16; offset > 0; offset >>= 1) top = max(top, __shfl_xor_sync(0xffffffffu, top, offset));
+  if (threadIdx.x != 0) return;
+  const uint32_t token = 0xffffffffu - (uint32_t)top;
+  picked[blockIdx.x] = (int)token;
+  ids[blockIdx.x] = (long long)token;
+  past[blockIdx.x] += step;
+}
+
+// Ends a step of one row per sequence: the picked token becomes the next input and the sequence has `step`
+// more tokens behind it.  Buffers [candidates, picked i32, ids i64, past u32]; params {rows, parts, step}.
+int launch_advance_tokens(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == 12, "expects 4 buffers and 12 parameter bytes");
+  const uint32_t rows = param_u32(args, 0), parts = param_u32(args, 1), step = param_u32(args, 2);
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)rows * parts * 8 && args.lengths[1] >= (size_t)rows * 4 &&
+                     args.lengths[2] >= (size_t)rows * 8 && args.lengths[3] >= (size_t)rows * 4,
+                 "buffer is too short");
+  if (rows == 0) return 0;
+  launch_kernel(args, advance_kernel, dim3(rows), dim3(32), 0, (const unsigned long long*)args.buffers[0],
+                (int*)args.buffers[1], (long long*)args.buffers[2], (uint32_t*)args.buffers[3], parts, step);
+  return check_launch(args);
+}
+
+}  // namespace
+
+const NamedLauncher* sequence_glue_launchers(size_t* count) {
+  static const NamedLauncher table[] = {
+      {"llmopt_embedding_residual_bf16", launch_embedding_residual<bf16>},
+      {"llmopt_embedding_residual_f32", launch_embedding_residual<float>},
+      {"llmopt_residual_norm_bf16", launch_residual_norm<bf16>},
+      {"llmopt_residual_norm_f32", launch_residual_norm<float>},
+      {"llmopt_gather_norm_bf16", launch_gather_norm<bf16>},
+      {"llmopt_gather_norm_f32", launch_gather_norm<float>},
+      {"llmopt_row_attention_prepare_bf16", launch_attention_prepare<bf16>},
+      {"llmopt_row_attention_prepare_f32", launch_attention_prepare<float>},
+      {"llmopt_head_norm_gate_bf16", launch_head_norm_gate<bf16>},
+      {"llmopt_head_norm_gate_f32", launch_head_norm_gate<float>},
+      {"llmopt_argmax_f32", launch_argmax_f32},
+      {"llmopt_advance_tokens", launch_advance_tokens},
+  };
+  *count = sizeof(table) / sizeof(table[0]);
+  return table;
+}
+
+}  // namespace llmopt

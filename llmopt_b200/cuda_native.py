@@ -112,6 +112,8 @@ SIGNATURES = {
     "llmopt_cuda_f16_argmax": (_I64, [_P, _SZ]),
     "llmopt_cuda_sample_f16": (_I, [_P, _SZ, ctypes.c_double, _I, ctypes.c_double, ctypes.c_double, ctypes.c_uint64,
                                    ctypes.POINTER(_I64)]),
+    "llmopt_cuda_sample_f32": (_I, [_P, _SZ, ctypes.c_double, _I, ctypes.c_double, ctypes.c_double, ctypes.c_uint64,
+                                   ctypes.POINTER(_I64)]),
     "llmopt_cuda_measure_hardware": (_I, [_I, _I, _I, _I64, ctypes.c_char_p, _SZ, ctypes.POINTER(_I),
                                          ctypes.POINTER(ctypes.c_double), ctypes.POINTER(ctypes.c_double)]),
     "llmopt_cuda_w4a16_linear": (_I, [_P, _P, _P, _P, _P, _P, _I64, _I64, _I64, _P]),
@@ -121,8 +123,21 @@ SIGNATURES = {
 }
 
 
+# entry points that belong to a kernel family; a library linked from other families has none of them
+_FAMILY_ENTRY_POINTS = {"llmopt_cuda_attention_q8_paged_static"}
+
+
 def library_path() -> str:
     return _LIBRARY_PATH
+
+
+def use_library(path: str) -> None:
+    """Takes ``path`` (for example the library of one kernel family, ``_build.FAMILIES``) for this process;
+    only before the first use of the native layer."""
+    global _LIBRARY_PATH
+    if _lib is not None and path != _LIBRARY_PATH:
+        raise NativeError(f"{_LIBRARY_PATH} is already loaded")
+    _LIBRARY_PATH = path
 
 
 def load_library() -> ctypes.CDLL:
@@ -134,7 +149,10 @@ def load_library() -> ctypes.CDLL:
                 f"{_LIBRARY_PATH} is missing: build it with `python -m llmopt_b200._build` (nvcc, sm_100a)"
             )
         lib = ctypes.CDLL(_LIBRARY_PATH)
+        partial = os.path.basename(_LIBRARY_PATH) != "libllmopt_cuda.so"
         for name, (restype, argtypes) in SIGNATURES.items():
+            if partial and name in _FAMILY_ENTRY_POINTS:
+                continue
             function = getattr(lib, name)
             function.restype = restype
             function.argtypes = argtypes
@@ -576,6 +594,18 @@ def sample_f16(data: bytes, count: int, *, temperature: float, top_k: int, top_p
     out = ctypes.c_int64()
     _check(load_library().llmopt_cuda_sample_f16(buffer, count, float(temperature), int(top_k), float(top_p),
                                                  float(min_p), int(seed) & 0xFFFFFFFFFFFFFFFF, ctypes.byref(out)))
+    return int(out.value)
+
+
+def sample_f32(logits, *, temperature: float, top_k: int, top_p: float, min_p: float, seed: int) -> int:
+    """The sampler of ``sample_f16`` over one row of fp32 logits (a numpy array)."""
+    import numpy as np
+
+    row = np.ascontiguousarray(logits, np.float32).reshape(-1)
+    out = ctypes.c_int64()
+    _check(load_library().llmopt_cuda_sample_f32(row.ctypes.data_as(ctypes.c_void_p), row.size, float(temperature),
+                                                 int(top_k), float(top_p), float(min_p),
+                                                 int(seed) & 0xFFFFFFFFFFFFFFFF, ctypes.byref(out)))
     return int(out.value)
 
 

@@ -501,3 +501,12 @@ class DecodeEngine:
         for b in range(1, self.batch):
             first.copy_to(self.cache.token_pool.view(b * self.capacity * stride, past_tokens * stride))
         self.runtime.synchronize()
+
+
+def create_engine(runtime: Runtime, config, weights, **options):
+    """The engine that serves a configuration: ``DecodeEngine`` for the W4A16 decoders (``ModelConfig``),
+    ``mixer_engine.MixerEngine`` for decoders composed of sequence mixers (``MixerConfig``)."""
+    from .mixer_engine import MixerEngine
+    from .model import MixerConfig
+
+    return (MixerEngine if isinstance(config, MixerConfig) else DecodeEngine)(runtime, config, weights, **options)

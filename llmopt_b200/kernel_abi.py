@@ -155,6 +155,21 @@ def _entries() -> list[Entry]:
     add("llmopt_embedding_f16", EMBEDDING, i64, f16)
     add("llmopt_chain_token_id", EMBEDDING, i64, i64, (32, 1, 1))
     add("llmopt_chain_token_ids", EMBEDDING, "int32", i64, (128, 1, 1))
+    # sequence-mixer kernels in the model's element type (no reference counterpart)
+    for suffix, element in (("bf16", "bfloat16"), ("f32", f32)):
+        add("llmopt_dense_linear_" + suffix, LINEAR, element, element)
+        add("llmopt_embedding_residual_" + suffix, EMBEDDING, element, f32)
+        add("llmopt_residual_norm_" + suffix, RMS_NORM, f32, element)
+        add("llmopt_gather_norm_" + suffix, RMS_NORM, f32, element)
+        add("llmopt_row_attention_prepare_" + suffix, CACHE, element, element)
+        add("llmopt_row_attention_" + suffix, ATTENTION, element, element)
+        add("llmopt_head_norm_gate_" + suffix, RMS_NORM, f32, element)
+        add("llmopt_delta_prepare_" + suffix, SHORT_CONV, element, f32)
+        add("llmopt_conv_state_" + suffix, SHORT_CONV, element, element)
+        add("llmopt_memory_scan_" + suffix, GATED_DELTA, element, f32)
+    add("llmopt_delta_scan_f32", GATED_DELTA, f32, f32)
+    add("llmopt_argmax_f32", POINTWISE, f32, i64)
+    add("llmopt_advance_tokens", EMBEDDING, i64, "int32")
     return table
 
 

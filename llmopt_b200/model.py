@@ -2,12 +2,21 @@
 Llama-style blocks (RMSNorm, fused QKV, RoPE, GQA attention over the Q8 cache,
 SwiGLU FFN) and LFM-style gated short-conv blocks (lib/lfm25.ml:18-34).  The
 weights are random-init and quantised W4A16 group-64; there is no checkpoint
-loader here — a compiled package brings its own tensors."""
+loader for them here — a compiled package brings its own tensors.
+
+The second part describes decoders composed of sequence mixers (attention over
+unquantised cache rows, gated delta rule, matrix memory, two of them side by side)
+with dense bfloat16 weights, which are read from a folder with a config.json and a
+safetensors checkpoint: ``ARCHITECTURES`` maps the config's architecture name to the
+function that reads it."""
 
 from __future__ import annotations
 
+import importlib
+import json
+import os
 from dataclasses import dataclass, field
-from typing import Sequence
+from typing import Callable, Dict, Optional, Sequence, Tuple, Union
 
 import numpy as np
 
@@ -113,3 +122,220 @@ def decode_bytes_per_token(config: ModelConfig, batch: int, past: int) -> dict:
     kv_per_token = 2 * config.kv_heads * dim + 2 * 2 * config.kv_heads * dim // config.kv_group_size
     attention = config.attention_layers * batch * (past * (kv_per_token + 4))
     return {"weights": weights, "attention": attention, "total": weights + attention + hidden * 2 * batch}
+
+
+# ---- decoders composed of sequence mixers --------------------------------------------------------------
+
+@dataclass(frozen=True)
+class YarnSpec:
+    """Frequencies of slow pairs divided by ``factor``, those of fast pairs kept, a linear ramp between."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """The first ``dims`` dimensions of a head turn, in pairs of neighbours (2i, 2i + 1)."""
+
+    dims: int
+    base: float
+    scaling: Optional[YarnSpec] = None
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: RotarySpec
+    bias: bool = False       # on q, k, v and the output projection
+    head_norm: bool = False  # RMS norm of every query and key head before rotation
+    sink: bool = False       # one more term exp(0) in the softmax denominator
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input; the mean of their outputs, each RMS-normed."""
+
+    left: Union[AttentionSpec, DeltaSpec, MatrixMemorySpec]
+    right: Union[AttentionSpec, DeltaSpec, MatrixMemorySpec]
+
+
+@dataclass(frozen=True)
+class FeedForwardSpec:
+    width: int
+    activation: str = "gelu"
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """Per-layer token input: a table row of ``dim`` per layer, gated by the residual."""
+
+    dim: int
+
+
+@dataclass(frozen=True)
+class MixerLayer:
+    mixer: Union[AttentionSpec, DeltaSpec, MatrixMemorySpec, ParallelSpec]
+    feed_forward: Optional[FeedForwardSpec]
+
+
+@dataclass(frozen=True)
+class MixerConfig:
+    """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), x <- x + norm(token side(x)) per layer; the sublayer
+    norms multiply by ``norm_offset`` + weight."""
+
+    name: str
+    width: int
+    vocabulary: int
+    layers: Tuple[MixerLayer, ...]
+    epsilon: float
+    norm_offset: float = 0.0
+    token_side: Optional[TokenSideSpec] = None
+
+    def __post_init__(self):
+        if self.width <= 0 or self.vocabulary <= 0 or not self.layers:
+            raise ValueError("a model needs a width, a vocabulary and layers")
+        for layer in self.layers:
+            mixers = (layer.mixer.left, layer.mixer.right) if isinstance(layer.mixer, ParallelSpec) else (layer.mixer,)
+            for mixer in mixers:
+                kv_heads = getattr(mixer, "kv_heads", mixer.heads)
+                if min(mixer.heads, kv_heads, mixer.dim, mixer.vdim) <= 0 or mixer.heads % kv_heads:
+                    raise ValueError("query heads must come in whole groups per key/value head")
+                if isinstance(mixer, AttentionSpec) and (mixer.rotary.dims % 2 or mixer.rotary.dims > mixer.dim):
+                    raise ValueError("rotated dimensions come in pairs inside the head")
+
+
+ARCHITECTURES: Dict[str, Callable[[dict], MixerConfig]] = {}
+# the module that registers each architecture, imported when it is first asked for
+ARCHITECTURE_MODULES = {"Bizodra": "bizodra"}
+
+
+def register_architecture(name: str):
+    def register(parse):
+        ARCHITECTURES[name] = parse
+        return parse
+    return register
+
+
+def parse_config(config: dict) -> MixerConfig:
+    name = config.get("architecture")
+    if name in ARCHITECTURE_MODULES:
+        importlib.import_module("." + ARCHITECTURE_MODULES[name], __package__)
+    if name not in ARCHITECTURES:
+        raise ValueError(f"unsupported architecture: {name}")
+    return ARCHITECTURES[name](config)
+
+
+def load_model(folder: str):
+    """(configuration, weights) of a folder with config.json and model.safetensors."""
+    from .safetensors_archive import Archive
+
+    with open(os.path.join(folder, "config.json")) as source:
+        config = parse_config(json.load(source))
+    return config, Archive(os.path.join(folder, "model.safetensors"))
+
+
+def mixer_tensors(config: MixerConfig) -> Dict[str, tuple]:
+    """Name and shape of every tensor of a checkpoint."""
+    width, shapes = config.width, {}
+    shapes["embed"] = (config.vocabulary, width)
+    if config.token_side:
+        shapes["side.embed"] = (config.vocabulary, len(config.layers) * config.token_side.dim)
+
+    def mixer(prefix, spec):
+        if isinstance(spec, ParallelSpec):
+            for side, one in (("left", spec.left), ("right", spec.right)):
+                mixer(f"{prefix}.{side}", one)
+                shapes[f"{prefix}.{side}.out"] = (width,)
+            return
+        heads, kv_heads = spec.heads, getattr(spec, "kv_heads", spec.heads)
+        query_heads = kv_heads if isinstance(spec, DeltaSpec) else heads
+        value_heads = heads if isinstance(spec, DeltaSpec) else kv_heads
+        for name, rows in (("q", query_heads * spec.dim), ("k", kv_heads * spec.dim), ("v", value_heads * spec.vdim)):
+            shapes[f"{prefix}.{name}"] = (rows, width)
+        shapes[f"{prefix}.o"] = (width, heads * spec.vdim)
+        if isinstance(spec, AttentionSpec):
+            if spec.bias:
+                for name in "qkvo":
+                    shapes[f"{prefix}.{name}.b"] = shapes[f"{prefix}.{name}"][:1]
+            if spec.head_norm:
+                shapes[f"{prefix}.q.norm"] = shapes[f"{prefix}.k.norm"] = (spec.dim,)
+            return
+        shapes[f"{prefix}.g"] = (heads * spec.vdim, width)
+        if isinstance(spec, DeltaSpec):
+            for name in "qkv":
+                shapes[f"{prefix}.{name}.conv"] = (shapes[f"{prefix}.{name}"][0], spec.taps)
+            shapes[f"{prefix}.b"] = shapes[f"{prefix}.a"] = (heads, width)
+            shapes[f"{prefix}.A_log"] = shapes[f"{prefix}.dt_bias"] = (heads,)
+            shapes[f"{prefix}.norm"] = (spec.vdim,)
+        else:
+            shapes[f"{prefix}.norm"] = (heads * spec.vdim,)
+            for name in "if":
+                shapes[f"{prefix}.{name}"] = (heads, width)
+                shapes[f"{prefix}.{name}.b"] = (heads,)
+
+    for index, layer in enumerate(config.layers):
+        shapes[f"l{index}.norm1"] = (width,)
+        mixer(f"l{index}.mix", layer.mixer)
+        if layer.feed_forward:
+            shapes[f"l{index}.norm2"] = (width,)
+            shapes[f"l{index}.mlp.up"] = (layer.feed_forward.width, width)
+            shapes[f"l{index}.mlp.down"] = (width, layer.feed_forward.width)
+        if config.token_side:
+            shapes[f"l{index}.side.gate"] = (config.token_side.dim, width)
+            shapes[f"l{index}.side.proj"] = (width, config.token_side.dim)
+            shapes[f"l{index}.side.norm"] = (width,)
+    shapes["final.norm"] = (width,)
+    shapes["head"] = (config.vocabulary, width)
+    return shapes
+
+
+def random_mixer_weights(config: MixerConfig, seed: int = 0, std: float = 0.02) -> Dict[str, np.ndarray]:
+    """Random-init weights under the checkpoint's names, as bfloat16 bits; matrices N(0, std), norm weights
+    near the value that leaves a vector as it is, decays of a few to a few hundred tokens."""
+    from .safetensors_archive import as_bfloat16_bits
+
+    rng = np.random.default_rng(seed)
+    weights = {}
+    for name, shape in mixer_tensors(config).items():
+        leaf = name.rsplit(".", 1)[-1]
+        offset = config.norm_offset if leaf in ("norm1", "norm2") or name == "final.norm" else 0.0
+        if leaf in ("norm1", "norm2", "norm", "out"):
+            value = rng.uniform(0.8, 1.2, size=shape) - offset
+        elif leaf == "A_log":
+            value = np.log(rng.uniform(1.0, 8.0, size=shape))
+        elif leaf == "dt_bias":
+            value = np.log(np.expm1(np.exp(rng.uniform(np.log(1e-3), np.log(0.1), size=shape))))
+        elif name.endswith(".f.b"):
+            value = rng.uniform(3.0, 6.0, size=shape)
+        elif leaf == "conv":
+            value = rng.standard_normal(shape) * 0.5
+        elif leaf == "b" and len(shape) == 1:
+            value = rng.standard_normal(shape) * 0.1
+        else:
+            value = rng.standard_normal(shape, dtype=np.float32) * np.float32(std)
+        weights[name] = as_bfloat16_bits(np.asarray(value, np.float32))
+    return weights

@@ -162,3 +162,52 @@ def pointwise(*, output_shape, left_shape=None, right_shape=None, left_scalar=No
                          float(right_scalar or 0.0))
     assert len(block) == 136
     return bytes(block)
+
+
+# ---- sequence-mixer kernels (no reference counterpart; layouts of csrc/dense_linear.cu, sequence_glue.cu,
+# ---- row_attention.cu and matrix_state.cu) ---------------------------------------------------------------
+
+DENSE_EPILOGUES = {None: 0, "gelu": 1, "token_gate": 2}
+
+
+def dense_linear(*, m, n, k, split, has_bias=False, epilogue=None, table_rows=0, table_stride=0, table_offset=0) -> bytes:
+    return u32s([m, n, k, split, 1 if has_bias else 0, DENSE_EPILOGUES[epilogue], table_rows, table_stride, table_offset])
+
+
+def residual_norm(*, rows, width, epsilon, weight_offset, pair=False) -> bytes:
+    return struct.pack("<IIffI", _u32(rows), _u32(width), epsilon, weight_offset, 1 if pair else 0)
+
+
+def gather_norm(*, count, source_rows, width, epsilon, weight_offset) -> bytes:
+    return struct.pack("<IIIff", _u32(count), _u32(source_rows), _u32(width), epsilon, weight_offset)
+
+
+def row_attention_prepare(*, sequences, tokens, heads, kv_heads, dim, vdim, stride, q_column, k_column, v_column,
+                          rotary_dims, trig_rows, token_stride, key_offset, value_offset, table_stride, table_rows,
+                          pool_rows, head_norm, epsilon) -> bytes:
+    return u32s([sequences, tokens, heads, kv_heads, dim, vdim, stride, q_column, k_column, v_column, rotary_dims,
+                 trig_rows, token_stride, key_offset, value_offset, table_stride, table_rows, pool_rows,
+                 1 if head_norm else 0]) + struct.pack("<f", epsilon)
+
+
+def row_attention(*, sequences, tokens, heads, kv_heads, dim, vdim, token_stride, key_offset, value_offset, table_stride,
+                  table_rows, pool_rows, sink, splits, scale) -> bytes:
+    return u32s([sequences, tokens, heads, kv_heads, dim, vdim, token_stride, key_offset, value_offset, table_stride,
+                 table_rows, pool_rows, 1 if sink else 0, splits]) + struct.pack("<f", scale)
+
+
+def head_norm_gate(*, rows, heads, dim, gate_stride, gate_column, weight_per_head, gate_sigmoid, epsilon) -> bytes:
+    return u32s([rows, heads, dim, gate_stride, gate_column, 1 if weight_per_head else 0,
+                 1 if gate_sigmoid else 0]) + struct.pack("<f", epsilon)
+
+
+def delta_prepare(*, sequences, tokens, heads, kv_heads, dim, vdim, taps, stride, q_column, k_column, v_column,
+                  scalar_stride, beta_column, decay_column, state_rows) -> bytes:
+    return u32s([sequences, tokens, heads, kv_heads, dim, vdim, taps, stride, q_column, k_column, v_column, scalar_stride,
+                 beta_column, decay_column, state_rows])
+
+
+def state_scan(*, sequences, tokens, heads, kv_heads, dim, vdim, q_stride, q_column, k_stride, k_column, v_stride,
+               v_column, scalar_stride, first_column, second_column, state_rows, state_stride, gate_cap=0.0) -> bytes:
+    return u32s([sequences, tokens, heads, kv_heads, dim, vdim, q_stride, q_column, k_stride, k_column, v_stride, v_column,
+                 scalar_stride, first_column, second_column, state_rows, state_stride]) + struct.pack("<f", gate_cap)

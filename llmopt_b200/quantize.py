@@ -56,6 +56,26 @@ def rope_tables(positions: int, head_dim: int, theta: float):
     return np.concatenate([cosine, cosine], axis=1), np.concatenate([sine, sine], axis=1)
 
 
+def rotary_pairs(positions: int, rotary) -> np.ndarray:
+    """f32 [positions, dims / 2, 2]: cos and sin of every pair's angle (a ``model.RotarySpec``), computed in
+    double precision; with YaRN scaling the slow pairs turn ``factor`` times slower, with a linear ramp
+    between the pairs that make ``fast`` and ``slow`` turns over the original length, and both
+    functions are scaled by 0.1 ln(factor) + 1."""
+    dims = rotary.dims
+    pair = np.arange(dims // 2, dtype=np.float64)
+    frequency, magnitude = rotary.base ** (-2.0 * pair / dims), 1.0
+    if rotary.scaling is not None:
+        scaling = rotary.scaling
+        turning = lambda turns: dims * np.log(scaling.original / (2.0 * np.pi * turns)) / (2.0 * np.log(rotary.base))
+        low = max(np.floor(turning(scaling.fast)), 0.0)
+        high = min(np.ceil(turning(scaling.slow)), dims - 1.0)
+        ramp = np.clip((pair - low) / max(high - low, 0.001), 0.0, 1.0)
+        frequency = frequency * (ramp / scaling.factor + (1.0 - ramp))
+        magnitude = 0.1 * np.log(scaling.factor) + 1.0
+    angle = np.arange(positions, dtype=np.float64)[:, None] * frequency[None, :]
+    return np.stack([magnitude * np.cos(angle), magnitude * np.sin(angle)], axis=-1).astype(np.float32)
+
+
 def q4_0_blocks(scales, nibbles):
     """Q4_0 weight rows from fp16 block scales [n, k/32] and nibbles 0..15 [n, k]
     (element i of a block in the low nibble of byte i for i < 16, in the high nibble of

@@ -96,9 +96,11 @@ def test_kernel_abi_surface():
     with pytest.raises(ValueError):
         kernel_abi.Entry("", kernel_abi.CACHE, "float16", "uint8")
     # every entry name is registered in the native library's table (checked textually: no GPU here)
-    source = open(os.path.join(ROOT, "llmopt_b200", "csrc", "runtime.cu")).read()
-    family = open(os.path.join(ROOT, "llmopt_b200", "csrc", "norm_family.cu")).read()  # its own name table
-    registered = set(re.findall(r'"(llmopt_[a-z0-9_]+)"', source + family))
+    # families that keep their own name table are registered from it
+    csrc = os.path.join(ROOT, "llmopt_b200", "csrc")
+    sources = [os.path.join(csrc, name + ".cu") for name in ("runtime", "norm_family", "dense_linear", "sequence_glue",
+                                                             "row_attention", "matrix_state")]
+    registered = set(re.findall(r'"(llmopt_[a-z0-9_]+)"', "".join(open(path).read() for path in sources)))
     assert {e.name for e in kernel_abi.ENTRIES} <= registered
 
 
