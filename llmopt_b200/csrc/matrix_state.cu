@@ -10,20 +10,22 @@
 // columns, because every slice's CTA needs them and keeps a copy of its own.  A sequence with nothing
 // behind it (past = 0) starts from zero whatever its pool row holds.
 //
-// Scan: a CTA owns kSlice value columns of one head of one sequence and walks over the tokens.  Eight lanes
-// share a column of S (each dim / 8 rows of it, in registers).  Compute warps work on a chunk of tokens in
+// Scan: a CTA owns kSlice value columns of one head of one sequence and walks over the tokens.  Sixteen lanes
+// share two columns of S (each lane dim / 16 rows of them, in registers).  Compute warps work on a chunk of tokens in
 // shared memory while producer warps bring in the next chunk (converted to fp32, with the per-token
 // scalars) and write out the previous one's results.  The read-out of the delta rule uses
 // S_new^T q = g S_old^T q + u (k . q), so that its sum and the one of S_old^T k are reduced at the same time.
+#include <type_traits>
+
 #include "element.cuh"
 
 namespace llmopt {
 namespace {
 
-constexpr uint32_t kSlice = 16;        // value columns per CTA
-constexpr uint32_t kLanes = 8;         // lanes per column
-constexpr uint32_t kChunk = 32;        // tokens per chunk
-constexpr uint32_t kColumnWarps = kSlice * kLanes / 32;  // 4
+constexpr uint32_t kSlice = 32;   // value columns per CTA
+constexpr uint32_t kLanes = 16;   // lanes per column
+constexpr uint32_t kColumns = 2;  // columns per thread
+constexpr uint32_t kColumnWarps = kSlice / kColumns * kLanes / 32;  // 4
 constexpr uint32_t kProducerWarps = 4;
 
 __host__ __device__ constexpr uint32_t slices_of(uint32_t vdim) { return (vdim + kSlice - 1u) / kSlice; }
@@ -224,23 +226,49 @@ struct StateRow {
 };
 
 // One chunk's inputs and results in shared memory.
-template <int R4>
+template <int R4, int CHUNK>
 struct ScanChunk {
-  float q[kChunk][R4 * 32], k[kChunk][R4 * 32];
-  float v[kChunk][kSlice];
-  float out[kChunk][kSlice];
-  float first[kChunk], second[kChunk];  // delta: decay, beta; memory: keep, write
-  float extra[kChunk];                  // delta: k . q; memory: exp(-m)
-  float norm_dot[kChunk];               // memory: n . q
+  float q[CHUNK][R4 * kLanes * 4], k[CHUNK][R4 * kLanes * 4];
+  float v[CHUNK][kSlice];
+  float out[CHUNK][kSlice];
+  float4 scalar[CHUNK];   // delta: decay, beta, k . q; memory: keep, write, exp(-m)
+  float norm_dot[CHUNK];  // memory: n . q
 };
+
+// Tokens whose read-outs are reduced together (a chunk's tokens are padded to a whole group with tokens that
+// leave the state as it is).
+template <int CHUNK> struct ScanGroup { static constexpr uint32_t kTokens = CHUNK >= 8 ? 4 : 1; };
 
 template <bool MEMORY> struct ScanThreads {
   static constexpr uint32_t kCompute = (kColumnWarps + (MEMORY ? 1u : 0u)) * 32u;  // one more warp carries n
   static constexpr uint32_t kAll = kCompute + kProducerWarps * 32u;
 };
 
+// Two fp32 numbers in one register pair (Blackwell's packed fp32 arithmetic).
+typedef unsigned long long Pair;
+__device__ __forceinline__ Pair pair_of(float low, float high) {
+  Pair d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(low), "f"(high));
+  return d;
+}
+__device__ __forceinline__ Pair pair_fma(Pair a, Pair b, Pair c) {
+  Pair d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ Pair pair_mul(Pair a, Pair b) {
+  Pair d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ float pair_sum(Pair a) {
+  float low, high;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(a));
+  return low + high;
+}
+
 // TQ: element of q, k, v (fp32 for the delta rule, whose unit vectors are fp32).
-template <typename TQ, bool MEMORY, int R4>
+template <typename TQ, bool MEMORY, int R4, int CHUNK>
 __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const TQ* query, const TQ* key, const TQ* value,
                                                                          const float* first, const float* second,
                                                                          float* state_pool, const uint32_t* past,
@@ -248,7 +276,8 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
                                                                          ScanParams p) {
   grid_chain_prologue();
   extern __shared__ __align__(16) unsigned char scan_shared[];
-  ScanChunk<R4>* chunks = reinterpret_cast<ScanChunk<R4>*>(scan_shared);
+  typedef ScanChunk<R4, CHUNK> Chunk;
+  Chunk* chunks = reinterpret_cast<Chunk*>(scan_shared);
   constexpr uint32_t kCompute = ScanThreads<MEMORY>::kCompute;
   const uint32_t slice = blockIdx.x, head = blockIdx.y, sequence = blockIdx.z;
   const uint32_t kv_head = head / (p.heads / p.kv_heads);
@@ -256,7 +285,7 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
   const bool fresh = past[sequence] == 0;
   float* state = state_pool + (size_t)min(sequence_rows[sequence], p.state_rows - 1u) * p.state_stride;
   const StateRow layout = {p.heads, p.dim, p.vdim};
-  const uint32_t chunk_count = (p.tokens + kChunk - 1u) / kChunk;
+  const uint32_t chunk_count = (p.tokens + CHUNK - 1u) / CHUNK;
 
   if (threadIdx.x >= kCompute) {
     // ------------------------------ producers ------------------------------
@@ -264,29 +293,57 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
     const float q_scale = MEMORY ? 1.0f / sqrtf((float)p.dim) : 1.0f;
     float top = 0.0f;  // memory form: running maximum (warp 0)
     if (MEMORY && !fresh) top = state[layout.top(head, slice)];
+    const uint32_t value_column = slice * kSlice + lane;
     auto produce = [&](uint32_t index) {
-      ScanChunk<R4>& chunk = chunks[index & 1u];
-      const uint32_t t0 = index * kChunk, count = min(kChunk, p.tokens - t0);
-      for (uint32_t t = warp; t < count; t += kProducerWarps) {
-        const size_t row = row0 + t0 + t;
-        const TQ* q = query + row * p.q_stride + p.q_column + kv_head * p.dim;
-        const TQ* k = key + row * p.k_stride + p.k_column + kv_head * p.dim;
-        float dot = 0.0f;
+      Chunk& chunk = chunks[index & 1u];
+      const uint32_t t0 = index * CHUNK, count = min((uint32_t)CHUNK, p.tokens - t0);
+      constexpr int kSteps = R4 * (int)kLanes / 8;  // 32-wide pieces of a row
+      constexpr uint32_t kBatch = kSteps <= 4 ? 4 : 2;  // tokens whose loads are in flight together
+      constexpr uint32_t kGroup = ScanGroup<CHUNK>::kTokens;
+      const uint32_t padded = (count + kGroup - 1u) / kGroup * kGroup;
+      for (uint32_t begin = warp; begin < padded; begin += kProducerWarps * kBatch) {
+        // loads without branches (absent elements read a present one), so that all of them are in flight at once
+        TQ q_raw[kBatch][kSteps], k_raw[kBatch][kSteps], v_raw[kBatch];
 #pragma unroll
-        for (int i = 0; i < R4; ++i) {
-          const uint32_t c = lane + i * 32u;
-          const float qv = c < p.dim ? as_float(q[c]) * q_scale : 0.0f, kv = c < p.dim ? as_float(k[c]) : 0.0f;
-          chunk.q[t][c] = qv;
-          chunk.k[t][c] = kv;
-          dot = fmaf(qv, kv, dot);
+        for (uint32_t b = 0; b < kBatch; ++b) {
+          const size_t row = row0 + t0 + min(begin + b * kProducerWarps, count - 1u);
+          const TQ* q = query + row * p.q_stride + p.q_column + kv_head * p.dim;
+          const TQ* k = key + row * p.k_stride + p.k_column + kv_head * p.dim;
+#pragma unroll
+          for (int i = 0; i < kSteps; ++i) {
+            const uint32_t c = min(lane + i * 32u, p.dim - 1u);
+            q_raw[b][i] = q[c];
+            k_raw[b][i] = k[c];
+          }
+          v_raw[b] = value[row * p.v_stride + p.v_column + head * p.vdim + min(value_column, p.vdim - 1u)];
         }
-        if (!MEMORY) {
-          dot = warp_sum(dot);
-          if (lane == 0) chunk.extra[t] = dot;
+        float qs[kBatch][kSteps], ks[kBatch][kSteps], vs[kBatch];
+#pragma unroll
+        for (uint32_t b = 0; b < kBatch; ++b) {
+#pragma unroll
+          for (int i = 0; i < kSteps; ++i) {
+            const bool present = lane + i * 32u < p.dim && begin + b * kProducerWarps < count;
+            qs[b][i] = present ? as_float(q_raw[b][i]) * q_scale : 0.0f;
+            ks[b][i] = present ? as_float(k_raw[b][i]) : 0.0f;
+          }
+          vs[b] = value_column < p.vdim ? as_float(v_raw[b]) : 0.0f;
         }
-        if (lane < kSlice) {
-          const uint32_t column = slice * kSlice + lane;
-          chunk.v[t][lane] = column < p.vdim ? as_float(value[row * p.v_stride + p.v_column + head * p.vdim + column]) : 0.0f;
+#pragma unroll
+        for (uint32_t b = 0; b < kBatch; ++b) {
+          const uint32_t t = begin + b * kProducerWarps;
+          if (t >= padded) break;
+          float dot = 0.0f;
+#pragma unroll
+          for (int i = 0; i < kSteps; ++i) {
+            chunk.q[t][lane + i * 32u] = qs[b][i];
+            chunk.k[t][lane + i * 32u] = ks[b][i];
+            dot = fmaf(qs[b][i], ks[b][i], dot);
+          }
+          chunk.v[t][lane] = vs[b];
+          if (!MEMORY) {
+            dot = warp_sum(dot);
+            if (lane == 0) chunk.scalar[t].z = dot;
+          }
         }
       }
       if (warp == 0) {
@@ -313,23 +370,22 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
           if (lane == 0) before = top;
           a = expf(log_forget + before - m);
           b = expf(log_input - m);
-          if (present) chunk.extra[lane] = expf(-m);
+          if (present) chunk.scalar[lane].z = expf(-m);
           top = __shfl_sync(0xffffffffu, m, count - 1u);
         }
-        if (present) {
-          chunk.first[lane] = a;
-          chunk.second[lane] = b;
+        if (lane < padded) {
+          chunk.scalar[lane].x = present ? a : 1.0f;
+          chunk.scalar[lane].y = present ? b : 0.0f;
         }
       }
     };
     auto write_out = [&](uint32_t index) {
-      const ScanChunk<R4>& chunk = chunks[index & 1u];
-      const uint32_t t0 = index * kChunk, count = min(kChunk, p.tokens - t0);
-      for (uint32_t i = thread; i < count * kSlice; i += kProducerWarps * 32u) {
-        const uint32_t t = i / kSlice, column = slice * kSlice + i % kSlice;
-        float o = chunk.out[t][i % kSlice];
-        if (MEMORY) o /= fmaxf(fabsf(chunk.norm_dot[t]), chunk.extra[t]) + 1e-6f;
-        if (column < p.vdim) out[((row0 + t0 + t) * p.heads + head) * p.vdim + column] = o;
+      const Chunk& chunk = chunks[index & 1u];
+      const uint32_t t0 = index * CHUNK, count = min((uint32_t)CHUNK, p.tokens - t0);
+      for (uint32_t t = warp; t < count; t += kProducerWarps) {
+        float o = chunk.out[t][lane];
+        if (MEMORY) o /= fmaxf(fabsf(chunk.norm_dot[t]), chunk.scalar[t].z) + 1e-6f;
+        if (value_column < p.vdim) out[((row0 + t0 + t) * p.heads + head) * p.vdim + value_column] = o;
       }
     };
     produce(0);
@@ -346,102 +402,170 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
     if (MEMORY && thread == 0) state[layout.top(head, slice)] = top;
   } else {
     // ------------------------------ state ------------------------------
-    const uint32_t column = threadIdx.x / kLanes, part = threadIdx.x % kLanes;
-    const bool is_norm = MEMORY && column >= kSlice;  // the extra warp: its first eight lanes carry n
-    const bool active = is_norm ? column == kSlice : slice * kSlice + column < p.vdim;
-    float* home = state + (is_norm ? layout.norm(head, slice)
-                                   : layout.matrix(head) + (size_t)(active ? slice * kSlice + column : 0u) * p.dim);
-    float4 s[R4];
+    const uint32_t column0 = threadIdx.x / kLanes * kColumns, part = threadIdx.x % kLanes;
+    const bool is_norm = MEMORY && column0 >= kSlice;  // the extra warp: the first column of its first lanes carries n
+    float* home[kColumns];
+    bool active[kColumns];
+    Pair s[kColumns][R4 * 2];
 #pragma unroll
-    for (int i = 0; i < R4; ++i) {
-      const uint32_t c = i * 32u + part * 4u;
-      s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (active && !fresh) {
-        if (c < p.dim) s[i].x = home[c];
-        if (c + 1u < p.dim) s[i].y = home[c + 1u];
-        if (c + 2u < p.dim) s[i].z = home[c + 2u];
-        if (c + 3u < p.dim) s[i].w = home[c + 3u];
+    for (int j = 0; j < (int)kColumns; ++j) {
+      const uint32_t column = slice * kSlice + column0 + j;
+      active[j] = is_norm ? column0 + j == kSlice : column < p.vdim;
+      home[j] = state + (is_norm ? layout.norm(head, slice) : layout.matrix(head) + (size_t)(active[j] ? column : 0u) * p.dim);
+#pragma unroll
+      for (int i = 0; i < R4 * 2; ++i) {
+        const uint32_t c = (i >> 1) * (kLanes * 4u) + part * 4u + (i & 1) * 2u;
+        const bool have = active[j] && !fresh;
+        s[j][i] = pair_of(have && c < p.dim ? home[j][c] : 0.0f, have && c + 1u < p.dim ? home[j][c + 1u] : 0.0f);
       }
     }
     __syncthreads();
     for (uint32_t index = 0; index < chunk_count; ++index) {
-      ScanChunk<R4>& chunk = chunks[index & 1u];
-      const uint32_t count = min(kChunk, p.tokens - index * kChunk);
-#pragma unroll 2
-      for (uint32_t t = 0; t < count; ++t) {
-        const float4* q = reinterpret_cast<const float4*>(chunk.q[t]) + part;
-        const float4* k = reinterpret_cast<const float4*>(chunk.k[t]) + part;
-        const float keep = chunk.first[t];
-        if (MEMORY) {
-          const float write = chunk.second[t] * (is_norm ? 1.0f : chunk.v[t][column % kSlice]);
-          float o = 0.0f, o2 = 0.0f;
+      Chunk& chunk = chunks[index & 1u];
+      const uint32_t count = min((uint32_t)CHUNK, p.tokens - index * CHUNK);
+      constexpr int G = ScanGroup<CHUNK>::kTokens;
+#pragma unroll 1
+      for (uint32_t t0 = 0; t0 < count; t0 += G) {
+        float partial[G][kColumns];  // this lane's share of the tokens' read-outs
+        float update[G][kColumns];   // delta rule
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+          const uint32_t t = t0 + g;
+          const ulonglong2* q = reinterpret_cast<const ulonglong2*>(chunk.q[t]) + part;
+          const ulonglong2* k = reinterpret_cast<const ulonglong2*>(chunk.k[t]) + part;
+          const float4 scalar = chunk.scalar[t];
+          const float2 values = *reinterpret_cast<const float2*>(&chunk.v[t][column0 % kSlice]);
+          const Pair keep2 = pair_of(scalar.x, scalar.x);
+          Pair kk[R4 * 2];
 #pragma unroll
           for (int i = 0; i < R4; ++i) {
-            const float4 kk = k[i * 8], qq = q[i * 8];
-            s[i].x = fmaf(kk.x, write, s[i].x * keep);
-            s[i].y = fmaf(kk.y, write, s[i].y * keep);
-            s[i].z = fmaf(kk.z, write, s[i].z * keep);
-            s[i].w = fmaf(kk.w, write, s[i].w * keep);
-            o = fmaf(s[i].x, qq.x, o);
-            o2 = fmaf(s[i].y, qq.y, o2);
-            o = fmaf(s[i].z, qq.z, o);
-            o2 = fmaf(s[i].w, qq.w, o2);
+            const ulonglong2 four = k[i * kLanes];
+            kk[2 * i] = four.x;
+            kk[2 * i + 1] = four.y;
           }
-          o += o2;
-          o += __shfl_xor_sync(0xffffffffu, o, 1);
-          o += __shfl_xor_sync(0xffffffffu, o, 2);
-          o += __shfl_xor_sync(0xffffffffu, o, 4);
-          if (part == 0) {
-            if (!is_norm) chunk.out[t][column] = o;
-            else if (active) chunk.norm_dot[t] = o;
+          Pair sums[kColumns][2];
+#pragma unroll
+          for (int j = 0; j < (int)kColumns; ++j) sums[j][0] = sums[j][1] = 0ull;
+          if (MEMORY) {
+            const float write = scalar.y;
+            const float target[kColumns] = {is_norm ? write : write * values.x, write * values.y};
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+              const ulonglong2 qq = q[i * kLanes];
+#pragma unroll
+              for (int j = 0; j < (int)kColumns; ++j) {
+                const Pair write2 = pair_of(target[j], target[j]);
+                s[j][2 * i] = pair_fma(kk[2 * i], write2, pair_mul(s[j][2 * i], keep2));
+                s[j][2 * i + 1] = pair_fma(kk[2 * i + 1], write2, pair_mul(s[j][2 * i + 1], keep2));
+                sums[j][0] = pair_fma(s[j][2 * i], qq.x, sums[j][0]);
+                sums[j][1] = pair_fma(s[j][2 * i + 1], qq.y, sums[j][1]);
+              }
+            }
+#pragma unroll
+            for (int j = 0; j < (int)kColumns; ++j) partial[g][j] = pair_sum(sums[j][0]) + pair_sum(sums[j][1]);
+          } else {
+            float with_key[kColumns];
+#pragma unroll
+            for (int i = 0; i < R4; ++i)
+#pragma unroll
+              for (int j = 0; j < (int)kColumns; ++j) {
+                sums[j][0] = pair_fma(s[j][2 * i], kk[2 * i], sums[j][0]);
+                sums[j][1] = pair_fma(s[j][2 * i + 1], kk[2 * i + 1], sums[j][1]);
+              }
+#pragma unroll
+            for (int j = 0; j < (int)kColumns; ++j) {
+              with_key[j] = pair_sum(sums[j][0]) + pair_sum(sums[j][1]);
+              sums[j][0] = sums[j][1] = 0ull;
+            }
+#pragma unroll
+            for (int offset = 1; offset < (int)kLanes; offset <<= 1)
+#pragma unroll
+              for (int j = 0; j < (int)kColumns; ++j) with_key[j] += __shfl_xor_sync(0xffffffffu, with_key[j], offset);
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+              const ulonglong2 qq = q[i * kLanes];
+#pragma unroll
+              for (int j = 0; j < (int)kColumns; ++j) {
+                sums[j][0] = pair_fma(s[j][2 * i], qq.x, sums[j][0]);
+                sums[j][1] = pair_fma(s[j][2 * i + 1], qq.y, sums[j][1]);
+              }
+            }
+            update[g][0] = scalar.y * (values.x - scalar.x * with_key[0]);
+            update[g][1] = scalar.y * (values.y - scalar.x * with_key[1]);
+#pragma unroll
+            for (int j = 0; j < (int)kColumns; ++j) {
+              partial[g][j] = pair_sum(sums[j][0]) + pair_sum(sums[j][1]);
+              const Pair update2 = pair_of(update[g][j], update[g][j]);
+#pragma unroll
+              for (int i = 0; i < R4 * 2; ++i) s[j][i] = pair_fma(kk[i], update2, pair_mul(s[j][i], keep2));
+            }
+          }
+        }
+        if (G == 4) {
+          // eight sums over a column's lanes: each exchange halves what a lane keeps, so that lane `part` ends with
+          // value part / (kLanes / 8); the lanes that hold the same value then add what they have
+          float v[8], u[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            v[i] = partial[i / 2 % G][i % 2];
+            u[i] = MEMORY ? 0.0f : update[i / 2 % G][i % 2];
+          }
+#pragma unroll
+          for (int half = 4; half > 0; half >>= 1) {
+            const uint32_t distance = half * (kLanes / 8u);
+            const bool upper = (part & distance) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+              const float sent = upper ? v[i] : v[i + half], kept = upper ? v[i + half] : v[i];
+              v[i] = kept + __shfl_xor_sync(0xffffffffu, sent, distance);
+              if (!MEMORY) u[i] = upper ? u[i + half] : u[i];
+            }
+          }
+#pragma unroll
+          for (uint32_t distance = kLanes / 16u; distance > 0; distance >>= 1)
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], distance);
+          const uint32_t which = part / (kLanes / 8u), t = t0 + which / 2u, j = which % 2u;
+          if (part % (kLanes / 8u) != 0) {
+            // another lane writes this value
+          } else if (MEMORY) {
+            if (!is_norm) chunk.out[t][column0 + j] = v[0];
+            else if (active[0] && j == 0u) chunk.norm_dot[t] = v[0];
+          } else {
+            const float4 scalar = chunk.scalar[t];
+            chunk.out[t][column0 + j] = fmaf(u[0], scalar.z, scalar.x * v[0]);
           }
         } else {
-          float4 kk[R4];
-          float with_key = 0.0f, with_key2 = 0.0f, with_query = 0.0f, with_query2 = 0.0f;
 #pragma unroll
-          for (int i = 0; i < R4; ++i) {
-            kk[i] = k[i * 8];
-            with_key = fmaf(s[i].x, kk[i].x, with_key);
-            with_key2 = fmaf(s[i].y, kk[i].y, with_key2);
-            with_key = fmaf(s[i].z, kk[i].z, with_key);
-            with_key2 = fmaf(s[i].w, kk[i].w, with_key2);
-          }
+          for (int j = 0; j < (int)kColumns; ++j)
 #pragma unroll
-          for (int i = 0; i < R4; ++i) {
-            const float4 qq = q[i * 8];
-            with_query = fmaf(s[i].x, qq.x, with_query);
-            with_query2 = fmaf(s[i].y, qq.y, with_query2);
-            with_query = fmaf(s[i].z, qq.z, with_query);
-            with_query2 = fmaf(s[i].w, qq.w, with_query2);
+            for (int offset = 1; offset < (int)kLanes; offset <<= 1)
+              partial[0][j] += __shfl_xor_sync(0xffffffffu, partial[0][j], offset);
+          if (part == 0) {
+            if (MEMORY) {
+              if (!is_norm) *reinterpret_cast<float2*>(&chunk.out[t0][column0]) = make_float2(partial[0][0], partial[0][1]);
+              else if (active[0]) chunk.norm_dot[t0] = partial[0][0];
+            } else {
+              const float4 scalar = chunk.scalar[t0];
+              *reinterpret_cast<float2*>(&chunk.out[t0][column0]) =
+                  make_float2(fmaf(update[0][0], scalar.z, scalar.x * partial[0][0]),
+                              fmaf(update[0][1], scalar.z, scalar.x * partial[0][1]));
+            }
           }
-          with_key += with_key2;
-          with_query += with_query2;
-#pragma unroll
-          for (int offset = 1; offset < (int)kLanes; offset <<= 1) {
-            with_key += __shfl_xor_sync(0xffffffffu, with_key, offset);
-            with_query += __shfl_xor_sync(0xffffffffu, with_query, offset);
-          }
-          const float update = chunk.second[t] * (chunk.v[t][column] - keep * with_key);
-#pragma unroll
-          for (int i = 0; i < R4; ++i) {
-            s[i].x = fmaf(kk[i].x, update, s[i].x * keep);
-            s[i].y = fmaf(kk[i].y, update, s[i].y * keep);
-            s[i].z = fmaf(kk[i].z, update, s[i].z * keep);
-            s[i].w = fmaf(kk[i].w, update, s[i].w * keep);
-          }
-          if (part == 0) chunk.out[t][column] = fmaf(update, chunk.extra[t], keep * with_query);
         }
       }
       __syncthreads();
     }
 #pragma unroll
-    for (int i = 0; i < R4; ++i) {
-      const uint32_t c = i * 32u + part * 4u;
-      if (!active) continue;
-      if (c < p.dim) home[c] = s[i].x;
-      if (c + 1u < p.dim) home[c + 1u] = s[i].y;
-      if (c + 2u < p.dim) home[c + 2u] = s[i].z;
-      if (c + 3u < p.dim) home[c + 3u] = s[i].w;
+    for (int j = 0; j < (int)kColumns; ++j) {
+      if (!active[j]) continue;
+#pragma unroll
+      for (int i = 0; i < R4 * 2; ++i) {
+        const uint32_t c = (i >> 1) * (kLanes * 4u) + part * 4u + (i & 1) * 2u;
+        float low, high;
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(s[j][i]));
+        if (c < p.dim) home[j][c] = low;
+        if (c + 1u < p.dim) home[j][c + 1u] = high;
+      }
     }
   }
 }
@@ -482,13 +606,17 @@ int launch_scan(const KernelArgs& args) {
                   (const uint32_t*)args.buffers[6], (const uint32_t*)args.buffers[7], (float*)args.buffers[8], p);
     return check_launch(args);
   };
-  const uint32_t quads = (p.dim + 31u) / 32u;
-  if (quads <= 1u) return run(scan_kernel<TQ, MEMORY, 1>, 2 * sizeof(ScanChunk<1>));
-  if (quads <= 2u) return run(scan_kernel<TQ, MEMORY, 2>, 2 * sizeof(ScanChunk<2>));
-  if (quads <= 3u) return run(scan_kernel<TQ, MEMORY, 3>, 2 * sizeof(ScanChunk<3>));
-  if (quads <= 4u) return run(scan_kernel<TQ, MEMORY, 4>, 2 * sizeof(ScanChunk<4>));
-  if (quads <= 6u) return run(scan_kernel<TQ, MEMORY, 6>, 2 * sizeof(ScanChunk<6>));
-  return run(scan_kernel<TQ, MEMORY, 8>, 2 * sizeof(ScanChunk<8>));
+  const uint32_t quads = (p.dim + kLanes * 4u - 1u) / (kLanes * 4u);
+  // few tokens: small chunks, so that more CTAs fit on an SM
+  auto sized = [&](auto r4) {
+    constexpr int R4 = decltype(r4)::value;
+    if (p.tokens <= 4u) return run(scan_kernel<TQ, MEMORY, R4, 4>, 2 * sizeof(ScanChunk<R4, 4>));
+    return run(scan_kernel<TQ, MEMORY, R4, 32>, 2 * sizeof(ScanChunk<R4, 32>));
+  };
+  if (quads <= 1u) return sized(std::integral_constant<int, 1>());
+  if (quads <= 2u) return sized(std::integral_constant<int, 2>());
+  if (quads <= 3u) return sized(std::integral_constant<int, 3>());
+  return sized(std::integral_constant<int, 4>());
 }
 
 }  // namespace

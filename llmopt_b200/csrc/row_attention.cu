@@ -321,7 +321,7 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
 }
 
 // ---- decode --------------------------------------------------------------------------------------
-constexpr uint32_t kWarpKeys = 16, kDecodeWarps = 4, kDecodeStages = 3;
+constexpr uint32_t kWarpKeys = 16, kDecodeWarps = 4, kDecodeStages = 3, kMostSplits = 64;
 
 // Record of one split: 16 maxima, 16 denominators, 16 x DV sums.
 template <int DV>
@@ -482,20 +482,56 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
   if (is_last == 0u) return;
   __threadfence();
   const float* first = records + ((size_t)sequence * p.kv_heads + kv_head) * p.splits * kRecord;
-  for (uint32_t index = threadIdx.x; index < query_rows * DV; index += 128u) {
-    const uint32_t row = index / DV, column = index % DV;
+  const uint32_t used = (keys + per_split - 1u) / per_split;  // the others saw no key
+  // weight of every split for every row, over the row's common denominator
+  float* weights = shared_records;  // [query rows][used]
+  for (uint32_t row = warp; row < query_rows; row += kDecodeWarps) {
     float top = p.sink ? 0.0f : kLowest;
-    for (uint32_t s = 0; s < p.splits; ++s) top = fmaxf(top, __ldcg(first + (size_t)s * kRecord + row));
-    float total = p.sink ? exp2f(-top) : 0.0f, sum = 0.0f;
-    for (uint32_t s = 0; s < p.splits; ++s) {
-      const float* one = first + (size_t)s * kRecord;
-      const float weight = exp2f(__ldcg(one + row) - top);
-      total += weight * __ldcg(one + 16 + row);
-      sum += weight * __ldcg(one + 32 + row * DV + column);
+    for (uint32_t s = lane; s < used; s += 32u) top = fmaxf(top, __ldcg(first + (size_t)s * kRecord + row));
+    top = warp_max(top);
+    float total = 0.0f;
+    for (uint32_t s = lane; s < used; s += 32u) {
+      const float weight = exp2f(__ldcg(first + (size_t)s * kRecord + row) - top);
+      total += weight * __ldcg(first + (size_t)s * kRecord + 16 + row);
+      weights[row * kMostSplits + s] = weight;
     }
-    if (column < p.vdim)
-      out[(((size_t)sequence * p.tokens + row / group) * p.heads + kv_head * group + row % group) * p.vdim + column] =
-          __float2bfloat16_rn(sum / total);
+    total = warp_sum(total) + (p.sink ? exp2f(-top) : 0.0f);
+    __syncwarp();
+    for (uint32_t s = lane; s < used; s += 32u) weights[row * kMostSplits + s] /= total;
+  }
+  __syncthreads();
+  for (uint32_t index = threadIdx.x; index < query_rows * (DV / 4); index += 128u) {
+    const uint32_t row = index / (DV / 4), column = index % (DV / 4) * 4u;
+    const float* source = first + 32 + row * DV + column;
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+    uint32_t s = 0;
+    for (; s + 8u <= used; s += 8u) {
+      float4 part[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) part[i] = __ldcg(reinterpret_cast<const float4*>(source + (size_t)(s + i) * kRecord));
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float weight = weights[row * kMostSplits + s + i];
+        sum.x = fmaf(weight, part[i].x, sum.x);
+        sum.y = fmaf(weight, part[i].y, sum.y);
+        sum.z = fmaf(weight, part[i].z, sum.z);
+        sum.w = fmaf(weight, part[i].w, sum.w);
+      }
+    }
+    for (; s < used; ++s) {
+      const float4 part = __ldcg(reinterpret_cast<const float4*>(source + (size_t)s * kRecord));
+      const float weight = weights[row * kMostSplits + s];
+      sum.x = fmaf(weight, part.x, sum.x);
+      sum.y = fmaf(weight, part.y, sum.y);
+      sum.z = fmaf(weight, part.z, sum.z);
+      sum.w = fmaf(weight, part.w, sum.w);
+    }
+    if (column < p.vdim) {  // vdim is a multiple of eight
+      __nv_bfloat162* target = reinterpret_cast<__nv_bfloat162*>(
+          out + (((size_t)sequence * p.tokens + row / group) * p.heads + kv_head * group + row % group) * p.vdim + column);
+      target[0] = __floats2bfloat162_rn(sum.x, sum.y);
+      target[1] = __floats2bfloat162_rn(sum.z, sum.w);
+    }
   }
 }
 
@@ -540,6 +576,7 @@ int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t merge = kDecodeWarps * record_floats<DV>() * 4u;
   if (bytes < merge) bytes = merge;
   const size_t heads = (size_t)p.sequences * p.kv_heads, counters = (heads * 4 + 255) / 256 * 256;
+  LLMOPT_REQUIRE(p.splits <= kMostSplits, "at most 64 splits");
   LLMOPT_REQUIRE(p.splits == 1u || args.lengths[6] >= counters + heads * p.splits * record_floats<DV>() * 4,
                  "split scratch is too short");
   auto kernel = attention_decode_kernel<DK, DV>;

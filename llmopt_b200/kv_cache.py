@@ -113,7 +113,7 @@ class RowLayout:
 
 
 # value columns one thread block of the state kernels owns
-MATRIX_STATE_SLICE = 16
+MATRIX_STATE_SLICE = 32
 
 
 def matrix_state_elements(heads: int, dim: int, vdim: int, *, normalized: bool) -> int:

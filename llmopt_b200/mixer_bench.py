@@ -1,0 +1,260 @@
+"""Prefill and decode throughput of decoders composed of sequence mixers, and the roofline share of every
+kernel of their steps, beside the W4A16 decoder of the same width, depth, heads and vocabulary and the
+like kernels of that path.  Used by ``bench.py --mixers``; random weights.
+
+  python -m llmopt_b200.mixer_bench [--size 2048|4096|all] [--tokens 2048] [--context 2048]"""
+
+from __future__ import annotations
+
+import argparse
+import json
+import statistics
+import struct
+import time
+from types import SimpleNamespace
+
+import numpy as np
+
+from .cuda_native import Batch, Runtime
+from .model import (AttentionSpec, DeltaSpec, FeedForwardSpec, MatrixMemorySpec, MixerConfig, MixerLayer, ModelConfig,
+                    ParallelSpec, RotarySpec, TokenSideSpec, YarnSpec, random_mixer_weights, random_weights)
+
+
+def sized_config(width: int) -> MixerConfig:
+    """Eight layers of a real model's proportions: matrix memory with 128 x 256 heads, attention and gated
+    delta rule with 128-wide heads, four query heads per key/value head."""
+    heads = width // 128
+    rotary = RotarySpec(dims=128, base=500000.0, scaling=YarnSpec(factor=4.0, original=8192, fast=32.0, slow=1.0))
+    memory = MatrixMemorySpec(heads=heads // 2, dim=128, vdim=256, gate_cap=15.0)
+    parallel = ParallelSpec(
+        left=AttentionSpec(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, rotary=rotary, bias=True,
+                           head_norm=True, sink=True),
+        right=DeltaSpec(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, taps=4))
+    feed_forward = FeedForwardSpec(width=7 * width // 2)
+    layers = tuple(MixerLayer(mixer=parallel if index % 2 else memory, feed_forward=feed_forward) for index in range(8))
+    return MixerConfig(name=f"mixers-{width}", width=width, vocabulary=32768, layers=layers, epsilon=1e-5, norm_offset=1.0,
+                       token_side=TokenSideSpec(dim=256))
+
+
+def like_config(config: MixerConfig) -> ModelConfig:
+    """The W4A16 decoder of the same size."""
+    heads = config.width // 128
+    return ModelConfig(f"w4a16-{config.width}", config.width, ("attention",) * len(config.layers), heads, heads // 4, 128,
+                       config.layers[0].feed_forward.width, config.vocabulary)
+
+
+# ---- algorithmic work of a dispatch ------------------------------------------------------------------------
+
+def work_of(item, past: int, itemsize: int):
+    """(label, bytes, flops) of a recorded dispatch; every operand once."""
+    stem = item.name.removeprefix("llmopt_").removesuffix("_bf16").removesuffix("_f32")
+    u = struct.unpack(f"<{len(item.parameters) // 4}I", item.parameters)
+    e = itemsize
+    if stem == "dense_linear":
+        m, n, k, split = u[:4]
+        return f"dense_linear n{n} k{k}", n * k * e + m * k * e + m * split * e + m * (n - split) * 4, 2 * m * n * k
+    if stem == "embedding_residual":
+        return stem, u[0] * u[2] * (2 * e + 4), 0
+    if stem == "residual_norm":
+        rows, width, _, _, pair = u
+        return stem + (" (two branches)" if pair else ""), rows * width * (4 + 4 + (4 if pair else 0) + 4 + e), 0
+    if stem == "gather_norm":
+        return stem, u[0] * u[2] * (4 + e), 0
+    if stem == "row_attention_prepare":
+        sequences, tokens, heads, kv_heads, dim, vdim = u[:6]
+        return stem, sequences * tokens * 2 * e * (heads * dim + kv_heads * (dim + vdim)), 0
+    if stem == "row_attention":
+        sequences, tokens, heads, kv_heads, dim, vdim = u[:6]
+        keys = past + tokens
+        pairs = tokens * past + tokens * (tokens + 1) // 2
+        return (stem, sequences * (keys * kv_heads * (dim + vdim) * e + tokens * heads * (dim + vdim) * e),
+                2 * sequences * heads * pairs * (dim + vdim))
+    if stem == "head_norm_gate":
+        return stem, u[0] * u[1] * u[2] * (4 + 2 * e), 0
+    if stem in ("delta_prepare", "conv_state"):
+        sequences, tokens, heads, kv_heads, dim, vdim, taps = u[:7]
+        channels = 2 * kv_heads * dim + heads * vdim
+        if stem == "conv_state":
+            return stem, sequences * channels * (taps - 1) * 2 * e, 0
+        return stem, sequences * tokens * (channels * (e + 4) + heads * 16), 0
+    if stem in ("delta_scan", "memory_scan"):
+        sequences, tokens, heads, kv_heads, dim, vdim = u[:6]
+        source = 4 if stem == "delta_scan" else e
+        vectors = (2 * kv_heads * dim + heads * vdim) * source + heads * (vdim * 4 + 8)
+        return stem, sequences * (tokens * vectors + heads * dim * vdim * 8), 0
+    if stem in ("delta_step", "memory_step"):
+        sequences, heads, kv_heads, dim, vdim = u[0], u[2], u[3], u[4], u[5]
+        return stem, sequences * (heads * dim * vdim * 8 + (2 * kv_heads * dim + 3 * heads * vdim) * e), 0
+    if stem == "argmax":
+        return stem, u[0] * u[1] * 4, 0
+    return stem, 0, 0
+
+
+def time_items(runtime, items, past: int, itemsize: int, peaks: dict) -> dict:
+    """Per kernel: all its launches of the step back to back (every layer's own operands)."""
+    groups = {}
+    for item in items:
+        label, nbytes, flops = work_of(item, past, itemsize)
+        groups.setdefault(label, {"items": [], "bytes": nbytes, "flops": flops})["items"].append(item)
+    table = {}
+    for label, group in groups.items():
+        launches = len(group["items"])
+        repeated = group["items"] * max(1, min(16, 64 // launches))
+        ms = runtime.time_dispatches(repeated, warmup=2, iterations=5)
+        floor = max(group["bytes"] / peaks["hbm_gbs"] / 1e6, group["flops"] / peaks["bf16_tflops"] / 1e9)
+        table[label] = {"launches": launches, "us": round(ms * 1e3, 2), "floor_us": round(floor * 1e3, 2),
+                        "frac": round(floor / ms, 3) if ms else None, "share_us": round(ms * 1e3 * launches, 1)}
+    return table
+
+
+# ---- whole steps ---------------------------------------------------------------------------------------------
+
+def decode_rate(engine, batch: int, context: int, steps: int = 32) -> dict:
+    if hasattr(engine, "rewind"):
+        engine.rewind(context)
+    first = [1 + index for index in range(batch)]
+    engine.generate_chained(first, context, 8)
+    times = []
+    for _ in range(5):
+        if hasattr(engine, "rewind"):
+            engine.rewind(context)
+        _, elapsed = engine.generate_chained(first, context, steps)
+        times.append(elapsed / steps)
+    ms = statistics.median(times)
+    return {"batch": batch, "context": context, "ms_per_step": round(ms, 4), "tokens_per_s": round(batch * 1e3 / ms, 1)}
+
+
+def prefill_rate(engine, tokens: int) -> dict:
+    prompt = np.random.default_rng(0).integers(0, engine.config.vocabulary, size=tokens).tolist()
+    engine.prefill(prompt)
+    times = []
+    for _ in range(5):
+        engine.runtime.synchronize()
+        started = time.perf_counter()
+        engine.prefill(prompt)
+        times.append(time.perf_counter() - started)
+    seconds = statistics.median(times)
+    return {"tokens": tokens, "ms": round(seconds * 1e3, 3), "tokens_per_s": round(tokens / seconds, 1)}
+
+
+def measure_mixers(runtime, peaks: dict, config: MixerConfig, tokens: int, context: int, batches=(1, 8, 32)) -> dict:
+    from .mixer_engine import MixerEngine
+
+    weights = random_mixer_weights(config, seed=0, fast=True)
+    result = {"model": config.name, "width": config.width, "layers": len(config.layers), "decode": [], "kernels": {}}
+    for batch in batches:
+        engine = MixerEngine(runtime, config, weights, batch=batch, capacity=context + 64 + (tokens if batch == 1 else 0),
+                             prompt_rows=tokens if batch == 1 else batch)
+        result["decode"].append(decode_rate(engine, batch, context))
+        plan = engine._decode_plan(batch)[0]
+        engine.rewind(context)
+        plan.write([1] * batch, [context] * batch, [engine._row(index) for index in range(batch)])
+        items = [item for item in plan.items if item.name != "llmopt_advance_tokens"]
+        result["kernels"][f"decode, {batch} sequences, {context} tokens behind"] = time_items(
+            runtime, items, context, engine.itemsize, peaks)
+        result["decode"][-1]["kernels_per_step"] = engine._decode_plan(batch)[1].kernel_count()
+        if batch == 1:
+            result["prefill"] = prefill_rate(engine, tokens)
+            plan = engine._prompt_plan(tokens)[0]
+            plan.write([1] * tokens, [0], [engine._row(0)])
+            result["kernels"][f"prompt of {tokens} tokens"] = time_items(runtime, plan.items, 0, engine.itemsize, peaks)
+    return result
+
+
+def measure_like(runtime, peaks: dict, config: MixerConfig, tokens: int, context: int, batches=(1, 8, 32)) -> dict:
+    from .decode_engine import DecodeEngine
+
+    like = like_config(config)
+    weights = random_weights(like, seed=0, fast=True)
+    result = {"model": like.name, "width": like.hidden, "layers": len(like.layers), "decode": []}
+    for batch in batches:
+        engine = DecodeEngine(runtime, like, weights, batch=batch, capacity=context + 64 + tokens)
+        engine.fill_cache_random(context)
+        engine.build(context)
+        result["decode"].append(decode_rate(engine, batch, context))
+        if batch == 1:
+            result["prefill"] = prefill_rate(engine, tokens)
+    return result
+
+
+def like_kernels(runtime, peaks: dict, config: MixerConfig, tokens: int, context: int) -> dict:
+    """The like kernels of the W4A16 path at the same sizes: share of the roofline of each."""
+    from . import dispatch, kernel_bench, parameters
+    from .cuda_native import Buffer, DispatchItem
+
+    width, heads = config.width, config.width // 128
+    table = {}
+
+    def note(label, ms, nbytes, flops=0.0):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e6, flops / peaks["bf16_tflops"] / 1e9)
+        table[label] = {"us": round(ms * 1e3, 2), "floor_us": round(floor * 1e3, 2), "frac": round(floor / ms, 3)}
+
+    def probe(label, op, copies, flops=0.0, **options):
+        args = SimpleNamespace(op=op, m=1, k=width, n=7 * width // 2, heads=heads, kv_heads=heads // 4, dim=128, group=64, layers=2,
+                               past=context)
+        args.__dict__.update(options)
+        keep, items = [], []
+        for _ in range(copies):
+            item, nbytes, context_ = kernel_bench.build_item(runtime, args)
+            keep.append(context_)
+            items.append(item)
+        note(label, runtime.time_dispatches(items, warmup=2, iterations=5), nbytes, flops)
+
+    for m in (1, 8, 32):
+        probe(f"w4a16 linear n{3 * width} k{width}, {m} rows", "linear", 24, m=m, n=3 * width)
+        probe(f"w4a16 linear n{width} k{width}, {m} rows", "linear", 64, m=m, n=width)
+        probe(f"paged attention q8, {m} sequences", "attention", 8, m=m)
+    probe(f"w4a16 linear n{7 * width // 2} k{width}, {tokens} rows", "linear", 8, m=tokens, flops=2.0 * tokens * width * 7 * width // 2)
+    probe(f"w4a16 linear n{width} k{width}, {tokens} rows", "linear", 8, m=tokens, n=width, flops=2.0 * tokens * width * width)
+    probe(f"dense attention, {tokens} tokens", "dense_attention", 2, m=tokens, flops=2.0 * tokens * tokens * 128 * heads)
+    rng = np.random.default_rng(0)
+    half = lambda *shape: dispatch.Tensor(Buffer.of_array(runtime, (rng.standard_normal(shape) * 0.1).astype(np.float16)), shape)
+    commands = Batch(runtime)
+    recurrent = dispatch.Context(runtime, batch=commands)
+    for count in (tokens, 1):
+        q, k, v, beta, out = (half(1, count, heads, 128), half(1, count, heads, 128), half(1, count, heads, 128),
+                              half(1, count, heads), half(1, count, heads, 128))
+        gate = dispatch.Tensor(Buffer.of_array(runtime, -np.ones((1, count, heads), np.float32)), (1, count, heads), "float32")
+        dispatch.dispatch_gated_delta(recurrent, query=q, key=k, value=v, gate=gate, beta=beta, output=out)
+        note(f"gated delta scan (from a zero state), {count} tokens",
+             runtime.time_dispatches([commands.pending.pop()] * 4, warmup=1, iterations=3), count * heads * (128 * 8 + 6))
+        rows = half(count, width)
+        item = DispatchItem("llmopt_rms_norm_f16_simd", [rows.buffer, half(width).buffer, half(count, width).buffer],
+                            parameters.rms_norm(rows=count, width=width, epsilon=1e-5),
+                            (dispatch.simd_rows_grid(count), 1, 1), (256, 1, 1))
+        note(f"rms norm, {count} rows", runtime.time_dispatches([item] * 32, warmup=2, iterations=5), count * width * 4)
+        conv = DispatchItem("llmopt_short_conv_silu_tm_f16", [rows.buffer, half(width, 4).buffer, half(count, width).buffer],
+                            parameters.short_conv_silu_tm(batches=1, tokens=count, channels=width, kernel_width=4, stride=1,
+                                                          padding=3, dilation=1, output_start=0), (1, 1, 1), (256, 1, 1))
+        note(f"short conv + silu, {count} rows", runtime.time_dispatches([conv] * 16, warmup=2, iterations=5), count * width * 4)
+    commands.abort()
+    return table
+
+
+def measure(runtime, peaks: dict, widths=(2048, 4096), tokens: int = 2048, context: int = 2048, like: bool = True) -> list:
+    results = []
+    for width in widths:
+        config = sized_config(width)
+        entry = {"mixers": measure_mixers(runtime, peaks, config, tokens, context)}
+        if like:
+            entry["w4a16"] = measure_like(runtime, peaks, config, tokens, context)
+            entry["w4a16_kernels"] = like_kernels(runtime, peaks, config, tokens, context)
+        results.append(entry)
+    return results
+
+
+def main() -> None:
+    parser = argparse.ArgumentParser()
+    parser.add_argument("--size", default="all", choices=["2048", "4096", "all"])
+    parser.add_argument("--tokens", type=int, default=2048)
+    parser.add_argument("--context", type=int, default=2048)
+    parser.add_argument("--no-like", action="store_true", help="only the mixer models")
+    args = parser.parse_args()
+    peaks = {"hbm_gbs": 6531.6, "bf16_tflops": 1657.8}
+    widths = (2048, 4096) if args.size == "all" else (int(args.size),)
+    for entry in measure(Runtime(), peaks, widths, args.tokens, args.context, not args.no_like):
+        print(json.dumps(entry, indent=1))
+
+
+if __name__ == "__main__":
+    main()

@@ -24,6 +24,17 @@ from .quantize import rotary_pairs
 from .safetensors_archive import as_bfloat16_bits, as_float32
 
 ARGMAX_PARTS = 32
+
+
+def _draw_seed(seed: int, *counters: int) -> int:
+    """A well-mixed 64-bit seed per draw (splitmix64 steps): neighbouring seeds and counters share nothing."""
+    mask, state = (1 << 64) - 1, seed
+    for counter in (0, *counters):
+        state = (state + counter + 0x9E3779B97F4A7C15) & mask
+        state = ((state ^ (state >> 30)) * 0xBF58476D1CE4E5B9) & mask
+        state = ((state ^ (state >> 27)) * 0x94D049BB133111EB) & mask
+        state ^= state >> 31
+    return state or 1
 GROUP = (256, 1, 1)
 
 
@@ -391,7 +402,7 @@ class MixerEngine:
 
         def pick(index: int, logits: np.ndarray) -> int:
             return sample_f32(logits, temperature=temperature, top_k=top_k, top_p=top_p, min_p=min_p,
-                              seed=seed + 1_000_003 * index + len(results[index]))
+                              seed=_draw_seed(seed, index, len(results[index])))
 
         def take(index: int, token: int) -> None:
             results[index].append(token)

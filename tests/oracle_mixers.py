@@ -42,9 +42,14 @@ def gelu_tanh(z):
     return 0.5 * z * (1.0 + np.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
 
 
+# Set by ``rounding_error`` while it measures what rounding alone does: applied to every matrix product.
+_disturb = None
+
+
 def linear(x, weight, bias=None):
     y = f64(x) @ f64(weight).T
-    return y if bias is None else y + f64(bias)
+    y = y if bias is None else y + f64(bias)
+    return y if _disturb is None else _disturb(y)
 
 
 def rms(x, eps):
@@ -218,3 +223,27 @@ def forward(config, w, tokens, per_layer=None):
         if per_layer is not None:
             per_layer.append(x.copy())
     return linear(rms(x, eps) * (1.0 + f64(w["final.norm"])), w["head"])
+
+
+def rounding_error(config, w, tokens, relative, draws=4):
+    """Per position, the largest root-mean-square change of the centred logits over some draws of relative
+    errors of size ``relative`` in every matrix product (and of that size times the row's scale): how much
+    of a difference rounding alone explains.  Positions where a read-out nearly cancels stand out."""
+    global _disturb
+    base, worst = forward(config, w, tokens), None
+    for draw in range(draws):
+        rng = np.random.default_rng(draw)
+
+        def disturb(y):
+            scale = np.sqrt(np.mean(y * y, axis=-1, keepdims=True))
+            return y + relative * (np.abs(y) * rng.uniform(-1, 1, y.shape) + 0.5 * scale * rng.uniform(-1, 1, y.shape))
+
+        _disturb = disturb
+        try:
+            change = forward(config, w, tokens) - base
+        finally:
+            _disturb = None
+        change -= change.mean(axis=-1, keepdims=True)
+        error = np.sqrt((change ** 2).mean(axis=-1))
+        worst = error if worst is None else np.maximum(worst, error)
+    return worst / np.sqrt(((base - base.mean(axis=-1, keepdims=True)) ** 2).mean())
