@@ -104,6 +104,26 @@ inline void launch_kernel(const KernelArgs& launch, void (*kernel)(Params...), d
   cudaLaunchKernelEx(&config, kernel, static_cast<Args&&>(args)...);
 }
 
+// The same with thread-block clusters of `cluster` CTAs along x.
+template <typename... Params, typename... Args>
+inline void launch_cluster_kernel(const KernelArgs& launch, void (*kernel)(Params...), dim3 grid, dim3 block, size_t shared,
+                                  uint32_t cluster, Args&&... args) {
+  cudaLaunchConfig_t config = {};
+  config.gridDim = grid;
+  config.blockDim = block;
+  config.dynamicSmemBytes = shared;
+  config.stream = launch.stream;
+  cudaLaunchAttribute attribute[2];
+  attribute[0].id = cudaLaunchAttributeClusterDimension;
+  attribute[0].val.clusterDim.x = cluster;
+  attribute[0].val.clusterDim.y = attribute[0].val.clusterDim.z = 1;
+  attribute[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attribute[1].val.programmaticStreamSerializationAllowed = 1;
+  config.attrs = attribute;
+  config.numAttrs = context_overlap(launch.ctx) ? 2 : 1;
+  cudaLaunchKernelEx(&config, kernel, static_cast<Args&&>(args)...);
+}
+
 inline int check_launch(const KernelArgs& args) {
   cudaError_t status = cudaGetLastError();
   if (status != cudaSuccess) return fail(args, std::string("launch failed: ") + cudaGetErrorString(status));
@@ -121,6 +141,20 @@ __device__ __forceinline__ void grid_launch_dependents() { asm volatile("griddep
 __device__ __forceinline__ void grid_chain_prologue() {
   grid_launch_dependents();
   grid_dependency_wait();
+}
+// ---- clusters: every CTA of a cluster takes part in each synchronisation --------------------------
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// A float at `local` in the shared memory of CTA `rank` of this cluster.
+__device__ __forceinline__ float cluster_load(const float* local, uint32_t rank) {
+  const uint32_t address = (uint32_t)__cvta_generic_to_shared(local);
+  uint32_t remote;
+  float value;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(address), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(value) : "r"(remote) : "memory");
+  return value;
 }
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -4,7 +4,7 @@
 // A persistent CTA walks over 128 x BN output tiles.  Warp 0 brings the x tile [128 x 64] and the w
 // tile [BN x 64] of every k-block into a shared-memory ring by TMA (128-byte swizzle); one thread of
 // warp 1 issues four tcgen05.mma (K = 16) per k-block into one of two accumulators in tensor memory;
-// warps 2-5 read the finished accumulator (each its quarter of the lanes = output rows), apply bias
+// warps 2-9 read the finished accumulator (each its quarter of the lanes = output rows), apply bias
 // and activation and store, while the next tile accumulates in the other one.  Rows, columns and k
 // beyond the matrices are zero-filled by TMA.
 //
@@ -23,14 +23,17 @@ uint32_t* context_device_error(Context* ctx);
 namespace {
 
 constexpr uint32_t kRows = 128, kDepth = 64;
-constexpr uint32_t kThreads = 192;  // TMA, MMA, four epilogue warps
+constexpr uint32_t kEpilogueWarps = 8;
+constexpr uint32_t kThreads = (2 + kEpilogueWarps) * 32;  // TMA, MMA, epilogue
 constexpr uint32_t kXTileBytes = kRows * kDepth * 2;
 
 template <uint32_t BN>
 struct Shape {
   static constexpr uint32_t kWTileBytes = BN * kDepth * 2;
-  static constexpr uint32_t kStageBytes = kXTileBytes + kWTileBytes;
-  static constexpr uint32_t kStages = BN == 256 ? 4 : (BN == 128 ? 6 : 8);
+  // 64-wide k-blocks per ring stage: a commit costs the issuing thread as much as several narrow MMAs
+  static constexpr uint32_t kBlocks = BN == 256 ? 1 : 2;
+  static constexpr uint32_t kStageBytes = (kXTileBytes + kWTileBytes) * kBlocks;
+  static constexpr uint32_t kStages = BN == 128 ? 3 : 4;
   static constexpr uint32_t kTmemColumns = 2 * BN;
   static constexpr uint32_t kBarriers = kStages * kStageBytes;
   static constexpr uint32_t kHolder = kBarriers + (2 * kStages + 4) * 8;
@@ -58,7 +61,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
   volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kAbort);
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
   const uint32_t m_tiles = (p.m + kRows - 1u) / kRows, n_tiles = (p.n + BN - 1u) / BN, tiles = m_tiles * n_tiles;
-  const uint32_t k_blocks = (p.k + kDepth - 1u) / kDepth;
+  const uint32_t k_stages = (p.k + kDepth * S::kBlocks - 1u) / (kDepth * S::kBlocks);
 
   if (threadIdx.x == 0) {
     for (uint32_t s = 0; s < S::kStages; ++s) {
@@ -67,7 +70,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
     }
     for (uint32_t s = 0; s < 2; ++s) {
       barrier_init(sums_full + s * 8, 1);   // one tcgen05.commit
-      barrier_init(sums_empty + s * 8, 4);  // one arrival per epilogue warp
+      barrier_init(sums_empty + s * 8, kEpilogueWarps);  // one arrival per epilogue warp
     }
     *abort_flag = 0u;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -93,7 +96,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
       bool ok = true;
       for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
         const uint32_t m0 = (tile % m_tiles) * kRows, n0 = (tile / m_tiles) * BN;
-        for (uint32_t kb = 0; kb < k_blocks; ++kb, ++issued) {
+        for (uint32_t ks = 0; ks < k_stages; ++ks, ++issued) {
           const uint32_t s = issued % S::kStages;
           ok = !*abort_flag && barrier_wait(empty + s * 8, ((issued / S::kStages) & 1u) ^ 1u);
           if (!ok) {
@@ -102,8 +105,12 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
           }
           barrier_expect_tx(full + s * 8, S::kStageBytes);
           const uint32_t stage = base + s * S::kStageBytes;
-          tma_load_2d(stage, &map_x, (int32_t)(kb * kDepth), (int32_t)m0, full + s * 8);
-          tma_load_2d(stage + kXTileBytes, &map_w, (int32_t)(kb * kDepth), (int32_t)n0, full + s * 8);
+#pragma unroll
+          for (uint32_t block = 0; block < S::kBlocks; ++block) {
+            const int32_t k0 = (int32_t)((ks * S::kBlocks + block) * kDepth);
+            tma_load_2d(stage + block * kXTileBytes, &map_x, k0, (int32_t)m0, full + s * 8);
+            tma_load_2d(stage + S::kBlocks * kXTileBytes + block * S::kWTileBytes, &map_w, k0, (int32_t)n0, full + s * 8);
+          }
         }
       }
       // on the way out after a failure the copies already started must land first
@@ -119,16 +126,19 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
         const uint32_t half = turn & 1u, sums = tmem_base + half * BN;
         ok = !*abort_flag && barrier_wait(sums_empty + half * 8, ((turn >> 1) & 1u) ^ 1u);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        for (uint32_t kb = 0; kb < k_blocks && ok; ++kb, ++consumed) {
+        for (uint32_t ks = 0; ks < k_stages && ok; ++ks, ++consumed) {
           const uint32_t s = consumed % S::kStages;
           ok = !*abort_flag && barrier_wait(full + s * 8, (consumed / S::kStages) & 1u);
           if (!ok) break;
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-          const uint32_t x_tile = base + s * S::kStageBytes, w_tile = x_tile + kXTileBytes;
+          const uint32_t x_tile = base + s * S::kStageBytes, w_tile = x_tile + S::kBlocks * kXTileBytes;
 #pragma unroll
-          for (uint32_t j = 0; j < kDepth / 16; ++j)
-            mma_f16(sums, operand_descriptor(x_tile + j * 32), operand_descriptor(w_tile + j * 32),
-                    (kb > 0 || j > 0) ? 1u : 0u, bf16_instruction(kRows, BN));
+          for (uint32_t j = 0; j < S::kBlocks * kDepth / 16; ++j) {
+            const uint32_t block = j / (kDepth / 16), at = j % (kDepth / 16) * 32;
+            mma_f16(sums, operand_descriptor(x_tile + block * kXTileBytes + at),
+                    operand_descriptor(w_tile + block * S::kWTileBytes + at), (ks > 0 || j > 0) ? 1u : 0u,
+                    bf16_instruction(kRows, BN));
+          }
           mma_commit(empty + s * 8);
         }
         if (ok) mma_commit(sums_full + half * 8);
@@ -136,7 +146,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
       if (!ok) give_up();
     }
   } else {
-    const uint32_t quarter = warp & 3u;
+    const uint32_t quarter = warp & 3u, side = (warp - 2u) >> 2;  // lanes of tensor memory; every other piece of the columns
     uint32_t turn = 0;
     bool ok = true;
     for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++turn) {
@@ -151,7 +161,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
       const uint32_t row = (tile % m_tiles) * kRows + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
       const uint32_t address = tmem_base + half * BN + ((quarter * 32u) << 16);
 #pragma unroll 1
-      for (uint32_t piece = 0; piece < BN / 32u; ++piece) {
+      for (uint32_t piece = side; piece < BN / 32u; piece += kEpilogueWarps / 4u) {
         uint32_t raw[32];
         tmem_load_32(address + piece * 32u, raw);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");

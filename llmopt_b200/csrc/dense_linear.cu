@@ -33,12 +33,13 @@ __device__ __forceinline__ uint4 load_stream(const bf16* source) {
   return v;
 }
 
-// NT: 8-row batch tiles.  One CTA: 16 weight rows.
+// NT: 8-row batch tiles.  16 weight rows per cluster of `cluster` CTAs, which share out the k-blocks (narrow
+// matrices would leave most SMs without a stream otherwise) and add their sums through distributed shared memory.
 template <int NT>
-__global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const DenseProblem p) {
+__global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const DenseProblem p, uint32_t cluster) {
   grid_launch_dependents();
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, g = lane >> 2, t = lane & 3u;
-  const uint32_t n0 = blockIdx.x * 16u;
+  const uint32_t n0 = blockIdx.x / cluster * 16u, rank = blockIdx.x % cluster, stride = kGemvWarps * cluster;
   const bf16* w = reinterpret_cast<const bf16*>(p.w);
   const bf16* w_low = w + (size_t)min(n0 + g, p.n - 1u) * p.k;
   const bf16* w_high = w + (size_t)min(n0 + g + 8u, p.n - 1u) * p.k;
@@ -56,7 +57,7 @@ __global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const Dense
   };
   // the weights are nobody's output: their first blocks may be requested before the predecessor ends
 #pragma unroll
-  for (int s = 0; s < kGemvStages; ++s) fetch(a[s], warp + s * kGemvWarps);
+  for (int s = 0; s < kGemvStages; ++s) fetch(a[s], rank * kGemvWarps + warp + s * stride);
   grid_dependency_wait();
 
   const bf16* x = reinterpret_cast<const bf16*>(p.x);
@@ -65,10 +66,10 @@ __global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const Dense
   for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
     for (int i = 0; i < 4; ++i) sum[nt][i] = 0.0f;
-  for (uint32_t first = warp; first < blocks; first += kGemvStages * kGemvWarps) {
+  for (uint32_t first = rank * kGemvWarps + warp; first < blocks; first += kGemvStages * stride) {
 #pragma unroll
     for (int s = 0; s < kGemvStages; ++s) {
-      const uint32_t block = first + s * kGemvWarps;
+      const uint32_t block = first + s * stride;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const uint32_t k = block * 64u + half * 32u + t * 8u;
@@ -81,7 +82,7 @@ __global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const Dense
           mma_bf16(sum[nt], low.z, high.z, low.w, high.w, b.z, b.w);
         }
       }
-      fetch(a[s], block + kGemvStages * kGemvWarps);
+      fetch(a[s], block + kGemvStages * stride);
     }
   }
 
@@ -97,8 +98,20 @@ __global__ void __launch_bounds__(kGemvWarps * 32) dense_gemv_kernel(const Dense
     float value = 0.0f;
 #pragma unroll
     for (int part = 0; part < kGemvWarps; ++part) value += partial[part][row][column];
+    if (cluster == 1u) dense_store<bf16>(p, row, n0 + column, value);
+    else partial[0][row][column] = value;  // read and written by this thread only
+  }
+  if (cluster == 1u) return;
+  cluster_sync();
+  // the cluster's CTAs share out the outputs; sums in rank order
+  for (uint32_t index = rank * kGemvWarps * 32 + threadIdx.x; index < NT * 8u * 16u; index += stride * 32u) {
+    const uint32_t column = index & 15u, row = index >> 4;
+    if (row >= p.m || n0 + column >= p.n) continue;
+    float value = 0.0f;
+    for (uint32_t other = 0; other < cluster; ++other) value += cluster_load(&partial[0][row][column], other);
     dense_store<bf16>(p, row, n0 + column, value);
   }
+  cluster_sync();  // nobody leaves while its sums may be read
 }
 
 // One warp per output column, up to eight rows.
@@ -178,12 +191,20 @@ int run_cuda_cores(const KernelArgs& args, const DenseProblem& p) {
 }
 
 int run_gemv(const KernelArgs& args, const DenseProblem& p) {
-  const dim3 grid((p.n + 15u) / 16u), block(kGemvWarps * 32);
-  if (p.m <= 8u) launch_kernel(args, dense_gemv_kernel<1>, grid, block, 0, p);
-  else if (p.m <= 16u) launch_kernel(args, dense_gemv_kernel<2>, grid, block, 0, p);
-  else if (p.m <= 32u) launch_kernel(args, dense_gemv_kernel<4>, grid, block, 0, p);
-  else launch_kernel(args, dense_gemv_kernel<8>, grid, block, 0, p);
-  return check_launch(args);
+  const uint32_t tiles = (p.n + 15u) / 16u, blocks = (p.k + 63u) / 64u;
+  // at least one CTA per SM; a warp of a split keeps at least one k-block
+  const uint32_t wanted = (uint32_t)context_sm_count(args.ctx);
+  uint32_t cluster = 1;
+  while (cluster < 8u && tiles * cluster < wanted && blocks >= 2u * cluster * kGemvWarps) cluster *= 2u;
+  auto run = [&](auto kernel) {
+    if (cluster == 1u) launch_kernel(args, kernel, dim3(tiles), dim3(kGemvWarps * 32), 0, p, cluster);
+    else launch_cluster_kernel(args, kernel, dim3(tiles * cluster), dim3(kGemvWarps * 32), 0, cluster, p, cluster);
+    return check_launch(args);
+  };
+  if (p.m <= 8u) return run(dense_gemv_kernel<1>);
+  if (p.m <= 16u) return run(dense_gemv_kernel<2>);
+  if (p.m <= 32u) return run(dense_gemv_kernel<4>);
+  return run(dense_gemv_kernel<8>);
 }
 
 // Buffers [x, w, bias, out, out32, ids, table] (an absent one repeats another); params

@@ -1,6 +1,8 @@
 // Recurrent mixers with a matrix state per head, carried in fp32 from token to token:
 //   llmopt_delta_prepare_{bf16,f32}    short convolutions, unit q and k, decay and step size of a gated delta rule
 //   llmopt_conv_state_{bf16,f32}       the convolutions' last inputs
+//   llmopt_delta_step_{bf16,f32}, llmopt_memory_step_{bf16,f32}   one token per sequence, everything between the input
+//                                      projections and the output projection in one launch
 //   llmopt_delta_scan_f32              S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   llmopt_memory_scan_{bf16,f32}      stabilised exponential gating (mLSTM): S <- a S + b k v^T, n <- a n + b k,
 //                                      o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)
@@ -38,17 +40,34 @@ struct DeltaPrepareParams {
   uint32_t state_rows;
 };
 
-// Input of channel `channel` (counted over q, k, v) at `token` - `back`, from the projections or, before
-// the step's first token, from the sequence's stored inputs [channels][taps - 1], oldest first.
+// Input of channel `channel` (counted over q, k, v; column `column` of the projections) at `token` of the step,
+// which may lie before it.  Earlier inputs are kept in a ring [taps][channels]: position p in row p % taps, so that
+// a step of one token overwrites what no kernel of that step reads.
 template <typename T>
 struct ConvInputs {
   const T* projected;  // first row of the sequence
-  const T* stored;     // or null: nothing before the step
-  uint32_t stride, taps;
+  const T* ring;
+  uint32_t stride, taps, channels, past;
   __device__ __forceinline__ float at(uint32_t column, uint32_t channel, int token) const {
     if (token >= 0) return as_float(projected[(size_t)token * stride + column]);
-    const int kept = (int)taps - 1 + token;
-    return stored != nullptr ? as_float(stored[(size_t)channel * (taps - 1u) + kept]) : 0.0f;
+    const int position = (int)past + token;
+    return position >= 0 ? as_float(ring[(size_t)((uint32_t)position % taps) * channels + channel]) : 0.0f;
+  }
+  // The convolution's value before its activation.
+  __device__ __forceinline__ float convolve(const float* __restrict__ weight, uint32_t column, uint32_t channel, int token) const {
+    const float* w = weight + (size_t)channel * taps;
+    float sum = 0.0f;
+    if (taps == 4u) {  // the usual length: all loads in flight at once
+      float x[4];
+#pragma unroll
+      for (int tap = 0; tap < 4; ++tap) x[tap] = at(column, channel, token - 3 + tap);
+#pragma unroll
+      for (int tap = 0; tap < 4; ++tap) sum = fmaf(__ldg(w + tap), x[tap], sum);
+      return sum;
+    }
+    for (uint32_t tap = 0; tap < taps; ++tap)
+      sum = fmaf(__ldg(w + tap), at(column, channel, token - (int)(taps - 1u - tap)), sum);
+    return sum;
   }
 };
 
@@ -91,15 +110,9 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* projected, 
   }
   const uint32_t state_row = min(sequence_rows[sequence], p.state_rows - 1u);
   const ConvInputs<T> inputs = {projected + (size_t)sequence * p.tokens * p.stride,
-                                past[sequence] > 0 ? conv_state + (size_t)state_row * channels * (p.taps - 1u) : nullptr,
-                                p.stride, p.taps};
-  auto convolved = [&](uint32_t c) {
-    float sum = 0.0f;
-    for (uint32_t tap = 0; tap < p.taps; ++tap)
-      sum = fmaf(__ldg(conv_weight + (size_t)(channel0 + c) * p.taps + tap),
-                 inputs.at(column0 + c, channel0 + c, (int)token - (int)(p.taps - 1u - tap)), sum);
-    return silu_f32(sum);
-  };
+                                conv_state + (size_t)state_row * channels * p.taps, p.stride, p.taps, channels,
+                                past[sequence]};
+  auto convolved = [&](uint32_t c) { return silu_f32(inputs.convolve(conv_weight, column0 + c, channel0 + c, (int)token)); };
   if (is_value) {
     for (uint32_t c = lane; c < size; c += 32u) target[c] = convolved(c);
     return;
@@ -122,6 +135,87 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* projected, 
   }
 }
 
+// Prompts, four taps, heads of at most 128: a warp walks over kStretch tokens of one head with the taps and the last
+// inputs in registers, so that every input is read once.
+constexpr uint32_t kStretch = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(128) delta_prepare_stream_kernel(const T* projected, const float* scalars,
+                                                                   const float* __restrict__ conv_weight,
+                                                                   const T* conv_state, const uint32_t* past,
+                                                                   const uint32_t* sequence_rows,
+                                                                   const float* __restrict__ a_log,
+                                                                   const float* __restrict__ dt_bias, float* q_out,
+                                                                   float* k_out, float* v_out, float* decay, float* beta,
+                                                                   DeltaPrepareParams p) {
+  grid_chain_prologue();
+  const uint32_t lane = threadIdx.x & 31u, item = blockIdx.x * 4u + (threadIdx.x >> 5);
+  const uint32_t parts = 2u * p.kv_heads + p.heads + 1u, stretches = (p.tokens + kStretch - 1u) / kStretch;
+  if (item >= p.sequences * stretches * parts) return;
+  const uint32_t part = item % parts, sequence = item / parts / stretches, t0 = item / parts % stretches * kStretch;
+  const uint32_t count = min(kStretch, p.tokens - t0);
+  const size_t row0 = (size_t)sequence * p.tokens + t0;
+  if (part == parts - 1u) {
+    for (uint32_t index = lane; index < count * p.heads; index += 32u) {
+      const uint32_t h = index % p.heads;
+      const size_t row = row0 + index / p.heads;
+      const float* source = scalars + row * p.scalar_stride;
+      beta[row * p.heads + h] = sigmoid_f32(source[p.beta_column + h]);
+      decay[row * p.heads + h] = expf(-expf(a_log[h]) * softplus_f32(source[p.decay_column + h] + dt_bias[h]));
+    }
+    return;
+  }
+  const uint32_t qk = p.kv_heads * p.dim, channels = 2u * qk + p.heads * p.vdim;
+  const bool is_value = part >= 2u * p.kv_heads, is_query = part < p.kv_heads;
+  const uint32_t head = is_query ? part : is_value ? part - 2u * p.kv_heads : part - p.kv_heads;
+  const uint32_t size = is_value ? p.vdim : p.dim, width = is_value ? p.heads * p.vdim : qk;
+  const uint32_t column0 = (is_query ? p.q_column : is_value ? p.v_column : p.k_column) + head * size;
+  const uint32_t channel0 = (is_query ? 0u : is_value ? 2u * qk : qk) + head * size;
+  float* target = (is_query ? q_out : is_value ? v_out : k_out) + row0 * width + head * size;
+  const uint32_t state_row = min(sequence_rows[sequence], p.state_rows - 1u);
+  const ConvInputs<T> inputs = {projected + (size_t)sequence * p.tokens * p.stride,
+                                conv_state + (size_t)state_row * channels * 4u, p.stride, 4u, channels, past[sequence]};
+  constexpr int kMost = 4;  // channels per lane
+  float4 w[kMost];
+  float last[kMost][3];
+#pragma unroll
+  for (int i = 0; i < kMost; ++i) {
+    const uint32_t c = min(lane + i * 32u, size - 1u);
+    w[i] = *reinterpret_cast<const float4*>(conv_weight + (size_t)(channel0 + c) * 4u);
+#pragma unroll
+    for (int back = 0; back < 3; ++back) last[i][back] = inputs.at(column0 + c, channel0 + c, (int)t0 - 3 + back);
+  }
+  const float extra = is_query ? 1.0f / sqrtf((float)p.dim) : 1.0f;
+  const T* source = inputs.projected + (size_t)t0 * p.stride + column0;
+  constexpr uint32_t kAhead = 4;  // tokens whose inputs are in flight together
+  for (uint32_t t = 0; t < count; t += kAhead) {
+    T raw[kAhead][kMost];
+#pragma unroll
+    for (uint32_t ahead = 0; ahead < kAhead; ++ahead)
+#pragma unroll
+      for (int i = 0; i < kMost; ++i)
+        raw[ahead][i] = source[(size_t)min(t + ahead, count - 1u) * p.stride + min(lane + i * 32u, size - 1u)];
+#pragma unroll
+    for (uint32_t ahead = 0; ahead < kAhead; ++ahead) {
+      if (t + ahead >= count) break;
+      float value[kMost], squares = 0.0f;
+#pragma unroll
+      for (int i = 0; i < kMost; ++i) {
+        const float now = as_float(raw[ahead][i]);
+        value[i] = silu_f32(fmaf(w[i].w, now, fmaf(w[i].z, last[i][2], fmaf(w[i].y, last[i][1], w[i].x * last[i][0]))));
+        last[i][0] = last[i][1];
+        last[i][1] = last[i][2];
+        last[i][2] = now;
+        if (lane + i * 32u < size) squares += value[i] * value[i];
+      }
+      const float scale = is_value ? 1.0f : extra / sqrtf(warp_sum(squares) + 1e-6f);
+#pragma unroll
+      for (int i = 0; i < kMost; ++i)
+        if (lane + i * 32u < size) target[(size_t)(t + ahead) * width + lane + i * 32u] = value[i] * scale;
+    }
+  }
+}
+
 bool delta_prepare_params(const KernelArgs& args, DeltaPrepareParams* p) {
   memcpy(p, args.params, sizeof(*p));
   return p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->dim <= 256u && p->vdim > 0 &&
@@ -141,45 +235,44 @@ int launch_delta_prepare(const KernelArgs& args) {
                  "scalar columns lie outside the row");
   LLMOPT_REQUIRE(args.lengths[0] >= rows * p.stride * sizeof(T) && args.lengths[1] >= rows * p.scalar_stride * 4 &&
                      args.lengths[2] >= channels * p.taps * 4 &&
-                     args.lengths[3] >= p.state_rows * channels * (p.taps - 1) * sizeof(T) &&
+                     args.lengths[3] >= p.state_rows * channels * p.taps * sizeof(T) &&
                      args.lengths[4] >= (size_t)p.sequences * 4 && args.lengths[5] >= (size_t)p.sequences * 4 &&
                      args.lengths[6] >= (size_t)p.heads * 4 && args.lengths[7] >= (size_t)p.heads * 4 &&
                      args.lengths[8] >= rows * qk * 4 && args.lengths[9] >= rows * qk * 4 && args.lengths[10] >= rows * vs * 4 &&
                      args.lengths[11] >= rows * p.heads * 4 && args.lengths[12] >= rows * p.heads * 4,
                  "buffer is too short");
   if (rows == 0) return 0;
-  const size_t items = rows * (2 * p.kv_heads + p.heads + 1);
-  launch_kernel(args, delta_prepare_kernel<T>, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0, (const T*)args.buffers[0],
-                (const float*)args.buffers[1], (const float*)args.buffers[2], (const T*)args.buffers[3],
-                (const uint32_t*)args.buffers[4], (const uint32_t*)args.buffers[5], (const float*)args.buffers[6],
-                (const float*)args.buffers[7], (float*)args.buffers[8], (float*)args.buffers[9], (float*)args.buffers[10],
-                (float*)args.buffers[11], (float*)args.buffers[12], p);
-  return check_launch(args);
+  const size_t parts = 2 * p.kv_heads + p.heads + 1;
+  auto run = [&](auto kernel, size_t items) {
+    launch_kernel(args, kernel, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0, (const T*)args.buffers[0],
+                  (const float*)args.buffers[1], (const float*)args.buffers[2], (const T*)args.buffers[3],
+                  (const uint32_t*)args.buffers[4], (const uint32_t*)args.buffers[5], (const float*)args.buffers[6],
+                  (const float*)args.buffers[7], (float*)args.buffers[8], (float*)args.buffers[9], (float*)args.buffers[10],
+                  (float*)args.buffers[11], (float*)args.buffers[12], p);
+    return check_launch(args);
+  };
+  if (p.taps == 4u && p.dim <= 128u && p.vdim <= 128u && p.tokens >= 8u && ((uintptr_t)args.buffers[2] & 15u) == 0)
+    return run(delta_prepare_stream_kernel<T>, (size_t)p.sequences * ((p.tokens + kStretch - 1u) / kStretch) * parts);
+  return run(delta_prepare_kernel<T>, rows * parts);
 }
 
 // ---- the convolutions' stored inputs ---------------------------------------------------------------
-constexpr uint32_t kMostTaps = 16;
-
 template <typename T>
 __global__ void __launch_bounds__(128) conv_state_kernel(const T* projected, T* conv_state, const uint32_t* past,
                                                          const uint32_t* sequence_rows, DeltaPrepareParams p) {
   grid_chain_prologue();
-  const uint32_t qk = p.kv_heads * p.dim, channels = 2u * qk + p.heads * p.vdim, kept = p.taps - 1u;
+  const uint32_t qk = p.kv_heads * p.dim, channels = 2u * qk + p.heads * p.vdim;
   const uint32_t channel = blockIdx.x * 128u + threadIdx.x, sequence = blockIdx.y;
   if (channel >= channels) return;
   const uint32_t column = channel < qk ? p.q_column + channel
                           : channel < 2u * qk ? p.k_column + channel - qk
                                               : p.v_column + channel - 2u * qk;
-  T* stored = conv_state + (size_t)min(sequence_rows[sequence], p.state_rows - 1u) * channels * kept;
-  const ConvInputs<T> inputs = {projected + (size_t)sequence * p.tokens * p.stride, past[sequence] > 0 ? stored : nullptr,
-                                p.stride, p.taps};
-  float next[kMostTaps];
-#pragma unroll
-  for (uint32_t i = 0; i < kMostTaps; ++i)
-    if (i < kept) next[i] = inputs.at(column, channel, (int)p.tokens - (int)kept + (int)i);
-#pragma unroll
-  for (uint32_t i = 0; i < kMostTaps; ++i)
-    if (i < kept) stored[(size_t)channel * kept + i] = from_float<T>(next[i]);
+  T* ring = conv_state + (size_t)min(sequence_rows[sequence], p.state_rows - 1u) * channels * p.taps;
+  const T* rows = projected + (size_t)sequence * p.tokens * p.stride;
+  for (uint32_t back = 1; back <= min(p.taps, p.tokens); ++back) {
+    const uint32_t token = p.tokens - back;
+    ring[(size_t)((past[sequence] + token) % p.taps) * channels + channel] = rows[(size_t)token * p.stride + column];
+  }
 }
 
 // Buffers [projected, conv state, past, sequence rows]; the parameter block of llmopt_delta_prepare.
@@ -188,13 +281,12 @@ int launch_conv_state(const KernelArgs& args) {
   DeltaPrepareParams p;
   LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == sizeof(p), "expects 4 buffers and 60 parameter bytes");
   LLMOPT_REQUIRE(delta_prepare_params(args, &p), "head sizes or projection columns are inconsistent");
-  LLMOPT_REQUIRE(p.taps <= kMostTaps + 1u, "at most 17 taps");
   const size_t channels = 2 * (size_t)p.kv_heads * p.dim + (size_t)p.heads * p.vdim;
   LLMOPT_REQUIRE(args.lengths[0] >= (size_t)p.sequences * p.tokens * p.stride * sizeof(T) &&
-                     args.lengths[1] >= p.state_rows * channels * (p.taps - 1) * sizeof(T) &&
+                     args.lengths[1] >= p.state_rows * channels * p.taps * sizeof(T) &&
                      args.lengths[2] >= (size_t)p.sequences * 4 && args.lengths[3] >= (size_t)p.sequences * 4,
                  "buffer is too short");
-  if (p.sequences == 0 || p.tokens == 0 || p.taps == 1u) return 0;
+  if (p.sequences == 0 || p.tokens == 0) return 0;
   launch_kernel(args, conv_state_kernel<T>, dim3((uint32_t)((channels + 127) / 128), p.sequences), dim3(128), 0,
                 (const T*)args.buffers[0], (T*)args.buffers[1], (const uint32_t*)args.buffers[2],
                 (const uint32_t*)args.buffers[3], p);
@@ -266,6 +358,61 @@ __device__ __forceinline__ float pair_sum(Pair a) {
   asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(a));
   return low + high;
 }
+
+// A lane's share of kColumns columns of a state: four rows every kLanes * 4.  Rows beyond dim hold some finite
+// value, which meets only zeros of q and k and is not stored.
+template <int R4>
+struct StateColumns {
+  float* home[kColumns];
+  bool active[kColumns];
+  Pair s[kColumns][R4 * 2];
+  __device__ __forceinline__ void load(uint32_t part, uint32_t dim, bool vectors, bool fresh) {
+    if (fresh) {
+#pragma unroll
+      for (int j = 0; j < (int)kColumns; ++j)
+#pragma unroll
+        for (int i = 0; i < R4 * 2; ++i) s[j][i] = 0ull;
+    } else if (vectors) {
+#pragma unroll
+      for (int j = 0; j < (int)kColumns; ++j)
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+          const ulonglong2 four = *reinterpret_cast<const ulonglong2*>(home[j] + min(i * kLanes * 4u + part * 4u, dim - 4u));
+          s[j][2 * i] = four.x;
+          s[j][2 * i + 1] = four.y;
+        }
+    } else {
+#pragma unroll
+      for (int j = 0; j < (int)kColumns; ++j)
+#pragma unroll
+        for (int i = 0; i < R4 * 2; ++i) {
+          const uint32_t c = (i >> 1) * (kLanes * 4u) + part * 4u + (i & 1) * 2u;
+          s[j][i] = pair_of(home[j][min(c, dim - 1u)], home[j][min(c + 1u, dim - 1u)]);
+        }
+    }
+  }
+  __device__ __forceinline__ void store(uint32_t part, uint32_t dim, bool vectors) const {
+#pragma unroll
+    for (int j = 0; j < (int)kColumns; ++j) {
+      if (!active[j]) continue;
+#pragma unroll
+      for (int i = 0; i < R4; ++i) {
+        const uint32_t c = i * kLanes * 4u + part * 4u;
+        if (vectors) {
+          if (c < dim) *reinterpret_cast<ulonglong2*>(home[j] + c) = make_ulonglong2(s[j][2 * i], s[j][2 * i + 1]);
+        } else {
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            float low, high;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(s[j][2 * i + h]));
+            if (c + 2u * h < dim) home[j][c + 2u * h] = low;
+            if (c + 2u * h + 1u < dim) home[j][c + 2u * h + 1u] = high;
+          }
+        }
+      }
+    }
+  }
+};
 
 // TQ: element of q, k, v (fp32 for the delta rule, whose unit vectors are fp32).
 template <typename TQ, bool MEMORY, int R4, int CHUNK>
@@ -404,21 +551,17 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
     // ------------------------------ state ------------------------------
     const uint32_t column0 = threadIdx.x / kLanes * kColumns, part = threadIdx.x % kLanes;
     const bool is_norm = MEMORY && column0 >= kSlice;  // the extra warp: the first column of its first lanes carries n
-    float* home[kColumns];
-    bool active[kColumns];
-    Pair s[kColumns][R4 * 2];
+    StateColumns<R4> columns;
+    auto& active = columns.active;
+    auto& s = columns.s;
 #pragma unroll
     for (int j = 0; j < (int)kColumns; ++j) {
       const uint32_t column = slice * kSlice + column0 + j;
       active[j] = is_norm ? column0 + j == kSlice : column < p.vdim;
-      home[j] = state + (is_norm ? layout.norm(head, slice) : layout.matrix(head) + (size_t)(active[j] ? column : 0u) * p.dim);
-#pragma unroll
-      for (int i = 0; i < R4 * 2; ++i) {
-        const uint32_t c = (i >> 1) * (kLanes * 4u) + part * 4u + (i & 1) * 2u;
-        const bool have = active[j] && !fresh;
-        s[j][i] = pair_of(have && c < p.dim ? home[j][c] : 0.0f, have && c + 1u < p.dim ? home[j][c + 1u] : 0.0f);
-      }
+      columns.home[j] = state + (is_norm ? layout.norm(head, slice) : layout.matrix(head) + (size_t)(active[j] ? column : 0u) * p.dim);
     }
+    const bool vectors = p.dim % 4u == 0 && p.state_stride % 4u == 0;
+    columns.load(part, p.dim, vectors, fresh);
     __syncthreads();
     for (uint32_t index = 0; index < chunk_count; ++index) {
       Chunk& chunk = chunks[index & 1u];
@@ -555,18 +698,7 @@ __global__ void __launch_bounds__(ScanThreads<MEMORY>::kAll) scan_kernel(const T
       }
       __syncthreads();
     }
-#pragma unroll
-    for (int j = 0; j < (int)kColumns; ++j) {
-      if (!active[j]) continue;
-#pragma unroll
-      for (int i = 0; i < R4 * 2; ++i) {
-        const uint32_t c = (i >> 1) * (kLanes * 4u) + part * 4u + (i & 1) * 2u;
-        float low, high;
-        asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(s[j][i]));
-        if (c < p.dim) home[j][c] = low;
-        if (c + 1u < p.dim) home[j][c + 1u] = high;
-      }
-    }
+    columns.store(part, p.dim, vectors);
   }
 }
 
@@ -619,6 +751,241 @@ int launch_scan(const KernelArgs& args) {
   return sized(std::integral_constant<int, 4>());
 }
 
+// ---- one token per sequence, fused -----------------------------------------------------------------
+struct StepParams {
+  uint32_t sequences, tokens /* 1 */, heads, kv_heads, dim, vdim, taps;
+  uint32_t stride, q_column, k_column, v_column, gate_column;  // projections, T [sequences, stride]
+  uint32_t scalar_stride, first_column, second_column;         // delta: beta, decay; memory: input gate, forget gate
+  uint32_t state_rows, state_stride;
+  float gate_cap, epsilon;
+};
+struct StepBuffers {
+  const void* projected;
+  const float* scalars;
+  const float* conv_weight;
+  void* conv_state;
+  const float* a_log;
+  const float* dt_bias;
+  const float* norm;  // delta: [vdim]; memory: [heads * vdim]
+  float* state;
+  const uint32_t* past;
+  const uint32_t* sequence_rows;
+  void* out;  // T [sequences, heads * vdim]
+};
+
+template <bool MEMORY> __host__ __device__ constexpr uint32_t step_threads() {
+  return (kColumnWarps + (MEMORY ? 1u : 0u)) * 32u;
+}
+
+// A CTA owns kSlice value columns of one head of one sequence, the CTAs of a head are one cluster: the
+// head's norm needs every column's square.  Lanes and columns as in the scan.
+template <typename T, bool MEMORY, int R4>
+__global__ void __launch_bounds__(step_threads<MEMORY>()) state_step_kernel(const StepBuffers b, const StepParams p) {
+  grid_chain_prologue();
+  constexpr uint32_t kRow = R4 * kLanes * 4u, kThreads = step_threads<MEMORY>();
+  __shared__ __align__(16) float q_row[kRow], k_row[kRow];
+  __shared__ float v_row[kSlice], o_row[kSlice];
+  __shared__ float norm_dot, cta_square;
+  const uint32_t slices = slices_of(p.vdim);
+  const uint32_t slice = blockIdx.x, head = blockIdx.y, sequence = blockIdx.z;
+  const uint32_t kv_head = head / (p.heads / p.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
+  const uint32_t past = b.past[sequence], state_row = min(b.sequence_rows[sequence], p.state_rows - 1u);
+  float* state = b.state + (size_t)state_row * p.state_stride;
+  const StateRow layout = {p.heads, p.dim, p.vdim};
+  const T* projected = reinterpret_cast<const T*>(b.projected) + (size_t)sequence * p.stride;
+  const float* scalars = b.scalars + (size_t)sequence * p.scalar_stride;
+
+  // the state is requested first; everything else is computed while it is on its way
+  const uint32_t column0 = threadIdx.x / kLanes * kColumns, part = threadIdx.x % kLanes;
+  const bool is_norm = MEMORY && column0 >= kSlice;
+  StateColumns<R4> columns;
+  auto& active = columns.active;
+  auto& s = columns.s;
+#pragma unroll
+  for (int j = 0; j < (int)kColumns; ++j) {
+    const uint32_t column = slice * kSlice + column0 + j;
+    active[j] = is_norm ? column0 + j == kSlice : column < p.vdim;
+    columns.home[j] = state + (is_norm ? layout.norm(head, slice) : layout.matrix(head) + (size_t)(active[j] ? column : 0u) * p.dim);
+  }
+  const bool vectors = p.dim % 4u == 0 && p.state_stride % 4u == 0;
+  columns.load(part, p.dim, vectors, past == 0);
+  float old_top = 0.0f;
+  if (MEMORY && past > 0) old_top = state[layout.top(head, slice)];
+  float keep, write, floor_value = 0.0f, new_top = 0.0f;
+  if (MEMORY) {
+    const float log_input = p.gate_cap * tanhf(scalars[p.first_column + head] / p.gate_cap);
+    const float log_forget = -softplus_f32(-p.gate_cap * tanhf(scalars[p.second_column + head] / p.gate_cap));
+    new_top = fmaxf(log_forget + old_top, log_input);
+    keep = expf(log_forget + old_top - new_top);
+    write = expf(log_input - new_top);
+    floor_value = expf(-new_top);
+  } else {
+    write = sigmoid_f32(scalars[p.first_column + head]);
+    keep = expf(-expf(b.a_log[head]) * softplus_f32(scalars[p.second_column + head] + b.dt_bias[head]));
+  }
+
+  // q, k and this slice's v
+  const uint32_t qk = p.kv_heads * p.dim, channels = 2u * qk + p.heads * p.vdim;
+  T* ring = MEMORY ? nullptr : reinterpret_cast<T*>(b.conv_state) + (size_t)state_row * channels * p.taps;
+  for (uint32_t index = threadIdx.x; index < 2u * kRow + kSlice; index += kThreads) {
+    const bool is_value = index >= 2u * kRow, is_key = !is_value && index >= kRow;
+    const uint32_t c = is_value ? slice * kSlice + index - 2u * kRow : index % kRow;
+    float value = 0.0f;
+    if (c < (is_value ? p.vdim : p.dim)) {
+      const uint32_t column = is_value ? p.v_column + head * p.vdim + c : (is_key ? p.k_column : p.q_column) + kv_head * p.dim + c;
+      if (MEMORY) {
+        value = as_float(projected[column]);
+        if (!is_value && !is_key) value *= 1.0f / sqrtf((float)p.dim);
+      } else {
+        const uint32_t channel = is_value ? 2u * qk + head * p.vdim + c : (is_key ? qk : 0u) + kv_head * p.dim + c;
+        const ConvInputs<T> inputs = {projected, ring, p.stride, p.taps, channels, past};
+        value = silu_f32(inputs.convolve(b.conv_weight, column, channel, 0));
+        // keep the input: once per channel, in a ring row that this step does not read
+        if (is_value || (slice == 0u && head % (p.heads / p.kv_heads) == 0u))
+          ring[(size_t)(past % p.taps) * channels + channel] = projected[column];
+      }
+    }
+    if (is_value) v_row[index - 2u * kRow] = value;
+    else (is_key ? k_row : q_row)[c] = value;
+  }
+  __syncthreads();
+  if (!MEMORY) {  // unit vectors
+    if (warp < 2u) {
+      float* row = warp == 0u ? q_row : k_row;
+      float sum = 0.0f;
+      for (uint32_t c = lane; c < kRow; c += 32u) sum += row[c] * row[c];
+      float scale = 1.0f / sqrtf(warp_sum(sum) + 1e-6f);
+      if (warp == 0u) scale *= 1.0f / sqrtf((float)p.dim);
+      for (uint32_t c = lane; c < kRow; c += 32u) row[c] *= scale;
+    }
+    __syncthreads();
+  }
+
+  const ulonglong2* q = reinterpret_cast<const ulonglong2*>(q_row) + part;
+  const ulonglong2* k = reinterpret_cast<const ulonglong2*>(k_row) + part;
+  const Pair keep2 = pair_of(keep, keep);
+#pragma unroll
+  for (int j = 0; j < (int)kColumns; ++j) {
+    const float value = is_norm ? 1.0f : v_row[(column0 + j) % kSlice];
+    float change = write * value;
+    if (!MEMORY) {
+      Pair sum = 0ull;
+#pragma unroll
+      for (int i = 0; i < R4; ++i) {
+        const ulonglong2 kk = k[i * kLanes];
+        sum = pair_fma(s[j][2 * i], kk.x, sum);
+        sum = pair_fma(s[j][2 * i + 1], kk.y, sum);
+      }
+      float with_key = pair_sum(sum);
+#pragma unroll
+      for (int offset = 1; offset < (int)kLanes; offset <<= 1) with_key += __shfl_xor_sync(0xffffffffu, with_key, offset);
+      change = write * (value - keep * with_key);
+    }
+    const Pair change2 = pair_of(change, change);
+    Pair sum = 0ull;
+#pragma unroll
+    for (int i = 0; i < R4; ++i) {
+      const ulonglong2 kk = k[i * kLanes], qq = q[i * kLanes];
+      s[j][2 * i] = pair_fma(kk.x, change2, pair_mul(s[j][2 * i], keep2));
+      s[j][2 * i + 1] = pair_fma(kk.y, change2, pair_mul(s[j][2 * i + 1], keep2));
+      sum = pair_fma(s[j][2 * i], qq.x, sum);
+      sum = pair_fma(s[j][2 * i + 1], qq.y, sum);
+    }
+    float o = pair_sum(sum);
+#pragma unroll
+    for (int offset = 1; offset < (int)kLanes; offset <<= 1) o += __shfl_xor_sync(0xffffffffu, o, offset);
+    if (part == 0) {
+      if (is_norm) {
+        if (active[j]) norm_dot = o;
+      } else {
+        o_row[column0 + j] = o;
+      }
+    }
+  }
+  columns.store(part, p.dim, vectors);
+  if (MEMORY && threadIdx.x == 0) state[layout.top(head, slice)] = new_top;
+  __syncthreads();
+  float value = 0.0f;
+  const uint32_t column = slice * kSlice + threadIdx.x;  // of the first warp's threads
+  if (warp == 0u) {
+    value = column < p.vdim ? o_row[threadIdx.x] : 0.0f;
+    if (MEMORY) value /= fmaxf(fabsf(norm_dot), floor_value) + 1e-6f;
+    const float sum = warp_sum(value * value);
+    if (lane == 0) cta_square = sum;
+  }
+  cluster_sync();
+  if (warp == 0u) {
+    float total = 0.0f;
+    for (uint32_t other = 0; other < slices; ++other) total += cluster_load(&cta_square, other);
+    const float scale = 1.0f / sqrtf(total / (float)p.vdim + p.epsilon);
+    if (column < p.vdim) {
+      const float z = as_float(projected[p.gate_column + head * p.vdim + column]);
+      const float weight = b.norm[MEMORY ? head * p.vdim + column : column];
+      reinterpret_cast<T*>(b.out)[((size_t)sequence * p.heads + head) * p.vdim + column] =
+          from_float<T>(value * scale * weight * (MEMORY ? sigmoid_f32(z) : silu_f32(z)));
+    }
+  }
+  cluster_sync();  // nobody leaves while its sum may be read
+}
+
+// Memory: buffers [projected, scalars, norm, state, past, sequence rows, out]; delta: [projected, scalars, conv weight,
+// conv state, A_log, dt_bias, norm, state, past, sequence rows, out].
+template <typename T, bool MEMORY>
+int launch_state_step(const KernelArgs& args) {
+  StepParams p;
+  constexpr int kCount = MEMORY ? 7 : 11;
+  LLMOPT_REQUIRE(args.buffer_count == kCount && args.param_bytes == sizeof(p),
+                 "expects 7 (memory) or 11 (delta) buffers and 76 parameter bytes");
+  memcpy(&p, args.params, sizeof(p));
+  LLMOPT_REQUIRE(p.tokens == 1u && p.heads > 0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.dim > 0 && p.dim <= 256u &&
+                     p.vdim > 0,
+                 "needs one token, whole groups of heads and a key size of at most 256");
+  const uint32_t slices = slices_of(p.vdim);
+  LLMOPT_REQUIRE(slices <= 8u, "a value size of at most 256");
+  const StateRow layout = {p.heads, p.dim, p.vdim};
+  const size_t qk = (size_t)p.kv_heads * p.dim, vs = (size_t)p.heads * p.vdim, rows = p.sequences;
+  LLMOPT_REQUIRE(p.q_column + qk <= p.stride && p.k_column + qk <= p.stride && p.v_column + vs <= p.stride &&
+                     p.gate_column + vs <= p.stride && p.first_column + p.heads <= p.scalar_stride &&
+                     p.second_column + p.heads <= p.scalar_stride,
+                 "columns lie outside their rows");
+  LLMOPT_REQUIRE(p.state_rows > 0 && p.state_stride >= layout.elements(MEMORY), "state rows are too short");
+  LLMOPT_REQUIRE(!MEMORY || p.gate_cap > 0.0f, "the gate cap must be positive");
+  LLMOPT_REQUIRE(MEMORY || p.taps > 0, "a convolution needs taps");
+  StepBuffers b = {};
+  int next = 0;
+  bool ok = true;
+  auto take = [&](auto& target, size_t bytes) {
+    ok = ok && args.lengths[next] >= bytes;
+    target = reinterpret_cast<std::remove_reference_t<decltype(target)>>(args.buffers[next]);
+    ++next;
+  };
+  take(b.projected, rows * p.stride * sizeof(T));
+  take(b.scalars, rows * p.scalar_stride * 4);
+  if (!MEMORY) {
+    take(b.conv_weight, (2 * qk + vs) * p.taps * 4);
+    take(b.conv_state, p.state_rows * (2 * qk + vs) * p.taps * sizeof(T));
+    take(b.a_log, (size_t)p.heads * 4);
+    take(b.dt_bias, (size_t)p.heads * 4);
+  }
+  take(b.norm, (MEMORY ? vs : (size_t)p.vdim) * 4);
+  take(b.state, (size_t)p.state_rows * p.state_stride * 4);
+  take(b.past, rows * 4);
+  take(b.sequence_rows, rows * 4);
+  take(b.out, rows * vs * sizeof(T));
+  LLMOPT_REQUIRE(ok, "buffer is too short");
+  LLMOPT_REQUIRE(p.sequences <= 65535u && p.heads <= 65535u, "too many sequences or heads");
+  if (rows == 0) return 0;
+  auto run = [&](auto kernel) {
+    launch_cluster_kernel(args, kernel, dim3(slices, p.heads, p.sequences), dim3(step_threads<MEMORY>()), 0, slices, b, p);
+    return check_launch(args);
+  };
+  const uint32_t quads = (p.dim + kLanes * 4u - 1u) / (kLanes * 4u);
+  if (quads <= 1u) return run(state_step_kernel<T, MEMORY, 1>);
+  if (quads <= 2u) return run(state_step_kernel<T, MEMORY, 2>);
+  if (quads <= 3u) return run(state_step_kernel<T, MEMORY, 3>);
+  return run(state_step_kernel<T, MEMORY, 4>);
+}
+
 }  // namespace
 
 const NamedLauncher* matrix_state_launchers(size_t* count) {
@@ -630,6 +997,10 @@ const NamedLauncher* matrix_state_launchers(size_t* count) {
       {"llmopt_delta_scan_f32", launch_scan<float, false>},
       {"llmopt_memory_scan_bf16", launch_scan<bf16, true>},
       {"llmopt_memory_scan_f32", launch_scan<float, true>},
+      {"llmopt_delta_step_bf16", launch_state_step<bf16, false>},
+      {"llmopt_delta_step_f32", launch_state_step<float, false>},
+      {"llmopt_memory_step_bf16", launch_state_step<bf16, true>},
+      {"llmopt_memory_step_f32", launch_state_step<float, true>},
   };
   *count = sizeof(table) / sizeof(table[0]);
   return table;

@@ -19,6 +19,20 @@ __global__ void __launch_bounds__(256) embedding_residual_kernel(const long long
   grid_chain_prologue();
   const uint32_t row = blockIdx.x;
   const size_t token = min((unsigned long long)ids[row], (unsigned long long)(vocabulary - 1u));
+  constexpr uint32_t kVector = 16 / sizeof(T);
+  if (width % kVector == 0) {  // 16 bytes of the table at a time (buffers are 16-byte aligned: checked at launch)
+    for (uint32_t c = threadIdx.x * kVector; c < width; c += blockDim.x * kVector) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(table + token * width + c);
+      const T* values = reinterpret_cast<const T*>(&raw);
+      float4* target = reinterpret_cast<float4*>(x + (size_t)row * width + c);
+#pragma unroll
+      for (uint32_t i = 0; i < kVector / 4; ++i)
+        target[i] = make_float4(as_float(values[4 * i]), as_float(values[4 * i + 1]), as_float(values[4 * i + 2]),
+                                as_float(values[4 * i + 3]));
+      if (sizeof(T) != 4) *reinterpret_cast<uint4*>(x_copy + (size_t)row * width + c) = raw;
+    }
+    return;
+  }
   for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) {
     const T value = table[token * width + c];
     x[(size_t)row * width + c] = as_float(value);
@@ -35,6 +49,7 @@ int launch_embedding_residual(const KernelArgs& args) {
   LLMOPT_REQUIRE(args.lengths[0] >= (size_t)rows * 8 && args.lengths[1] >= (size_t)vocabulary * width * sizeof(T) &&
                      args.lengths[2] >= (size_t)rows * width * 4 && args.lengths[3] >= (size_t)rows * width * sizeof(T),
                  "buffer is too short");
+  for (int i = 1; i < 4; ++i) LLMOPT_REQUIRE(((uintptr_t)args.buffers[i] & 15u) == 0, "buffers must be 16-byte aligned");
   if (rows == 0) return 0;
   launch_kernel(args, embedding_residual_kernel<T>, dim3(rows), dim3(256), 0, (const long long*)args.buffers[0],
                 (const T*)args.buffers[1], (float*)args.buffers[2], (T*)args.buffers[3], rows, vocabulary, width);
@@ -187,11 +202,35 @@ __global__ void __launch_bounds__(256) gather_norm_kernel(const float* x, const 
   grid_chain_prologue();
   __shared__ float scratch[8];
   const float* source = x + (size_t)min(rows[blockIdx.x], source_rows - 1u) * width;
+  T* target = out + (size_t)blockIdx.x * width;
+  constexpr int kVectors = 4;  // float4 of a row a thread keeps between the passes
+  if (width % 4u == 0 && width <= 1024u * kVectors) {
+    float4 value[kVectors];
+    float sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kVectors; ++i) {
+      const uint32_t c = (threadIdx.x + i * 256u) * 4u;
+      value[i] = *reinterpret_cast<const float4*>(source + min(c, width - 4u));
+      if (c < width)
+        sum += value[i].x * value[i].x + value[i].y * value[i].y + value[i].z * value[i].z + value[i].w * value[i].w;
+    }
+    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + epsilon);
+#pragma unroll
+    for (int i = 0; i < kVectors; ++i) {
+      const uint32_t c = (threadIdx.x + i * 256u) * 4u;
+      if (c >= width) continue;
+      const float4 weight = *reinterpret_cast<const float4*>(w + c);
+      target[c] = from_float<T>(value[i].x * scale * (weight_offset + weight.x));
+      target[c + 1] = from_float<T>(value[i].y * scale * (weight_offset + weight.y));
+      target[c + 2] = from_float<T>(value[i].z * scale * (weight_offset + weight.z));
+      target[c + 3] = from_float<T>(value[i].w * scale * (weight_offset + weight.w));
+    }
+    return;
+  }
   float sum = 0.0f;
   for (uint32_t c = threadIdx.x; c < width; c += 256u) sum += source[c] * source[c];
   const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + epsilon);
-  for (uint32_t c = threadIdx.x; c < width; c += 256u)
-    out[(size_t)blockIdx.x * width + c] = from_float<T>(source[c] * scale * (weight_offset + w[c]));
+  for (uint32_t c = threadIdx.x; c < width; c += 256u) target[c] = from_float<T>(source[c] * scale * (weight_offset + w[c]));
 }
 
 // Buffers [x, rows u32, weight, out]; params {count, source rows, width, epsilon, weight offset}.
@@ -203,6 +242,7 @@ int launch_gather_norm(const KernelArgs& args) {
   LLMOPT_REQUIRE(args.lengths[0] >= (size_t)source_rows * width * 4 && args.lengths[1] >= (size_t)count * 4 &&
                      args.lengths[2] >= (size_t)width * 4 && args.lengths[3] >= (size_t)count * width * sizeof(T),
                  "buffer is too short");
+  for (int i : {0, 2, 3}) LLMOPT_REQUIRE(((uintptr_t)args.buffers[i] & 15u) == 0, "buffers must be 16-byte aligned");
   if (count == 0) return 0;
   launch_kernel(args, gather_norm_kernel<T>, dim3(count), dim3(256), 0, (const float*)args.buffers[0],
                 (const uint32_t*)args.buffers[1], (const float*)args.buffers[2], (T*)args.buffers[3], source_rows, width,
@@ -220,74 +260,111 @@ struct AttentionPrepareParams {
   uint32_t table_stride, table_rows, pool_rows;
   uint32_t head_norm;
   float epsilon;
+  uint32_t pairs;  // set by the launcher: every head starts at an even element
 };
 
-// One warp per (row, head): query heads are normed, rotated and stored; key heads too, into the
-// cache row of the token; value heads are copied there.  Dimensions 2i, 2i + 1 turn together; `trig`
-// holds [positions][dims / 2] pairs (cos, sin).
+// One CTA per row (or, with few rows, several that share its heads), its warps take the heads in turn: query heads are
+// normed, rotated and stored; key heads too, into the cache row of the token; value heads are copied there.
+// Dimensions 2i, 2i + 1 turn together; `trig` holds [positions][dims / 2] pairs (cos, sin).
 template <typename T>
-__global__ void __launch_bounds__(128) attention_prepare_kernel(const T* projected, const float* __restrict__ q_weight,
+__global__ void __launch_bounds__(256) attention_prepare_kernel(const T* projected, const float* __restrict__ q_weight,
                                                                 const float* __restrict__ k_weight,
                                                                 const float2* __restrict__ trig, T* q_out, T* pool,
                                                                 const uint32_t* slots, const uint32_t* past,
                                                                 const uint32_t* sequence_rows, AttentionPrepareParams p,
                                                                 uint32_t* error_word) {
   grid_chain_prologue();
-  const uint32_t lane = threadIdx.x & 31u, item = blockIdx.x * 4u + (threadIdx.x >> 5);
-  const uint32_t per_row = p.heads + 2u * p.kv_heads;
-  if (item >= p.sequences * p.tokens * per_row) return;
-  const uint32_t row = item / per_row, head = item % per_row, sequence = row / p.tokens;
-  const uint32_t position = past[sequence] + row % p.tokens;
-  const T* source = projected + (size_t)row * p.stride;
-  if (head < p.heads) source += p.q_column + head * p.dim;
-  else if (head < p.heads + p.kv_heads) source += p.k_column + (head - p.heads) * p.dim;
-  else source += p.v_column + (head - p.heads - p.kv_heads) * p.vdim;
-
-  T* target;
-  if (head < p.heads) {
-    target = q_out + ((size_t)row * p.heads + head) * p.dim;
-  } else {
-    const uint32_t table_row = sequence_rows[sequence];
-    uint32_t slot = p.pool_rows;
-    if (table_row < p.table_rows && position < p.table_stride) slot = slots[(size_t)table_row * p.table_stride + position];
-    if (slot >= p.pool_rows) {  // never write outside the pool
-      if (error_word && lane == 0) atomicExch(error_word, 1u);
-      return;
-    }
-    target = pool + (size_t)slot * p.token_stride;
-    if (head >= p.heads + p.kv_heads) {
-      target += p.value_offset + (head - p.heads - p.kv_heads) * p.vdim;
-      for (uint32_t c = lane; c < p.vdim; c += 32u) target[c] = source[c];
-      return;
-    }
-    target += p.key_offset + (head - p.heads) * p.dim;
-  }
-  const float* weight = head < p.heads ? q_weight : k_weight;
-  float scale = 1.0f;
-  if (p.head_norm) {
-    float sum = 0.0f;
-    for (uint32_t c = lane; c < p.dim; c += 32u) {
-      const float v = as_float(source[c]);
-      sum += v * v;
-    }
-    scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
-  }
+  const uint32_t lane = threadIdx.x & 31u, row = blockIdx.x, sequence = row / p.tokens;
+  const uint32_t position = past[sequence] + row % p.tokens, table_row = sequence_rows[sequence];
+  uint32_t slot = p.pool_rows;
+  if (table_row < p.table_rows && position < p.table_stride) slot = slots[(size_t)table_row * p.table_stride + position];
+  if (slot >= p.pool_rows && error_word && threadIdx.x == 0) atomicExch(error_word, 1u);
+  T* const cached = pool + (size_t)(slot < p.pool_rows ? slot : 0u) * p.token_stride;
   const uint32_t trig_row = min(position, p.trig_rows - 1u);
-  for (uint32_t pair = lane; pair * 2u < p.dim; pair += 32u) {
-    const uint32_t c = pair * 2u;
-    float u = as_float(source[c]) * scale, v = c + 1u < p.dim ? as_float(source[c + 1u]) * scale : 0.0f;
+  const float2* turns = trig + (size_t)trig_row * (p.rotary_dims / 2u);
+  const uint32_t per_row = p.heads + 2u * p.kv_heads;
+  for (uint32_t head = blockIdx.y * 8u + (threadIdx.x >> 5); head < per_row; head += 8u * gridDim.y) {
+    const T* source = projected + (size_t)row * p.stride;
+    if (head < p.heads) source += p.q_column + head * p.dim;
+    else if (head < p.heads + p.kv_heads) source += p.k_column + (head - p.heads) * p.dim;
+    else source += p.v_column + (head - p.heads - p.kv_heads) * p.vdim;
+
+    T* target;
+    if (head < p.heads) {
+      target = q_out + ((size_t)row * p.heads + head) * p.dim;
+    } else {
+      if (slot >= p.pool_rows) continue;  // never write outside the pool
+      target = cached;
+      if (head >= p.heads + p.kv_heads) {
+        target += p.value_offset + (head - p.heads - p.kv_heads) * p.vdim;
+        for (uint32_t c = lane; c < p.vdim; c += 32u) target[c] = source[c];
+        continue;
+      }
+      target += p.key_offset + (head - p.heads) * p.dim;
+    }
+    const float* weight = head < p.heads ? q_weight : k_weight;
+    if (p.pairs) {  // neighbours travel together, the head in registers between the passes
+      constexpr int kPairs = 4;  // dim <= 256
+      struct alignas(2 * sizeof(T)) Two {
+        T u, v;
+      };
+      Two raw[kPairs];
+      float sum = 0.0f;
+#pragma unroll
+      for (int i = 0; i < kPairs; ++i)
+        if (i * 64u < p.dim) raw[i] = *reinterpret_cast<const Two*>(source + min((lane + i * 32u) * 2u, p.dim - 2u));
+#pragma unroll
+      for (int i = 0; i < kPairs; ++i)
+        if ((lane + i * 32u) * 2u < p.dim) sum += as_float(raw[i].u) * as_float(raw[i].u) + as_float(raw[i].v) * as_float(raw[i].v);
+      const float scale = p.head_norm ? 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon) : 1.0f;
+#pragma unroll
+      for (int i = 0; i < kPairs; ++i) {
+        const uint32_t pair = lane + i * 32u, c = pair * 2u;
+        if (c >= p.dim) continue;
+        float u = as_float(raw[i].u) * scale, v = as_float(raw[i].v) * scale;
+        if (p.head_norm) {
+          const float2 w = *reinterpret_cast<const float2*>(weight + c);
+          u *= w.x;
+          v *= w.y;
+        }
+        if (c < p.rotary_dims) {
+          const float2 turn = turns[pair];
+          const float rotated = u * turn.x - v * turn.y;
+          v = v * turn.x + u * turn.y;
+          u = rotated;
+        }
+        Two result;
+        result.u = from_float<T>(u);
+        result.v = from_float<T>(v);
+        *reinterpret_cast<Two*>(target + c) = result;
+      }
+      continue;
+    }
+    float scale = 1.0f;
     if (p.head_norm) {
-      u *= weight[c];
-      if (c + 1u < p.dim) v *= weight[c + 1u];
+      float sum = 0.0f;
+      for (uint32_t c = lane; c < p.dim; c += 32u) {
+        const float v = as_float(source[c]);
+        sum += v * v;
+      }
+      scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
     }
-    if (c + 1u < p.rotary_dims) {
-      const float2 turn = trig[(size_t)trig_row * (p.rotary_dims / 2u) + pair];
-      const float rotated = u * turn.x - v * turn.y;
-      v = v * turn.x + u * turn.y;
-      u = rotated;
+    for (uint32_t pair = lane; pair * 2u < p.dim; pair += 32u) {
+      const uint32_t c = pair * 2u;
+      float u = as_float(source[c]) * scale, v = c + 1u < p.dim ? as_float(source[c + 1u]) * scale : 0.0f;
+      if (p.head_norm) {
+        u *= weight[c];
+        if (c + 1u < p.dim) v *= weight[c + 1u];
+      }
+      if (c + 1u < p.rotary_dims) {
+        const float2 turn = turns[pair];
+        const float rotated = u * turn.x - v * turn.y;
+        v = v * turn.x + u * turn.y;
+        u = rotated;
+      }
+      target[c] = from_float<T>(u);
+      if (c + 1u < p.dim) target[c + 1u] = from_float<T>(v);
     }
-    target[c] = from_float<T>(u);
-    if (c + 1u < p.dim) target[c + 1u] = from_float<T>(v);
   }
 }
 
@@ -299,8 +376,12 @@ namespace {
 template <typename T>
 int launch_attention_prepare(const KernelArgs& args) {
   AttentionPrepareParams p;
-  LLMOPT_REQUIRE(args.buffer_count == 9 && args.param_bytes == sizeof(p), "expects 9 buffers and 80 parameter bytes");
-  memcpy(&p, args.params, sizeof(p));
+  LLMOPT_REQUIRE(args.buffer_count == 9 && args.param_bytes == 80, "expects 9 buffers and 80 parameter bytes");
+  memcpy(&p, args.params, 80);
+  p.pairs = p.dim % 2u == 0 && p.dim <= 256u && p.stride % 2u == 0 && p.q_column % 2u == 0 && p.k_column % 2u == 0 &&
+            p.token_stride % 2u == 0 && p.key_offset % 2u == 0;
+  for (int i : {0, 1, 2, 4, 5})
+    if ((uintptr_t)args.buffers[i] & 7u) p.pairs = 0;
   const size_t rows = (size_t)p.sequences * p.tokens, e = sizeof(T);
   LLMOPT_REQUIRE(p.heads > 0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.dim > 0 && p.vdim > 0,
                  "needs whole groups of query heads");
@@ -320,8 +401,9 @@ int launch_attention_prepare(const KernelArgs& args) {
                      args.lengths[7] >= (size_t)p.sequences * 4 && args.lengths[8] >= (size_t)p.sequences * 4,
                  "cache buffer is too short");
   if (rows == 0) return 0;
-  const size_t items = rows * (p.heads + 2u * p.kv_heads);
-  launch_kernel(args, attention_prepare_kernel<T>, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0,
+  // few rows: a row's heads are spread over several CTAs
+  const uint32_t spread = rows < 256 ? (p.heads + 2u * p.kv_heads + 7u) / 8u : 1u;
+  launch_kernel(args, attention_prepare_kernel<T>, dim3((uint32_t)rows, spread), dim3(256), 0,
                 (const T*)args.buffers[0], (const float*)args.buffers[1], (const float*)args.buffers[2],
                 (const float2*)args.buffers[3], (T*)args.buffers[4], (T*)args.buffers[5], (const uint32_t*)args.buffers[6],
                 (const uint32_t*)args.buffers[7], (const uint32_t*)args.buffers[8], p, context_device_error(args.ctx));
@@ -335,6 +417,7 @@ struct HeadNormGateParams {
   uint32_t weight_per_head;  // 1: weight [heads * dim]; 0: weight [dim] shared by the heads
   uint32_t gate_sigmoid;     // 1: sigmoid, 0: silu
   float epsilon;
+  uint32_t vectors;  // set by the launcher: all rows start at whole vectors of four
 };
 
 template <typename T>
@@ -346,13 +429,45 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* o, con
   const uint32_t row = item / p.heads, head = item % p.heads;
   const float* source = o + (size_t)item * p.dim;
   const T* gate_row = gate + (size_t)row * p.gate_stride + p.gate_column + head * p.dim;
+  const float* weight_row = weight + (p.weight_per_head ? head * p.dim : 0u);
+  if (p.vectors) {  // four columns at a time, the row in registers between the passes
+    constexpr int kVectors = 4;
+    float4 value[kVectors];
+    float sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kVectors; ++i) {
+      const uint32_t c = (lane + i * 32u) * 4u;
+      value[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i * 128u < p.dim) value[i] = *reinterpret_cast<const float4*>(source + min(c, p.dim - 4u));
+      if (c < p.dim) sum += value[i].x * value[i].x + value[i].y * value[i].y + value[i].z * value[i].z + value[i].w * value[i].w;
+    }
+    const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
+#pragma unroll
+    for (int i = 0; i < kVectors; ++i) {
+      const uint32_t c = (lane + i * 32u) * 4u;
+      if (c >= p.dim) continue;
+      struct alignas(4 * sizeof(T)) Four {
+        T v[4];
+      };
+      const Four z = *reinterpret_cast<const Four*>(gate_row + c);
+      const float4 w = *reinterpret_cast<const float4*>(weight_row + c);
+      const float values[4] = {value[i].x * w.x, value[i].y * w.y, value[i].z * w.z, value[i].w * w.w};
+      Four result;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float g = as_float(z.v[e]);
+        result.v[e] = from_float<T>(values[e] * scale * (p.gate_sigmoid ? sigmoid_f32(g) : silu_f32(g)));
+      }
+      *reinterpret_cast<Four*>(out + (size_t)item * p.dim + c) = result;
+    }
+    return;
+  }
   float sum = 0.0f;
   for (uint32_t c = lane; c < p.dim; c += 32u) sum += source[c] * source[c];
   const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)p.dim + p.epsilon);
   for (uint32_t c = lane; c < p.dim; c += 32u) {
     const float z = as_float(gate_row[c]);
-    const float w = weight[p.weight_per_head ? head * p.dim + c : c];
-    out[(size_t)item * p.dim + c] = from_float<T>(source[c] * scale * w * (p.gate_sigmoid ? sigmoid_f32(z) : silu_f32(z)));
+    out[(size_t)item * p.dim + c] = from_float<T>(source[c] * scale * weight_row[c] * (p.gate_sigmoid ? sigmoid_f32(z) : silu_f32(z)));
   }
 }
 
@@ -360,8 +475,11 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* o, con
 template <typename T>
 int launch_head_norm_gate(const KernelArgs& args) {
   HeadNormGateParams p;
-  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == sizeof(p), "expects 4 buffers and 32 parameter bytes");
-  memcpy(&p, args.params, sizeof(p));
+  LLMOPT_REQUIRE(args.buffer_count == 4 && args.param_bytes == 32, "expects 4 buffers and 32 parameter bytes");
+  memcpy(&p, args.params, 32);
+  p.vectors = p.dim % 4u == 0 && p.dim <= 512u && p.gate_stride % 4u == 0 && p.gate_column % 4u == 0;
+  for (int i = 0; i < 4; ++i)
+    if ((uintptr_t)args.buffers[i] & 15u) p.vectors = 0;
   const size_t items = (size_t)p.rows * p.heads;
   LLMOPT_REQUIRE(p.gate_column + p.heads * p.dim <= p.gate_stride, "gate columns lie outside the row");
   LLMOPT_REQUIRE(args.lengths[0] >= items * p.dim * 4 && args.lengths[1] >= (size_t)p.rows * p.gate_stride * sizeof(T) &&

@@ -167,6 +167,8 @@ def _entries() -> list[Entry]:
         add("llmopt_delta_prepare_" + suffix, SHORT_CONV, element, f32)
         add("llmopt_conv_state_" + suffix, SHORT_CONV, element, element)
         add("llmopt_memory_scan_" + suffix, GATED_DELTA, element, f32)
+        add("llmopt_memory_step_" + suffix, GATED_DELTA, element, element)
+        add("llmopt_delta_step_" + suffix, GATED_DELTA, element, element)
     add("llmopt_delta_scan_f32", GATED_DELTA, f32, f32)
     add("llmopt_argmax_f32", POINTWISE, f32, i64)
     add("llmopt_advance_tokens", EMBEDDING, i64, "int32")

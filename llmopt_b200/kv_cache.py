@@ -118,9 +118,11 @@ MATRIX_STATE_SLICE = 32
 
 def matrix_state_elements(heads: int, dim: int, vdim: int, *, normalized: bool) -> int:
     """fp32 elements of one sequence's state: the transposed matrices [heads][vdim][dim] and, in the
-    normalised form, n [dim] and m per head and slice of value columns."""
+    normalised form, n [dim] and m per head and slice of value columns; a multiple of four, so that a row
+    starts at a 16-byte boundary."""
     slices = (vdim + MATRIX_STATE_SLICE - 1) // MATRIX_STATE_SLICE
-    return heads * vdim * dim + (heads * slices * (dim + 1) if normalized else 0)
+    elements = heads * vdim * dim + (heads * slices * (dim + 1) if normalized else 0)
+    return (elements + 3) // 4 * 4
 
 
 class SequenceTable:

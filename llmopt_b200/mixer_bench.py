@@ -83,7 +83,7 @@ def work_of(item, past: int, itemsize: int):
         vectors = (2 * kv_heads * dim + heads * vdim) * source + heads * (vdim * 4 + 8)
         return stem, sequences * (tokens * vectors + heads * dim * vdim * 8), 0
     if stem in ("delta_step", "memory_step"):
-        sequences, heads, kv_heads, dim, vdim = u[0], u[2], u[3], u[4], u[5]
+        sequences, heads, kv_heads, dim, vdim = u[0], u[2], u[3], u[4], u[5]  # u[1]: one token
         return stem, sequences * (heads * dim * vdim * 8 + (2 * kv_heads * dim + 3 * heads * vdim) * e), 0
     if stem == "argmax":
         return stem, u[0] * u[1] * 4, 0
@@ -223,6 +223,15 @@ def like_kernels(runtime, peaks: dict, config: MixerConfig, tokens: int, context
                             parameters.rms_norm(rows=count, width=width, epsilon=1e-5),
                             (dispatch.simd_rows_grid(count), 1, 1), (256, 1, 1))
         note(f"rms norm, {count} rows", runtime.time_dispatches([item] * 32, warmup=2, iterations=5), count * width * 4)
+        q_in, k_in = half(count, heads * 128), half(count, heads // 4 * 128)
+        rotary = DispatchItem("llmopt_rotary_qk_f16_simd_h64",
+                              [q_in.buffer, k_in.buffer, half(count, 128).buffer, half(count, 128).buffer,
+                               half(count, heads * 128).buffer, half(count, heads // 4 * 128).buffer],
+                              parameters.rotary_qk(batches=1, tokens=count, q_heads=heads, k_heads=heads // 4, width=128,
+                                                   half_dimension=64, trig_batches=1),
+                              (dispatch.simd_rows_grid(count * (heads + heads // 4)), 1, 1), (256, 1, 1))
+        note(f"rotary q k, {count} rows", runtime.time_dispatches([rotary] * 16, warmup=2, iterations=5),
+             count * (heads + heads // 4) * 128 * 4)
         conv = DispatchItem("llmopt_short_conv_silu_tm_f16", [rows.buffer, half(width, 4).buffer, half(count, width).buffer],
                             parameters.short_conv_silu_tm(batches=1, tokens=count, channels=width, kernel_width=4, stride=1,
                                                           padding=3, dilation=1, output_start=0), (1, 1, 1), (256, 1, 1))

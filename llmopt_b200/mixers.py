@@ -17,7 +17,7 @@ import numpy as np
 
 from . import parameters
 from .cuda_native import Buffer
-from .kv_cache import matrix_state_elements
+from .kv_cache import MATRIX_STATE_SLICE, matrix_state_elements
 from .model import AttentionSpec, DeltaSpec, MatrixMemorySpec, ParallelSpec
 
 
@@ -76,6 +76,14 @@ class Projection:
         engine.record_linear(step, x, self.weight, projected, m=step.rows, n=self.total, k=engine.config.width,
                              split=self.split, out32=scalars, bias=self.bias)
         return projected, scalars
+
+
+def fused_step(step: Step, spec) -> bool:
+    """Whether the one-launch form of a recurrent mixer takes this step: one token per sequence, a head's
+    value columns fit the thread blocks of one cluster, and there are few enough of those blocks for the
+    step to be a matter of launches rather than of state traffic (which the scan streams better)."""
+    slices = (spec.vdim + MATRIX_STATE_SLICE - 1) // MATRIX_STATE_SLICE
+    return step.tokens == 1 and slices <= 8 and step.sequences * spec.heads * slices <= 2048
 
 
 class AttentionMixer:
@@ -137,7 +145,7 @@ class DeltaMixer:
         self.state_stride = matrix_state_elements(spec.heads, spec.dim, spec.vdim, normalized=False)
         rows = engine.sequences.rows
         self.state = engine.empty_bytes(rows * self.state_stride * 4)
-        self.conv_state = engine.empty_bytes(max(rows * self.channels * (spec.taps - 1) * engine.itemsize, 16))
+        self.conv_state = engine.empty_bytes(rows * self.channels * spec.taps * engine.itemsize)
 
     def record(self, step: Step, projected: Buffer, scalars: Buffer, y: Buffer) -> None:
         engine, spec, columns = step.engine, self.spec, self.projection.columns
@@ -148,6 +156,19 @@ class DeltaMixer:
         shape = dict(sequences=step.sequences, tokens=step.tokens, heads=spec.heads, kv_heads=spec.kv_heads, dim=spec.dim,
                      vdim=spec.vdim)
         rows = engine.sequences.rows
+        if fused_step(step, spec):
+            step.run(step.element("delta_step"),
+                     [projected, scalars, self.conv, self.conv_state, self.a_log, self.dt_bias, self.norm, self.state, step.past,
+                      step.sequence_rows, mixed],
+                     parameters.state_step(
+                         sequences=step.sequences, heads=spec.heads, kv_heads=spec.kv_heads, dim=spec.dim, vdim=spec.vdim,
+                         taps=spec.taps, stride=self.projection.split, q_column=columns[f"{self.prefix}.q"],
+                         k_column=columns[f"{self.prefix}.k"], v_column=columns[f"{self.prefix}.v"],
+                         gate_column=columns[f"{self.prefix}.g"], scalar_stride=self.projection.scalars,
+                         first_column=columns[f"{self.prefix}.b"], second_column=columns[f"{self.prefix}.a"], state_rows=rows,
+                         state_stride=self.state_stride, gate_cap=0.0, epsilon=engine.config.epsilon))
+            engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+            return
         prepare = parameters.delta_prepare(
             **shape, taps=spec.taps, stride=self.projection.split, q_column=columns[f"{self.prefix}.q"],
             k_column=columns[f"{self.prefix}.k"], v_column=columns[f"{self.prefix}.v"],
@@ -186,6 +207,18 @@ class MatrixMemoryMixer:
         engine, spec, columns = step.engine, self.spec, self.projection.columns
         vs, stride = spec.heads * spec.vdim, self.projection.split
         read_out, mixed = engine.work32("read_out", vs), engine.work("mixed", vs)
+        if fused_step(step, spec):
+            step.run(step.element("memory_step"),
+                     [projected, scalars, self.norm, self.state, step.past, step.sequence_rows, mixed],
+                     parameters.state_step(
+                         sequences=step.sequences, heads=spec.heads, kv_heads=spec.heads, dim=spec.dim, vdim=spec.vdim, taps=0,
+                         stride=stride, q_column=columns[f"{self.prefix}.q"], k_column=columns[f"{self.prefix}.k"],
+                         v_column=columns[f"{self.prefix}.v"], gate_column=columns[f"{self.prefix}.g"],
+                         scalar_stride=self.projection.scalars, first_column=columns[f"{self.prefix}.i"],
+                         second_column=columns[f"{self.prefix}.f"], state_rows=engine.sequences.rows,
+                         state_stride=self.state_stride, gate_cap=spec.gate_cap, epsilon=engine.config.epsilon))
+            engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+            return
         step.run(step.element("memory_scan"),
                  [projected, projected, projected, scalars, scalars, self.state, step.past, step.sequence_rows, read_out],
                  parameters.state_scan(

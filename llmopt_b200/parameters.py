@@ -211,3 +211,9 @@ def state_scan(*, sequences, tokens, heads, kv_heads, dim, vdim, q_stride, q_col
                v_column, scalar_stride, first_column, second_column, state_rows, state_stride, gate_cap=0.0) -> bytes:
     return u32s([sequences, tokens, heads, kv_heads, dim, vdim, q_stride, q_column, k_stride, k_column, v_stride, v_column,
                  scalar_stride, first_column, second_column, state_rows, state_stride]) + struct.pack("<f", gate_cap)
+
+
+def state_step(*, sequences, heads, kv_heads, dim, vdim, taps, stride, q_column, k_column, v_column, gate_column,
+               scalar_stride, first_column, second_column, state_rows, state_stride, gate_cap, epsilon) -> bytes:
+    return u32s([sequences, 1, heads, kv_heads, dim, vdim, taps, stride, q_column, k_column, v_column, gate_column,
+                 scalar_stride, first_column, second_column, state_rows, state_stride]) + struct.pack("<ff", gate_cap, epsilon)

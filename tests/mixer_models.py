@@ -70,6 +70,9 @@ MODELS = {
     "odd": config_of([parallel_layer(heads=8, kv_heads=1, dim=18, vdim=10, rot={"base": 1e6, "dims": 4}, scale=0.5,
                                      right={"heads": 6, "kv_heads": 1, "dim": 10, "vdim": 33, "conv": 5}, ff=31),
                       memory_layer(heads=5, dim=7, vdim=9, gate_cap=1.0, ff=17)], width=50, vocab=61, side=3),
+    # value heads wider than one cluster of thread blocks carries
+    "tall": config_of([memory_layer(heads=1, dim=20, vdim=300), parallel_layer(right={"heads": 2, "kv_heads": 2, "dim": 12,
+                                                                                      "vdim": 264, "conv": 4})], width=56, vocab=90),
     # a kernel's own tile sizes
     "square": config_of([memory_layer(heads=2, dim=64, vdim=128, gate_cap=15.0, ff=256),
                          parallel_layer(heads=4, kv_heads=2, dim=64, vdim=64, scale=0.125,

@@ -96,7 +96,8 @@ def test_row_layout_and_state_sizes():
     assert [(r.key_offset, r.value_offset) for r in layout.regions] == [(0, 72), (192, 216)]
     assert layout.token_elements == 232 and RowLayout([]).token_elements == 8
     assert matrix_state_elements(2, 10, 33, normalized=False) == 660
-    assert matrix_state_elements(2, 10, 33, normalized=True) == 660 + 2 * 2 * 11
+    assert matrix_state_elements(3, 10, 33, normalized=True) == 990 + 3 * 2 * 11
+    assert matrix_state_elements(1, 9, 3, normalized=False) == 28  # 27 rounded up
 
 
 def test_sequence_table_hands_out_rows_and_pages_again():
