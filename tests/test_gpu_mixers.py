@@ -612,3 +612,19 @@ def test_trace_runner(runtime, tmp_path):
     reference.check(read(2), [19], "float32")
     reference.check(read(3), [0], "float32")
     assert not (out / "1.f32").exists()
+
+
+def test_generate_command(runtime, tmp_path, capsys):
+    import json
+
+    from llmopt_b200 import generate
+    from llmopt_b200.safetensors_archive import as_bfloat16_bits
+    from test_mixers_cpu import write_checkpoint
+
+    config = MODELS["mixed"]
+    weights = weights_of(config, seed=3)
+    (tmp_path / "config.json").write_text(json.dumps(config))
+    write_checkpoint(tmp_path / "model.safetensors", {name: ("BF16", as_bfloat16_bits(value)) for name, value in weights.items()})
+    generate.main(["--model", str(tmp_path), "--prompt", "3,99,41", "--prompt", "7", "--tokens", "6", "--dtype", "float32"])
+    wanted = [greedy(config, weights, prompt, 6)[0] for prompt in ([3, 99, 41], [7])]
+    assert capsys.readouterr().out.splitlines() == [",".join(map(str, tokens)) for tokens in wanted]
