@@ -14,8 +14,10 @@ OBJECTS = os.path.join(PACKAGE_DIR, "build")
 
 # Kernel families that are enough to serve one kind of model: a host that needs no others can build
 # and load libllmopt_cuda_<family>.so (the runtime registers only the names that were linked in).
+_ATTENTION = ("runtime", "sampling", "dense_linear", "dense_gemm_tc", "sequence_glue", "row_attention", "experts")
 FAMILIES = {
-    "mixers": ("runtime", "sampling", "dense_linear", "dense_gemm_tc", "sequence_glue", "row_attention", "matrix_state"),
+    "attention": _ATTENTION,  # decoders whose mixers all are attention
+    "mixers": _ATTENTION + ("matrix_state",),
 }
 
 NVCC_FLAGS = [

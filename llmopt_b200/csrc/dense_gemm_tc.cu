@@ -1,5 +1,7 @@
 // Prompt rows of the dense bfloat16 linear layer on the 5th-generation tensor cores:
 //   y[m, n] = x[m, k] . w[n, k]^T, fp32 accumulation in tensor memory.
+// With a plan the rows are sorted by expert and a tile multiplies with its expert's n rows of w [experts n, k];
+// the rows of a box that belong to the next expert are computed and dropped.
 //
 // A persistent CTA walks over 128 x BN output tiles.  Warp 0 brings the x tile [128 x 64] and the w
 // tile [BN x 64] of every k-block into a shared-memory ring by TMA (128-byte swizzle); one thread of
@@ -22,7 +24,7 @@ uint32_t* context_device_error(Context* ctx);
 
 namespace {
 
-constexpr uint32_t kRows = 128, kDepth = 64;
+constexpr uint32_t kRows = kExpertTile, kDepth = 64;
 constexpr uint32_t kEpilogueWarps = 8;
 constexpr uint32_t kThreads = (2 + kEpilogueWarps) * 32;  // TMA, MMA, epilogue
 constexpr uint32_t kXTileBytes = kRows * kDepth * 2;
@@ -49,7 +51,7 @@ __host__ __device__ constexpr uint32_t bf16_instruction(uint32_t m, uint32_t n) 
 template <uint32_t BN>
 __global__ void __launch_bounds__(kThreads, 1)
 dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                     const DenseProblem p, uint32_t* error_word) {
+                     const DenseProblem p, uint32_t most_tiles, uint32_t* error_word) {
   using S = Shape<BN>;
   extern __shared__ unsigned char shared_raw[];
   grid_chain_prologue();
@@ -60,7 +62,15 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
   volatile uint32_t* holder = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kHolder);
   volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kAbort);
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
-  const uint32_t m_tiles = (p.m + kRows - 1u) / kRows, n_tiles = (p.n + BN - 1u) / BN, tiles = m_tiles * n_tiles;
+  const uint32_t m_tiles = p.plan ? min(p.plan[0], most_tiles) : (p.m + kRows - 1u) / kRows;
+  const uint32_t n_tiles = (p.n + BN - 1u) / BN, tiles = m_tiles * n_tiles;
+  // first row, row end, and first row of the weights (column of the output) of a tile
+  auto place = [&](uint32_t tile) -> DenseTile {
+    const uint32_t m_tile = tile % m_tiles, n0 = tile / m_tiles * BN;
+    if (!p.plan) return {n0, m_tile * kRows, p.m};
+    const DenseTile rows = dense_tile(p, m_tile);
+    return {rows.expert * p.n + n0, rows.first, min(rows.end, p.m)};
+  };
   const uint32_t k_stages = (p.k + kDepth * S::kBlocks - 1u) / (kDepth * S::kBlocks);
 
   if (threadIdx.x == 0) {
@@ -95,7 +105,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
       uint32_t issued = 0;  // k-blocks over all tiles of this CTA
       bool ok = true;
       for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
-        const uint32_t m0 = (tile % m_tiles) * kRows, n0 = (tile / m_tiles) * BN;
+        const DenseTile at = place(tile);
         for (uint32_t ks = 0; ks < k_stages; ++ks, ++issued) {
           const uint32_t s = issued % S::kStages;
           ok = !*abort_flag && barrier_wait(empty + s * 8, ((issued / S::kStages) & 1u) ^ 1u);
@@ -108,8 +118,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
 #pragma unroll
           for (uint32_t block = 0; block < S::kBlocks; ++block) {
             const int32_t k0 = (int32_t)((ks * S::kBlocks + block) * kDepth);
-            tma_load_2d(stage + block * kXTileBytes, &map_x, k0, (int32_t)m0, full + s * 8);
-            tma_load_2d(stage + S::kBlocks * kXTileBytes + block * S::kWTileBytes, &map_w, k0, (int32_t)n0, full + s * 8);
+            tma_load_2d(stage + block * kXTileBytes, &map_x, k0, (int32_t)at.first, full + s * 8);
+            tma_load_2d(stage + S::kBlocks * kXTileBytes + block * S::kWTileBytes, &map_w, k0, (int32_t)at.expert, full + s * 8);
           }
         }
       }
@@ -158,7 +168,10 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
         break;
       }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const uint32_t row = (tile % m_tiles) * kRows + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
+      const DenseTile rows = place(tile);
+      const uint32_t row = rows.first + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
+      bf16* const cached = p.cache.pool && row < p.m ? dense_cache_row<bf16>(p, row) : nullptr;
+      const uint32_t kept = dense_cache_columns(p);
       const uint32_t address = tmem_base + half * BN + ((quarter * 32u) << 16);
 #pragma unroll 1
       for (uint32_t piece = side; piece < BN / 32u; piece += kEpilogueWarps / 4u) {
@@ -167,10 +180,65 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         const uint32_t column = n0 + piece * 32u;
         const size_t at = (size_t)row * p.split + column;
-        const size_t at32 = (size_t)row * (p.n - p.split) + (column - p.split);
-        if (row >= p.m || column >= p.n) {
+        const size_t at32 = (size_t)row * (p.n - p.split - kept) + (column - p.split - kept);
+        if (row >= rows.end || column >= p.n) {
           // absent
-        } else if (column + 32u <= p.split && (at & 7u) == 0) {
+        } else if (p.epilogue == kDenseSiluPair) {
+          bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * (p.n / 2u) + column / 2u;
+          const bool whole = column + 32u <= p.n && ((uintptr_t)target & 15u) == 0;
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            uint32_t packed[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const int e = i * 16 + j * 4;
+              float pair[2];
+#pragma unroll
+              for (int h = 0; h < 2; ++h)
+                pair[h] = column + e + 2 * h < p.n ? dense_pair(p, row, column + e + 2 * h, __uint_as_float(raw[e + 2 * h]),
+                                                                __uint_as_float(raw[e + 2 * h + 1]))
+                                                   : 0.0f;
+              const __nv_bfloat162 both = __floats2bfloat162_rn(pair[0], pair[1]);
+              packed[j] = *reinterpret_cast<const uint32_t*>(&both);
+              if (!whole) {
+                if (column + e < p.n) target[i * 8 + j * 2] = both.x;
+                if (column + e + 2 < p.n) target[i * 8 + j * 2 + 1] = both.y;
+              }
+            }
+            if (whole) reinterpret_cast<uint4*>(target)[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+          }
+        } else if (p.epilogue == kDenseResidualTanh && column + 32u <= p.n && p.n % 4u == 0) {
+          const TanhNorm post(p.post_norm, p.n), next(p.next_norm, p.n);
+          float* residual = p.residual + (size_t)row * p.n + column;
+          bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * p.n + column;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            float v[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[j] = dense_finish<bf16>(p, row, column + i * 4 + j, __uint_as_float(raw[i * 4 + j]));
+            float4 x = reinterpret_cast<const float4*>(residual)[i];
+            const float4 y = post.four(make_float4(v[0], v[1], v[2], v[3]), column + i * 4);
+            x.x += y.x, x.y += y.y, x.z += y.z, x.w += y.w;
+            reinterpret_cast<float4*>(residual)[i] = x;
+            store_four(target + i * 4, next.four(x, column + i * 4));
+          }
+        } else if (p.epilogue != kDenseResidualTanh && column >= p.split && column + 32u <= p.split + kept) {
+          // one head may end and the next begin inside the piece, and keys may end and values begin
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            const uint32_t at_cache = column - p.split + i;
+            if (!cached) continue;
+            const float low = dense_finish<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+            const float high = dense_finish<bf16>(p, row, column + i + 1, __uint_as_float(raw[i + 1]));
+            const uint32_t first = dense_cache_offset(p.cache, at_cache), second = dense_cache_offset(p.cache, at_cache + 1u);
+            if (second == first + 1u && (((uintptr_t)(cached + first)) & 3u) == 0) {
+              *reinterpret_cast<__nv_bfloat162*>(cached + first) = __floats2bfloat162_rn(low, high);
+            } else {
+              cached[first] = __float2bfloat16_rn(low);
+              cached[second] = __float2bfloat16_rn(high);
+            }
+          }
+        } else if (p.epilogue != kDenseResidualTanh && column + 32u <= p.split && (at & 7u) == 0) {
           uint4* target = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + at);
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -185,7 +253,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
             }
             target[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
           }
-        } else if (column >= p.split && column + 32u <= p.n && (at32 & 3u) == 0) {
+        } else if (p.epilogue != kDenseResidualTanh && column >= p.split + kept && column + 32u <= p.n && (at32 & 3u) == 0) {
           float4* target = reinterpret_cast<float4*>(p.out32 + at32);
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
@@ -239,18 +307,26 @@ bool make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer
                 CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+// Row tiles; of rows sorted by expert, the most there can be.
+uint32_t most_tiles(const DenseProblem& p) {
+  if (!p.plan) return (p.m + kRows - 1u) / kRows;
+  return p.m / kRows + (p.experts < p.m ? p.experts : p.m);
+}
+
 template <uint32_t BN>
 int run(const KernelArgs& args, const DenseProblem& p, uint32_t sms) {
   using S = Shape<BN>;
   CUtensorMap map_x, map_w;
-  if (!make_map(&map_x, p.x, p.k, p.m, kRows) || !make_map(&map_w, p.w, p.k, p.n, BN)) return -1;
+  if (!make_map(&map_x, p.x, p.k, p.m, kRows) ||
+      !make_map(&map_w, p.w, p.k, (uint64_t)p.n * (p.plan ? p.experts : 1u), BN))
+    return -1;
   auto kernel = dense_gemm_tc_kernel<BN>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSharedBytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
   }
-  const uint32_t tiles = ((p.m + kRows - 1u) / kRows) * ((p.n + BN - 1u) / BN);
-  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, p,
+  const uint32_t most = most_tiles(p), tiles = most * ((p.n + BN - 1u) / BN);
+  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, p, most,
                 context_device_error(args.ctx));
   return check_launch(args);
 }
@@ -261,7 +337,7 @@ int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& p) {
   if (args.ctx == nullptr || p.k % 8u != 0 || ((uintptr_t)p.x & 15u) != 0 || ((uintptr_t)p.w & 15u) != 0) return -1;
   const uint32_t sms = (uint32_t)context_sm_count(args.ctx);
   // waves times the cost of one MMA (an MMA of up to 128 columns costs about two thirds of one of 256)
-  const uint32_t m_tiles = (p.m + kRows - 1u) / kRows;
+  const uint32_t m_tiles = most_tiles(p);
   auto cost = [&](uint32_t columns, uint32_t mma) {
     const uint32_t tiles = m_tiles * ((p.n + columns - 1u) / columns);
     return (tiles + sms - 1u) / sms * mma;

@@ -2,8 +2,11 @@
 //   llmopt_row_attention_{bf16,f32}
 // A sequence's token p sits in pool row slots[sequence row][p]; a pool row holds, per attention layer, the
 // kv_heads key vectors (size dim) and value vectors (size vdim, which may differ).  The rows of the step's
-// own tokens are in the pool already.  Row t of a sequence sees keys 0 .. past + t.  With `sink` the softmax
-// denominator counts one more score of zero that has no value.
+// own tokens are in the pool already.  Row t of a sequence sees keys 0 .. past + t; with a `window` only the
+// last `window` of them (its own included) and the first `keep_first` of the sequence.  With `softcap` a score
+// becomes softcap * tanh(score / softcap).  With `sink` the softmax denominator counts one more score of zero that
+// has no value.  With `gate_stride` the read-out is multiplied by the sigmoid of the row's gate columns.
+// Queries and gates are read where the projections left them: row stride, first column.
 //
 // Kernels behind the names:
 //  * bf16, at most 16 (query head, token) rows per key/value head (decode): split over the keys;
@@ -26,7 +29,10 @@ struct RowAttentionParams {
   uint32_t token_stride, key_offset, value_offset;  // in elements
   uint32_t table_stride, table_rows, pool_rows;
   uint32_t sink, splits;
-  float scale;
+  float scale, softcap;        // 0: scores are not capped
+  uint32_t window, keep_first; // 0: no window
+  uint32_t query_stride, query_column, gate_stride, gate_column;  // in elements; gate_stride 0: no gate
+  uint32_t weights32;  // softmax weights meet the values in 32 bits (two bfloat16 parts), not rounded to bfloat16
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
@@ -48,28 +54,50 @@ __device__ __forceinline__ KeyRows key_rows(const RowAttentionParams& p, const u
   return {table + (present ? (size_t)row * p.table_stride : 0u), present ? p.table_stride : 0u, p.pool_rows};
 }
 
+// The keys a run of rows sees, positions first .. last of them: the kept ones, then those from `begin` on.
+struct Visible {
+  uint32_t kept, begin, end;
+  __device__ __forceinline__ Visible(const RowAttentionParams& p, uint32_t first, uint32_t last) {
+    end = last + 1u;
+    begin = p.window && first + 1u > p.window ? first + 1u - p.window : 0u;
+    kept = p.window ? min(p.keep_first, begin) : 0u;
+  }
+  __device__ __forceinline__ uint32_t count() const { return kept + end - begin; }
+  __device__ __forceinline__ uint32_t position(uint32_t index) const { return index < kept ? index : index - kept + begin; }
+};
+__device__ __forceinline__ bool sees(const RowAttentionParams& p, uint32_t position, uint32_t key) {
+  return key <= position && (!p.window || position - key < p.window || key < p.keep_first);
+}
+
+// Factor of a read-out.
+template <typename T>
+__device__ __forceinline__ float gate_of(const RowAttentionParams& p, const T* gate, size_t row, uint32_t head, uint32_t column) {
+  return p.gate_stride ? sigmoid_f32(as_float(gate[row * p.gate_stride + p.gate_column + head * p.vdim + column])) : 1.0f;
+}
+
 // ---- one warp per (row, head) --------------------------------------------------------------------
 template <typename T, int SEGMENTS>
 __global__ void __launch_bounds__(128) attention_rows_kernel(const T* query, const T* pool, const uint32_t* table,
                                                              const uint32_t* past, const uint32_t* sequence_rows, T* out,
-                                                             RowAttentionParams p, uint32_t* error_word) {
+                                                             const T* gate, RowAttentionParams p, uint32_t* error_word) {
   grid_chain_prologue();
   const uint32_t lane = threadIdx.x & 31u, item = blockIdx.x * 4u + (threadIdx.x >> 5);
   if (item >= p.sequences * p.tokens * p.heads) return;
   const uint32_t row = item / p.heads, head = item % p.heads, sequence = row / p.tokens;
   const uint32_t kv_head = head / (p.heads / p.kv_heads);
-  const uint32_t keys = past[sequence] + row % p.tokens + 1u;
+  const uint32_t position = past[sequence] + row % p.tokens;
+  const Visible visible(p, position, position);
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
   float q[SEGMENTS], o[SEGMENTS];
 #pragma unroll
   for (int s = 0; s < SEGMENTS; ++s) {
     const uint32_t c = lane + s * 32u;
-    q[s] = c < p.dim ? as_float(query[(size_t)item * p.dim + c]) : 0.0f;
+    q[s] = c < p.dim ? as_float(query[(size_t)row * p.query_stride + p.query_column + head * p.dim + c]) : 0.0f;
     o[s] = 0.0f;
   }
   float top = p.sink ? 0.0f : kLowest, total = p.sink ? 1.0f : 0.0f;
-  for (uint32_t key = 0; key < keys; ++key) {
-    const T* cached = pool + (size_t)rows(key, error_word) * p.token_stride;
+  for (uint32_t index = 0; index < visible.count(); ++index) {
+    const T* cached = pool + (size_t)rows(visible.position(index), error_word) * p.token_stride;
     const T* k = cached + p.key_offset + kv_head * p.dim;
     const T* v = cached + p.value_offset + kv_head * p.vdim;
     float score = 0.0f;
@@ -79,6 +107,7 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(const T* query, con
       if (c < p.dim) score = fmaf(q[s], as_float(k[c]), score);
     }
     score = warp_sum(score) * p.scale;
+    if (p.softcap > 0.0f) score = p.softcap * tanhf(score / p.softcap);
     const float next = fmaxf(top, score), keep = expf(top - next), weight = expf(score - next);
     top = next;
     total = total * keep + weight;
@@ -91,7 +120,7 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(const T* query, con
 #pragma unroll
   for (int s = 0; s < SEGMENTS; ++s) {
     const uint32_t c = lane + s * 32u;
-    if (c < p.vdim) out[(size_t)item * p.vdim + c] = from_float<T>(o[s] / total);
+    if (c < p.vdim) out[(size_t)item * p.vdim + c] = from_float<T>(o[s] / total * gate_of(p, gate, row, head, c));
   }
 }
 
@@ -128,7 +157,8 @@ __host__ __device__ constexpr uint32_t round16(uint32_t v) { return (v + 15u) & 
 
 // Online softmax of one warp's 16 rows (this lane: rows r and r + 8) over KEYS keys, scores already in units
 // of log2 e with invisible ones at -inf; then O += P V from the value tile at `v_tile` (row stride v_stride).
-template <int KEYS, int DV>
+// FINE: P enters the product as its bfloat16 rounding plus the bfloat16 rounding of what that leaves.
+template <int KEYS, int DV, bool FINE>
 struct Softmax {
   float top[2], total[2], out[DV / 8][4];
   __device__ __forceinline__ void reset() {
@@ -158,7 +188,7 @@ struct Softmax {
         out[t][2 * h + 1] *= keep;
       }
     }
-    uint32_t weights[KEYS / 16][4];
+    uint32_t weights[KEYS / 16][4], rests[FINE ? KEYS / 16 : 1][4];
 #pragma unroll
     for (int j = 0; j < KEYS / 8; ++j) {
       float e[4];
@@ -169,6 +199,12 @@ struct Softmax {
       const __nv_bfloat162 low = __floats2bfloat162_rn(e[0], e[1]), high = __floats2bfloat162_rn(e[2], e[3]);
       weights[j >> 1][(j & 1) * 2] = *reinterpret_cast<const uint32_t*>(&low);
       weights[j >> 1][(j & 1) * 2 + 1] = *reinterpret_cast<const uint32_t*>(&high);
+      if (FINE) {
+        const __nv_bfloat162 low_rest = __floats2bfloat162_rn(e[0] - __low2float(low), e[1] - __high2float(low));
+        const __nv_bfloat162 high_rest = __floats2bfloat162_rn(e[2] - __low2float(high), e[3] - __high2float(high));
+        rests[FINE ? j >> 1 : 0][(j & 1) * 2] = *reinterpret_cast<const uint32_t*>(&low_rest);
+        rests[FINE ? j >> 1 : 0][(j & 1) * 2 + 1] = *reinterpret_cast<const uint32_t*>(&high_rest);
+      }
     }
 #pragma unroll
     for (int s = 0; s < KEYS / 16; ++s)
@@ -178,7 +214,22 @@ struct Softmax {
         ldmatrix_x4_trans(b, v_tile + (16 * s + (lane & 7u) + ((lane >> 3) & 1u) * 8u) * v_stride + 16 * t + (lane >> 4) * 8u);
         mma_bf16(out[2 * t], weights[s], b[0], b[1]);
         mma_bf16(out[2 * t + 1], weights[s], b[2], b[3]);
+        if (FINE) {
+          mma_bf16(out[2 * t], rests[FINE ? s : 0], b[0], b[1]);
+          mma_bf16(out[2 * t + 1], rests[FINE ? s : 0], b[2], b[3]);
+        }
       }
+  }
+};
+
+// A raw score in units of log2 e.
+struct ScoreScale {
+  float scale, cap;  // cap 0: none
+  __device__ __forceinline__ explicit ScoreScale(const RowAttentionParams& p)
+      : scale(p.softcap > 0.0f ? p.scale / p.softcap : p.scale * kLog2e), cap(p.softcap * kLog2e) {}
+  __device__ __forceinline__ float operator()(float raw) const {
+    const float score = raw * scale;
+    return cap > 0.0f ? cap * tanh_f32(score) : score;
   }
 };
 
@@ -215,10 +266,10 @@ __device__ __forceinline__ void scores(float (&score)[KEYS / 8][4], const uint32
 // ---- prompts -------------------------------------------------------------------------------------
 constexpr uint32_t kQueryTile = 64, kKeyTile = 64;
 
-template <int DK, int DV>
+template <int DK, int DV, bool FINE>
 __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
                                                                const uint32_t* past_lengths, const uint32_t* sequence_rows,
-                                                               bf16* out, RowAttentionParams p, uint32_t* error_word) {
+                                                               bf16* out, const bf16* gate, RowAttentionParams p, uint32_t* error_word) {
   grid_chain_prologue();
   extern __shared__ __align__(16) unsigned char attention_shared[];
   const uint32_t padded = DK > 0 ? DK : round16(p.dim), k_stride = padded + 8u, v_stride = DV + 8u;
@@ -231,7 +282,13 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, r = lane >> 2, c = lane & 3u;
   const uint32_t past = past_lengths[sequence];
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
-  const uint32_t key_end = past + min(q0 + kQueryTile, p.tokens), tiles = (key_end + kKeyTile - 1u) / kKeyTile;
+  const uint32_t key_end = past + min(q0 + kQueryTile, p.tokens);
+  // whole key tiles: those with kept keys, then from the first row's window on
+  const Visible visible(p, past + q0, key_end - 1u);
+  const uint32_t kept_tiles = (visible.kept + kKeyTile - 1u) / kKeyTile;
+  const uint32_t skipped = max(visible.begin / kKeyTile, kept_tiles) - kept_tiles;
+  const uint32_t tiles = (key_end + kKeyTile - 1u) / kKeyTile - skipped;
+  auto first_key = [&](uint32_t tile) { return (tile < kept_tiles ? tile : tile + skipped) * kKeyTile; };
   const uint32_t k_chunks = padded / 8u, v_chunks = DV / 8u;
 
   auto fetch_tile = [&](uint32_t tile) {
@@ -239,7 +296,7 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
       bf16* k_tile = k_tiles + (tile & 1u) * kKeyTile * k_stride;
       bf16* v_tile = v_tiles + (tile & 1u) * kKeyTile * v_stride;
       // two threads per key row: one slot look-up, half of the chunks each
-      const uint32_t key = threadIdx.x >> 1, half = threadIdx.x & 1u, position = tile * kKeyTile + key;
+      const uint32_t key = threadIdx.x >> 1, half = threadIdx.x & 1u, position = first_key(tile) + key;
       const bool present = position < key_end;
       const bf16* cached = pool + (size_t)(present ? rows(position, error_word) : 0u) * p.token_stride;
       const bf16* k = cached + p.key_offset + kv_head * p.dim;
@@ -260,7 +317,8 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
     const uint32_t row = index / k_chunks, chunk = index % k_chunks;
     uint4 data = make_uint4(0u, 0u, 0u, 0u);
     if (q0 + row < p.tokens && chunk * 8u < p.dim)
-      data = *reinterpret_cast<const uint4*>(query + (((size_t)sequence * p.tokens + q0 + row) * p.heads + head) * p.dim + chunk * 8u);
+      data = *reinterpret_cast<const uint4*>(query + ((size_t)sequence * p.tokens + q0 + row) * p.query_stride +
+                                             p.query_column + head * p.dim + chunk * 8u);
     *reinterpret_cast<uint4*>(q_tile + row * k_stride + chunk * 8u) = data;
   }
   __syncthreads();
@@ -272,24 +330,26 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
       ldmatrix_x4(q_frag[s], q_rows + ((lane & 7u) + ((lane >> 3) & 1u) * 8u) * k_stride + 16 * s + (lane >> 4) * 8u);
   }
   const uint32_t row_low = q0 + warp * 16u + r;  // and row_low + 8
-  const float score_scale = p.scale * kLog2e;
-  Softmax<kKeyTile, DV> state;
+  const ScoreScale score_of(p);
+  Softmax<kKeyTile, DV, FINE> state;
   state.reset();
 
   for (uint32_t tile = 0; tile < tiles; ++tile) {
-    const uint32_t k0 = tile * kKeyTile;
+    const uint32_t k0 = first_key(tile);
     fetch_tile(tile + 1u);  // into the other buffer, which the previous iteration's last barrier released
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
     float score[kKeyTile / 8][4];
     scores<kKeyTile, DK>(score, q_frag, q_rows, k_tiles + (tile & 1u) * kKeyTile * k_stride, k_stride, padded / 16u, lane);
-    const bool all_visible = k0 + kKeyTile - 1u <= past + q0 + warp * 16u;
+    const uint32_t first_row = past + q0 + warp * 16u;  // of this warp
+    const bool all_visible = k0 + kKeyTile - 1u <= first_row &&
+                             (!p.window || first_row + 15u - k0 < p.window || k0 + kKeyTile <= p.keep_first);
 #pragma unroll
     for (int j = 0; j < (int)kKeyTile / 8; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const uint32_t token = row_low + ((i & 2) ? 8u : 0u), key = k0 + 8u * j + 2u * c + (i & 1);
-        score[j][i] = all_visible || key <= past + token ? score[j][i] * score_scale : -INFINITY;
+        score[j][i] = all_visible || sees(p, past + token, key) ? score_of(score[j][i]) : -INFINITY;
       }
     state.absorb(score, v_tiles + (tile & 1u) * kKeyTile * v_stride, v_stride, lane);
     __syncthreads();  // every warp is done with this buffer before the next iteration's fetch refills it
@@ -309,13 +369,15 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
     scale /= total;
     const uint32_t token = row_low + h * 8u;
     if (token >= p.tokens) continue;
-    bf16* target = out + (((size_t)sequence * p.tokens + token) * p.heads + head) * p.vdim;
+    const size_t row = (size_t)sequence * p.tokens + token;
+    bf16* target = out + (row * p.heads + head) * p.vdim;
 #pragma unroll
     for (int t = 0; t < DV / 8; ++t) {
       const uint32_t column = 8u * t + 2u * c;
       if (column < p.vdim)  // vdim is a multiple of eight
         *reinterpret_cast<__nv_bfloat162*>(target + column) =
-            __floats2bfloat162_rn(state.out[t][2 * h] * scale, state.out[t][2 * h + 1] * scale);
+            __floats2bfloat162_rn(state.out[t][2 * h] * scale * gate_of(p, gate, row, head, column),
+                                  state.out[t][2 * h + 1] * scale * gate_of(p, gate, row, head, column + 1u));
     }
   }
 }
@@ -327,10 +389,10 @@ constexpr uint32_t kWarpKeys = 16, kDecodeWarps = 4, kDecodeStages = 3, kMostSpl
 template <int DV>
 __host__ __device__ constexpr uint32_t record_floats() { return 32u + 16u * DV; }
 
-template <int DK, int DV>
+template <int DK, int DV, bool FINE>
 __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
                                                                const uint32_t* past_lengths, const uint32_t* sequence_rows,
-                                                               bf16* out, uint32_t* counters, float* records,
+                                                               bf16* out, const bf16* gate, uint32_t* counters, float* records,
                                                                RowAttentionParams p, uint32_t* error_word) {
   grid_chain_prologue();
   extern __shared__ __align__(16) unsigned char attention_shared[];
@@ -341,7 +403,9 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
   bf16* ring = q_tile + 16u * k_stride + warp * kDecodeStages * stage_elements;
   const uint32_t split = blockIdx.x, kv_head = blockIdx.y, sequence = blockIdx.z;
   const uint32_t group = p.heads / p.kv_heads, query_rows = p.tokens * group;
-  const uint32_t past = past_lengths[sequence], keys = past + p.tokens;
+  const uint32_t past = past_lengths[sequence];
+  const Visible visible(p, past, past + p.tokens - 1u);
+  const uint32_t keys = visible.count();
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
   // whole 64-key stretches per split
   const uint32_t stretch = (kWarpKeys * kDecodeWarps);
@@ -354,9 +418,9 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
     if (tile < tiles) {
       bf16* k_tile = ring + (tile % kDecodeStages) * stage_elements;
       bf16* v_tile = k_tile + kWarpKeys * k_stride;
-      const uint32_t key = lane >> 1, half = lane & 1u, position = begin + tile * stretch + warp * kWarpKeys + key;
-      const bool present = position < end;
-      const bf16* cached = pool + (size_t)(present ? rows(position, error_word) : 0u) * p.token_stride;
+      const uint32_t key = lane >> 1, half = lane & 1u, index = begin + tile * stretch + warp * kWarpKeys + key;
+      const bool present = index < end;
+      const bf16* cached = pool + (size_t)(present ? rows(visible.position(index), error_word) : 0u) * p.token_stride;
       const bf16* k = cached + p.key_offset + kv_head * p.dim;
       const bf16* v = cached + p.value_offset + kv_head * p.vdim;
       for (uint32_t chunk = half; chunk < k_chunks; chunk += 2u) {
@@ -376,8 +440,8 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
     const uint32_t row = index / k_chunks, chunk = index % k_chunks;
     uint4 data = make_uint4(0u, 0u, 0u, 0u);
     if (row < query_rows && chunk * 8u < p.dim)
-      data = *reinterpret_cast<const uint4*>(
-          query + (((size_t)sequence * p.tokens + row / group) * p.heads + kv_head * group + row % group) * p.dim + chunk * 8u);
+      data = *reinterpret_cast<const uint4*>(query + ((size_t)sequence * p.tokens + row / group) * p.query_stride + p.query_column +
+                                             (kv_head * group + row % group) * p.dim + chunk * 8u);
     *reinterpret_cast<uint4*>(q_tile + row * k_stride + chunk * 8u) = data;
   }
   __syncthreads();
@@ -388,8 +452,8 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
       ldmatrix_x4(q_frag[s], q_tile + ((lane & 7u) + ((lane >> 3) & 1u) * 8u) * k_stride + 16 * s + (lane >> 4) * 8u);
   }
   const uint32_t token_low = r / group, token_high = (r + 8u) / group;
-  const float score_scale = p.scale * kLog2e;
-  Softmax<kWarpKeys, DV> state;
+  const ScoreScale score_of(p);
+  Softmax<kWarpKeys, DV, FINE> state;
   state.reset();
   for (uint32_t tile = 0; tile < tiles; ++tile) {
     fetch_tile(tile + kDecodeStages - 1u);
@@ -403,9 +467,9 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
     for (int j = 0; j < (int)kWarpKeys / 8; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const uint32_t key = k0 + 8u * j + 2u * c + (i & 1);
-        const bool visible = key < end && key <= past + ((i & 2) ? token_high : token_low);
-        score[j][i] = visible ? score[j][i] * score_scale : -INFINITY;
+        const uint32_t index = k0 + 8u * j + 2u * c + (i & 1);
+        const bool seen = index < end && sees(p, past + ((i & 2) ? token_high : token_low), visible.position(index));
+        score[j][i] = seen ? score_of(score[j][i]) : -INFINITY;
       }
     state.absorb(score, k_tile + kWarpKeys * k_stride, v_stride, lane);
     __syncwarp();
@@ -455,9 +519,11 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
         sum *= keep;
         total = total * keep + exp2f(-both);
       }
+      const size_t token = (size_t)sequence * p.tokens + row / group;
+      const uint32_t head = kv_head * group + row % group;
       if (column < p.vdim)
-        out[(((size_t)sequence * p.tokens + row / group) * p.heads + kv_head * group + row % group) * p.vdim + column] =
-            __float2bfloat16_rn(sum / total);
+        out[(token * p.heads + head) * p.vdim + column] =
+            __float2bfloat16_rn(sum / total * gate_of(p, gate, token, head, column));
     } else {
       record[32 + row * DV + column] = sum;
       if (column == 0) {
@@ -527,10 +593,13 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
       sum.w = fmaf(weight, part.w, sum.w);
     }
     if (column < p.vdim) {  // vdim is a multiple of eight
-      __nv_bfloat162* target = reinterpret_cast<__nv_bfloat162*>(
-          out + (((size_t)sequence * p.tokens + row / group) * p.heads + kv_head * group + row % group) * p.vdim + column);
-      target[0] = __floats2bfloat162_rn(sum.x, sum.y);
-      target[1] = __floats2bfloat162_rn(sum.z, sum.w);
+      const size_t token = (size_t)sequence * p.tokens + row / group;
+      const uint32_t head = kv_head * group + row % group;
+      sum.x *= gate_of(p, gate, token, head, column);
+      sum.y *= gate_of(p, gate, token, head, column + 1u);
+      sum.z *= gate_of(p, gate, token, head, column + 2u);
+      sum.w *= gate_of(p, gate, token, head, column + 3u);
+      store_four(out + (token * p.heads + head) * p.vdim + column, sum);
     }
   }
 }
@@ -543,7 +612,7 @@ int run_rows(const KernelArgs& args, const RowAttentionParams& p) {
   auto run = [&](auto kernel) {
     launch_kernel(args, kernel, dim3((uint32_t)((items + 3) / 4)), dim3(128), 0, (const T*)args.buffers[0],
                   (const T*)args.buffers[1], (const uint32_t*)args.buffers[2], (const uint32_t*)args.buffers[3],
-                  (const uint32_t*)args.buffers[4], (T*)args.buffers[5], p, context_device_error(args.ctx));
+                  (const uint32_t*)args.buffers[4], (T*)args.buffers[5], (const T*)args.buffers[7], p, context_device_error(args.ctx));
   };
   if (widest <= 64u) run(attention_rows_kernel<T, 2>);
   else if (widest <= 128u) run(attention_rows_kernel<T, 4>);
@@ -553,23 +622,24 @@ int run_rows(const KernelArgs& args, const RowAttentionParams& p) {
   return check_launch(args);
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool FINE>
 int run_prompt(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t padded = DK > 0 ? DK : round16(p.dim);
   const uint32_t bytes = ((kQueryTile + 2u * kKeyTile) * (padded + 8u) + 2u * kKeyTile * (DV + 8u)) * 2u;
-  auto kernel = attention_prompt_kernel<DK, DV>;
+  auto kernel = attention_prompt_kernel<DK, DV, FINE>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
   }
   launch_kernel(args, kernel, dim3((p.tokens + kQueryTile - 1u) / kQueryTile, p.heads, p.sequences), dim3(128), bytes,
                 (const bf16*)args.buffers[0], (const bf16*)args.buffers[1], (const uint32_t*)args.buffers[2],
-                (const uint32_t*)args.buffers[3], (const uint32_t*)args.buffers[4], (bf16*)args.buffers[5], p,
+                (const uint32_t*)args.buffers[3], (const uint32_t*)args.buffers[4], (bf16*)args.buffers[5],
+                (const bf16*)args.buffers[7], p,
                 context_device_error(args.ctx));
   return check_launch(args);
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool FINE>
 int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t padded = DK > 0 ? DK : round16(p.dim);
   uint32_t bytes = (16u * (padded + 8u) + kDecodeWarps * kDecodeStages * kWarpKeys * (padded + 8u + DV + 8u)) * 2u;
@@ -579,21 +649,24 @@ int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
   LLMOPT_REQUIRE(p.splits <= kMostSplits, "at most 64 splits");
   LLMOPT_REQUIRE(p.splits == 1u || args.lengths[6] >= counters + heads * p.splits * record_floats<DV>() * 4,
                  "split scratch is too short");
-  auto kernel = attention_decode_kernel<DK, DV>;
+  auto kernel = attention_decode_kernel<DK, DV, FINE>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
   }
   launch_kernel(args, kernel, dim3(p.splits, p.kv_heads, p.sequences), dim3(128), bytes, (const bf16*)args.buffers[0],
                 (const bf16*)args.buffers[1], (const uint32_t*)args.buffers[2], (const uint32_t*)args.buffers[3],
-                (const uint32_t*)args.buffers[4], (bf16*)args.buffers[5], (uint32_t*)args.buffers[6],
+                (const uint32_t*)args.buffers[4], (bf16*)args.buffers[5], (const bf16*)args.buffers[7],
+                (uint32_t*)args.buffers[6],
                 (float*)((uint8_t*)args.buffers[6] + counters), p, context_device_error(args.ctx));
   return check_launch(args);
 }
 
 template <int DK, int DV>
 int run_tensor(const KernelArgs& args, const RowAttentionParams& p) {
-  return p.tokens * (p.heads / p.kv_heads) <= 16u ? run_decode<DK, DV>(args, p) : run_prompt<DK, DV>(args, p);
+  if (p.tokens * (p.heads / p.kv_heads) <= 16u)
+    return p.weights32 ? run_decode<DK, DV, true>(args, p) : run_decode<DK, DV, false>(args, p);
+  return p.weights32 ? run_prompt<DK, DV, true>(args, p) : run_prompt<DK, DV, false>(args, p);
 }
 
 int run_tensor_shapes(const KernelArgs& args, const RowAttentionParams& p) {
@@ -605,11 +678,12 @@ int run_tensor_shapes(const KernelArgs& args, const RowAttentionParams& p) {
   return run_tensor<0, 256>(args, p);
 }
 
-// Buffers [query, pool, slot table, past, sequence rows, out, split scratch (counters zero between launches)].
+// Buffers [query, pool, slot table, past, sequence rows, out, split scratch (counters zero between launches),
+// gates (an absent one repeats the queries)].
 template <typename T>
 int launch_row_attention(const KernelArgs& args) {
   RowAttentionParams p;
-  LLMOPT_REQUIRE(args.buffer_count == 7 && args.param_bytes == sizeof(p), "expects 7 buffers and 60 parameter bytes");
+  LLMOPT_REQUIRE(args.buffer_count == 8 && args.param_bytes == sizeof(p), "expects 8 buffers and 92 parameter bytes");
   memcpy(&p, args.params, sizeof(p));
   const size_t rows = (size_t)p.sequences * p.tokens, e = sizeof(T);
   LLMOPT_REQUIRE(p.heads > 0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.dim > 0 && p.vdim > 0 && p.splits > 0,
@@ -617,14 +691,18 @@ int launch_row_attention(const KernelArgs& args) {
   LLMOPT_REQUIRE(p.key_offset + p.kv_heads * p.dim <= p.token_stride && p.value_offset + p.kv_heads * p.vdim <= p.token_stride,
                  "key or value segment lies outside the cache row");
   LLMOPT_REQUIRE(p.sequences <= 65535u && p.heads <= 65535u, "too many sequences or heads");
-  LLMOPT_REQUIRE(args.lengths[0] >= rows * p.heads * p.dim * e && args.lengths[5] >= rows * p.heads * p.vdim * e &&
+  LLMOPT_REQUIRE((size_t)p.query_column + p.heads * p.dim <= p.query_stride &&
+                     (!p.gate_stride || (size_t)p.gate_column + p.heads * p.vdim <= p.gate_stride),
+                 "query or gate columns lie outside the row");
+  LLMOPT_REQUIRE(args.lengths[7] >= rows * p.gate_stride * e, "gate buffer is too short");
+  LLMOPT_REQUIRE(args.lengths[0] >= rows * p.query_stride * e && args.lengths[5] >= rows * p.heads * p.vdim * e &&
                      args.lengths[1] >= (size_t)p.pool_rows * p.token_stride * e && p.pool_rows > 0 &&
                      args.lengths[2] >= (size_t)p.table_rows * p.table_stride * 4 &&
                      args.lengths[3] >= (size_t)p.sequences * 4 && args.lengths[4] >= (size_t)p.sequences * 4,
                  "buffer is too short");
   if (rows == 0) return 0;
   const bool vectors = e == 2 && p.dim % 8u == 0 && p.vdim % 8u == 0 && p.dim <= 256u && p.vdim <= 256u &&
-                       p.token_stride % 8u == 0 && p.key_offset % 8u == 0 && p.value_offset % 8u == 0 &&
+                       p.query_stride % 8u == 0 && p.query_column % 8u == 0 && p.token_stride % 8u == 0 && p.key_offset % 8u == 0 && p.value_offset % 8u == 0 &&
                        ((uintptr_t)args.buffers[0] & 15u) == 0 && ((uintptr_t)args.buffers[1] & 15u) == 0;
   if (vectors) {
     const int status = run_tensor_shapes(args, p);

@@ -82,6 +82,7 @@ LLMOPT_FAMILY const NamedLauncher* dense_linear_launchers(size_t* count);
 LLMOPT_FAMILY const NamedLauncher* sequence_glue_launchers(size_t* count);
 LLMOPT_FAMILY const NamedLauncher* row_attention_launchers(size_t* count);
 LLMOPT_FAMILY const NamedLauncher* matrix_state_launchers(size_t* count);
+LLMOPT_FAMILY const NamedLauncher* expert_launchers(size_t* count);
 struct ExprProgram {
   uint8_t code[192];
   uint32_t length;
@@ -384,7 +385,7 @@ static void register_kernels(llmopt_cuda_library* library) {
   // the sequence-mixer kernels
   const NamedLauncher* (*const families[])(size_t*) = {norm_family_launchers, dense_linear_launchers,
                                                        sequence_glue_launchers, row_attention_launchers,
-                                                       matrix_state_launchers};
+                                                       matrix_state_launchers, expert_launchers};
   for (auto family : families) {
     size_t count = 0;
     const NamedLauncher* table = family != nullptr ? family(&count) : nullptr;

@@ -1,6 +1,8 @@
 // Row-wise kernels of decoders whose residual stream is kept in fp32 and whose sublayers read it
 // directly (T: bfloat16 or float, the element of activations and weights):
 //   llmopt_embedding_residual_{bf16,f32}   x = table[token], with a T copy for the next product
+//   llmopt_embedding_sinusoid_{bf16,f32}   x = table[token] + sinusoidal position, with its tanh norm for the next product
+//   llmopt_gather_rows_{bf16,f32}          chosen rows in a new order
 //   llmopt_residual_norm_{bf16,f32}        x += norm(y), or of the mean of two normed branches
 //   llmopt_gather_norm_{bf16,f32}          norm of chosen rows (input of the output projection)
 //   llmopt_row_attention_prepare_{bf16,f32} head norm + rotary of q and k, k and v into the cache
@@ -53,6 +55,88 @@ int launch_embedding_residual(const KernelArgs& args) {
   if (rows == 0) return 0;
   launch_kernel(args, embedding_residual_kernel<T>, dim3(rows), dim3(256), 0, (const long long*)args.buffers[0],
                 (const T*)args.buffers[1], (float*)args.buffers[2], (T*)args.buffers[3], rows, vocabulary, width);
+  return check_launch(args);
+}
+
+// ---- embedding with absolute positions -----------------------------------------------------------
+// Columns 2i, 2i + 1 take sine and cosine of position * frequency[i].  The angle is formed and reduced to one turn in
+// double precision, so that late positions lose nothing.
+template <typename T>
+__global__ void __launch_bounds__(256) embedding_sinusoid_kernel(const long long* ids, const T* __restrict__ table,
+                                                                 const uint32_t* past, const double* __restrict__ frequency,
+                                                                 const float* __restrict__ norm, float* x, T* normed,
+                                                                 uint32_t tokens, uint32_t vocabulary, uint32_t width) {
+  grid_chain_prologue();
+  const uint32_t row = blockIdx.y;
+  const size_t token = min((unsigned long long)ids[row], (unsigned long long)(vocabulary - 1u));
+  const double position = (double)(past[row / tokens] + row % tokens);
+  const TanhNorm next(norm, width);
+  constexpr double kTurn = 6.283185307179586476925;
+  const uint32_t pair = blockIdx.x * 256u + threadIdx.x, column = pair * 2u;
+  if (column >= width) return;
+  const double angle = position * frequency[pair];
+  float sine, cosine;
+  sincosf((float)(angle - kTurn * rint(angle / kTurn)), &sine, &cosine);
+  const size_t at = (size_t)row * width + column;
+  const float first = as_float(table[token * width + column]) + sine;
+  x[at] = first;
+  normed[at] = from_float<T>(next(first, column));
+  if (column + 1u < width) {
+    const float second = as_float(table[token * width + column + 1u]) + cosine;
+    x[at + 1] = second;
+    normed[at + 1] = from_float<T>(next(second, column + 1u));
+  }
+}
+
+// Buffers [ids, table, past, frequencies f64, following norm, x, normed]; params {rows, tokens per sequence, vocabulary, width}.
+template <typename T>
+int launch_embedding_sinusoid(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 7 && args.param_bytes == 16, "expects 7 buffers and 16 parameter bytes");
+  const uint32_t rows = param_u32(args, 0), tokens = param_u32(args, 1), vocabulary = param_u32(args, 2), width = param_u32(args, 3);
+  LLMOPT_REQUIRE(vocabulary > 0 && width > 0 && tokens > 0 && rows % tokens == 0 && rows <= 65535u,
+                 "needs a vocabulary, a width and whole sequences of at most 65535 rows");
+  const uint32_t pairs = (width + 1u) / 2u;
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)rows * 8 && args.lengths[1] >= (size_t)vocabulary * width * sizeof(T) &&
+                     args.lengths[2] >= (size_t)(rows / tokens) * 4 && args.lengths[3] >= (size_t)pairs * 8 &&
+                     args.lengths[4] >= (2 * (size_t)width + 1) * 4 && args.lengths[5] >= (size_t)rows * width * 4 &&
+                     args.lengths[6] >= (size_t)rows * width * sizeof(T),
+                 "buffer is too short");
+  if (rows == 0) return 0;
+  launch_kernel(args, embedding_sinusoid_kernel<T>, dim3((pairs + 255u) / 256u, rows), dim3(256), 0,
+                (const long long*)args.buffers[0], (const T*)args.buffers[1], (const uint32_t*)args.buffers[2],
+                (const double*)args.buffers[3], (const float*)args.buffers[4], (float*)args.buffers[5], (T*)args.buffers[6],
+                tokens, vocabulary, width);
+  return check_launch(args);
+}
+
+// ---- rows in a new order -------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) gather_rows_kernel(const T* x, const uint32_t* rows, T* out, uint32_t source_rows,
+                                                          uint32_t width, uint32_t vectors) {
+  grid_chain_prologue();
+  const T* source = x + (size_t)min(rows[blockIdx.x], source_rows - 1u) * width;
+  T* target = out + (size_t)blockIdx.x * width;
+  if (vectors) {
+    for (uint32_t c = threadIdx.x; c < vectors; c += blockDim.x)
+      reinterpret_cast<uint4*>(target)[c] = reinterpret_cast<const uint4*>(source)[c];
+  } else {
+    for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) target[c] = source[c];
+  }
+}
+
+// Buffers [x, rows u32, out]; params {count, source rows, width}.
+template <typename T>
+int launch_gather_rows(const KernelArgs& args) {
+  LLMOPT_REQUIRE(args.buffer_count == 3 && args.param_bytes == 12, "expects 3 buffers and 12 parameter bytes");
+  const uint32_t count = param_u32(args, 0), source_rows = param_u32(args, 1), width = param_u32(args, 2);
+  LLMOPT_REQUIRE(source_rows > 0 && width > 0, "needs source rows and a width");
+  LLMOPT_REQUIRE(args.lengths[0] >= (size_t)source_rows * width * sizeof(T) && args.lengths[1] >= (size_t)count * 4 &&
+                     args.lengths[2] >= (size_t)count * width * sizeof(T),
+                 "buffer is too short");
+  if (count == 0) return 0;
+  const bool aligned = width * sizeof(T) % 16u == 0 && ((uintptr_t)args.buffers[0] & 15u) == 0 && ((uintptr_t)args.buffers[2] & 15u) == 0;
+  launch_kernel(args, gather_rows_kernel<T>, dim3(count), dim3(256), 0, (const T*)args.buffers[0], (const uint32_t*)args.buffers[1],
+                (T*)args.buffers[2], source_rows, width, aligned ? (uint32_t)(width * sizeof(T) / 16u) : 0u);
   return check_launch(args);
 }
 
@@ -260,6 +344,7 @@ struct AttentionPrepareParams {
   uint32_t table_stride, table_rows, pool_rows;
   uint32_t head_norm;
   float epsilon;
+  uint32_t own_keys;  // 0: only the queries (the layer reads another layer's keys and values)
   uint32_t pairs;  // set by the launcher: every head starts at an even element
 };
 
@@ -282,7 +367,7 @@ __global__ void __launch_bounds__(256) attention_prepare_kernel(const T* project
   T* const cached = pool + (size_t)(slot < p.pool_rows ? slot : 0u) * p.token_stride;
   const uint32_t trig_row = min(position, p.trig_rows - 1u);
   const float2* turns = trig + (size_t)trig_row * (p.rotary_dims / 2u);
-  const uint32_t per_row = p.heads + 2u * p.kv_heads;
+  const uint32_t per_row = p.heads + (p.own_keys ? 2u * p.kv_heads : 0u);
   for (uint32_t head = blockIdx.y * 8u + (threadIdx.x >> 5); head < per_row; head += 8u * gridDim.y) {
     const T* source = projected + (size_t)row * p.stride;
     if (head < p.heads) source += p.q_column + head * p.dim;
@@ -376,8 +461,8 @@ namespace {
 template <typename T>
 int launch_attention_prepare(const KernelArgs& args) {
   AttentionPrepareParams p;
-  LLMOPT_REQUIRE(args.buffer_count == 9 && args.param_bytes == 80, "expects 9 buffers and 80 parameter bytes");
-  memcpy(&p, args.params, 80);
+  LLMOPT_REQUIRE(args.buffer_count == 9 && args.param_bytes == 84, "expects 9 buffers and 84 parameter bytes");
+  memcpy(&p, args.params, 84);
   p.pairs = p.dim % 2u == 0 && p.dim <= 256u && p.stride % 2u == 0 && p.q_column % 2u == 0 && p.k_column % 2u == 0 &&
             p.token_stride % 2u == 0 && p.key_offset % 2u == 0;
   for (int i : {0, 1, 2, 4, 5})
@@ -386,8 +471,8 @@ int launch_attention_prepare(const KernelArgs& args) {
   LLMOPT_REQUIRE(p.heads > 0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.dim > 0 && p.vdim > 0,
                  "needs whole groups of query heads");
   LLMOPT_REQUIRE(p.rotary_dims <= p.dim && p.rotary_dims % 2u == 0, "rotated dimensions come in pairs inside the head");
-  LLMOPT_REQUIRE(p.q_column + p.heads * p.dim <= p.stride && p.k_column + p.kv_heads * p.dim <= p.stride &&
-                     p.v_column + p.kv_heads * p.vdim <= p.stride,
+  LLMOPT_REQUIRE(p.q_column + p.heads * p.dim <= p.stride &&
+                     (!p.own_keys || (p.k_column + p.kv_heads * p.dim <= p.stride && p.v_column + p.kv_heads * p.vdim <= p.stride)),
                  "projection columns lie outside the row");
   LLMOPT_REQUIRE(p.key_offset + p.kv_heads * p.dim <= p.token_stride && p.value_offset + p.kv_heads * p.vdim <= p.token_stride,
                  "key or value segment lies outside the cache row");
@@ -494,13 +579,6 @@ int launch_head_norm_gate(const KernelArgs& args) {
 }
 
 // ---- greedy pick and bookkeeping ----------------------------------------------------------------
-// Larger logits first, then smaller columns, as one unsigned integer.
-__device__ __forceinline__ unsigned long long ranked(float value, uint32_t column) {
-  uint32_t bits = __float_as_uint(value);
-  bits = (bits & 0x80000000u) ? ~bits : bits | 0x80000000u;
-  return ((unsigned long long)bits << 32) | (0xffffffffu - column);
-}
-
 __global__ void __launch_bounds__(256) argmax_kernel(const float* logits, unsigned long long* best, uint32_t columns,
                                                      uint32_t parts) {
   grid_chain_prologue();
@@ -563,6 +641,10 @@ const NamedLauncher* sequence_glue_launchers(size_t* count) {
   static const NamedLauncher table[] = {
       {"llmopt_embedding_residual_bf16", launch_embedding_residual<bf16>},
       {"llmopt_embedding_residual_f32", launch_embedding_residual<float>},
+      {"llmopt_embedding_sinusoid_bf16", launch_embedding_sinusoid<bf16>},
+      {"llmopt_embedding_sinusoid_f32", launch_embedding_sinusoid<float>},
+      {"llmopt_gather_rows_bf16", launch_gather_rows<bf16>},
+      {"llmopt_gather_rows_f32", launch_gather_rows<float>},
       {"llmopt_residual_norm_bf16", launch_residual_norm<bf16>},
       {"llmopt_residual_norm_f32", launch_residual_norm<float>},
       {"llmopt_gather_norm_bf16", launch_gather_norm<bf16>},

@@ -158,7 +158,13 @@ def _entries() -> list[Entry]:
     # sequence-mixer kernels in the model's element type (no reference counterpart)
     for suffix, element in (("bf16", "bfloat16"), ("f32", f32)):
         add("llmopt_dense_linear_" + suffix, LINEAR, element, element)
+        add("llmopt_dense_cached_" + suffix, LINEAR, element, element)
+        add("llmopt_dense_residual_" + suffix, LINEAR, element, element)
+        add("llmopt_expert_rows_" + suffix, LINEAR, element, element)
+        add("llmopt_expert_combine_" + suffix, RMS_NORM, f32, element)
         add("llmopt_embedding_residual_" + suffix, EMBEDDING, element, f32)
+        add("llmopt_embedding_sinusoid_" + suffix, EMBEDDING, element, f32)
+        add("llmopt_gather_rows_" + suffix, EMBEDDING, element, element)
         add("llmopt_residual_norm_" + suffix, RMS_NORM, f32, element)
         add("llmopt_gather_norm_" + suffix, RMS_NORM, f32, element)
         add("llmopt_row_attention_prepare_" + suffix, CACHE, element, element)
@@ -169,6 +175,11 @@ def _entries() -> list[Entry]:
         add("llmopt_memory_scan_" + suffix, GATED_DELTA, element, f32)
         add("llmopt_memory_step_" + suffix, GATED_DELTA, element, element)
         add("llmopt_delta_step_" + suffix, GATED_DELTA, element, element)
+    add("llmopt_expert_step_bf16", LINEAR, "bfloat16", "bfloat16")
+    add("llmopt_expert_step_residual_bf16", LINEAR, "bfloat16", "bfloat16")
+    add("llmopt_route_step_f32", POINTWISE, f32, "uint32")
+    add("llmopt_route_rows_f32", POINTWISE, f32, "uint32")
+    add("llmopt_route_plan", POINTWISE, "uint32", "uint32")
     add("llmopt_delta_scan_f32", GATED_DELTA, f32, f32)
     add("llmopt_argmax_f32", POINTWISE, f32, i64)
     add("llmopt_advance_tokens", EMBEDDING, i64, "int32")

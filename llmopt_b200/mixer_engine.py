@@ -17,10 +17,12 @@ import numpy as np
 
 from . import parameters
 from .cuda_native import Batch, Buffer, DispatchItem, Prebaked, Runtime, pack_records, sample_f32
-from .kv_cache import RowLayout, SequenceTable
+from .feed_forward import FEED_FORWARDS
+from .kv_cache import RowLayout, RowRegion, SequenceTable
 from .mixers import LayerMixer, Step, attention_specs
 from .model import AttentionSpec, MixerConfig
 from .quantize import rotary_pairs
+from .residual import RESIDUALS
 from .safetensors_archive import as_bfloat16_bits, as_float32
 
 ARGMAX_PARTS = 32
@@ -44,12 +46,10 @@ class _Layer:
     def __init__(self, engine: "MixerEngine", index: int, weights):
         layer, prefix = engine.config.layers[index], f"l{index}"
         self.index = index
-        self.mixer = LayerMixer(engine, layer.mixer, weights, f"{prefix}.mix")
-        self.norm1 = engine.upload_vector(weights[f"{prefix}.norm1"])
-        self.feed_forward = layer.feed_forward
+        self.mixer = LayerMixer(engine, layer.mixer, weights, f"{prefix}.mix", index)
+        self.feed_forward = None
         if layer.feed_forward:
-            self.up, self.down = (engine.upload_matrix(weights[f"{prefix}.mlp.{name}"]) for name in ("up", "down"))
-            self.norm2 = engine.upload_vector(weights[f"{prefix}.norm2"])
+            self.feed_forward = FEED_FORWARDS[type(layer.feed_forward)](engine, layer.feed_forward, weights, f"{prefix}.mlp")
         if engine.config.token_side:
             self.side_gate, self.side_proj = (engine.upload_matrix(weights[f"{prefix}.side.{name}"]) for name in ("gate", "proj"))
             self.side_norm = engine.upload_vector(weights[f"{prefix}.side.norm"])
@@ -98,18 +98,22 @@ class MixerEngine:
         pages = lambda tokens: (tokens + page - 1) // page * page
         self.token_capacity = pages(token_capacity) if token_capacity else rows * pages(capacity)
         self.sequences = SequenceTable(rows, capacity, self.token_capacity, page)
-        self.layout = RowLayout([(spec.kv_heads, spec.dim, spec.vdim) for spec in attention_specs(config)])
-        self._regions = iter(self.layout.regions)
+        owners = attention_specs(config)
+        self.layout = RowLayout([(spec.kv_heads, spec.dim, spec.vdim) for _, spec in owners])
+        self._regions: Dict[int, List[RowRegion]] = {}  # of every layer with keys and values of its own
+        for (layer, _), region in zip(owners, self.layout.regions):
+            self._regions.setdefault(layer, []).append(region)
+        self._claimed: Dict[int, int] = {}
         self.token_pool = self.empty_bytes(self.token_capacity * self.layout.token_elements * self.itemsize)
         self.slot_table = self.empty_bytes(rows * capacity * 4)
         self._work: Dict[tuple, Buffer] = {}
         self._trig: Dict[object, Buffer] = {}
         self._prompt_plans: "OrderedDict[int, tuple]" = OrderedDict()
         self._decode_plans: Dict[int, tuple] = {}
-        self.embedding = self.upload_matrix(weights["embed"])
+        self.residual = RESIDUALS[config.norm](self, weights)
         self.token_side = self.upload_matrix(weights["side.embed"]) if config.token_side else None
         self.layers = [_Layer(self, index, weights) for index in range(len(config.layers))]
-        self.final_norm, self.head = self.upload_vector(weights["final.norm"]), self.upload_matrix(weights["head"])
+        self.head = self.residual.embedding if config.tied_head else self.upload_matrix(weights["head"])
         self._lockstep = None  # rows of the sequences ``step`` decodes, once opened
 
     # ---- device memory --------------------------------------------------------------------------
@@ -132,93 +136,86 @@ class MixerEngine:
         return self._workspace(name, columns, 4)
 
     def _workspace(self, name: str, columns: int, itemsize: int) -> Buffer:
-        key = (name, columns, itemsize)
-        if key not in self._work:
-            self._work[key] = self.empty_bytes(max(self.max_rows * columns * itemsize, 16))
-        return self._work[key]
+        return self._workspace_bytes((name, columns, itemsize), self.max_rows * columns * itemsize)
 
     def rotary_table(self, rotary) -> Buffer:
         if rotary not in self._trig:
             self._trig[rotary] = Buffer.of_array(self.runtime, rotary_pairs(self.capacity, rotary))
         return self._trig[rotary]
 
-    def next_attention_region(self):
-        return next(self._regions)
+    def scratch(self, name: str, nbytes: int) -> Buffer:
+        """Workspace of another shape; users of the same name and size share it."""
+        return self._workspace_bytes((name, nbytes), nbytes)
+
+    def _workspace_bytes(self, key: tuple, nbytes: int) -> Buffer:
+        if key not in self._work:
+            self._work[key] = self.empty_bytes(max(nbytes, 16))
+        return self._work[key]
+
+    def attention_region(self, layer: int, spec: AttentionSpec) -> RowRegion:
+        """Where a cache row holds the keys and values that an attention mixer of the layer reads."""
+        if spec.kv_from is not None:
+            return self._regions[spec.kv_from][0]
+        place = self._claimed.get(layer, 0)
+        self._claimed[layer] = place + 1
+        return self._regions[layer][place]
+
+    def cache_rows(self, region: RowRegion) -> dict:
+        """Parameters of the kernels that reach into the cache."""
+        return dict(token_stride=self.layout.token_elements, key_offset=region.key_offset, value_offset=region.value_offset,
+                    table_stride=self.sequences.stride, table_rows=self.sequences.rows, pool_rows=self.token_capacity)
 
     def attention_splits(self, step: Step, spec: AttentionSpec) -> Tuple[int, Buffer]:
         """How many thread blocks share the keys of a (sequence, key/value head) when few rows ask, and
         the scratch their partial results meet in."""
         heads = step.sequences * spec.kv_heads
-        splits = max(1, min(64, 444 // heads, (self.capacity + 63) // 64))
+        visible = self.capacity
+        if spec.window:
+            visible = min(visible, spec.window.keep_first + spec.window.size + step.tokens - 1)
+        splits = max(1, min(64, 444 // heads, (visible + 63) // 64))
         if step.tokens * (spec.heads // spec.kv_heads) > 16:
             splits = 1
         width = next((v for v in (32, 64, 128) if spec.vdim <= v), 256)
-        nbytes = (heads * 4 + 255) // 256 * 256 + heads * splits * (32 + 16 * width) * 4
-        key = ("attention_scratch", nbytes)
-        if key not in self._work:
-            self._work[key] = self.empty_bytes(nbytes)  # zero-filled: the arrival counters start at zero
-        return splits, self._work[key]
+        counters = (heads * 4 + 255) // 256 * 256
+        nbytes = counters + heads * splits * (32 + 16 * width) * 4
+        return splits, self.scratch(f"attention_scratch_{counters}", nbytes)  # zero-filled: the arrival counters start at zero
 
     # ---- recording --------------------------------------------------------------------------------
     def record_linear(self, step: Step, x: Buffer, weight: Buffer, out: Optional[Buffer], *, m: int, n: int, k: int,
                       split: int, out32: Optional[Buffer] = None, bias: Optional[Buffer] = None, epilogue=None,
-                      table: Optional[Buffer] = None, table_stride: int = 0, table_offset: int = 0) -> None:
+                      table: Optional[Buffer] = None, table_stride: int = 0, table_offset: int = 0, scale: float = 1.0) -> None:
         absent = weight
         step.run(step.element("dense_linear"),
                  [x, weight, bias or absent, out or absent, out32 or absent, step.ids, table or absent],
                  parameters.dense_linear(m=m, n=n, k=k, split=split, has_bias=bias is not None, epilogue=epilogue,
                                          table_rows=self.config.vocabulary if table else 0, table_stride=table_stride,
-                                         table_offset=table_offset))
+                                         table_offset=table_offset, scale=scale))
 
-    def _record_layers(self, step: Step) -> Buffer:
-        """The residual after the last layer."""
+    def _record_layers(self, step: Step) -> None:
+        """The stream of the step ends with the output of the last layer."""
         config, width = self.config, self.config.width
-        residuals = [self.work32("residual_a", width), self.work32("residual_b", width)]
-        copies = residuals if self.itemsize == 4 else [self.work("copy_a", width), self.work("copy_b", width)]
-        current = 0
-        step.run(step.element("embedding_residual"), [step.ids, self.embedding, residuals[0], copies[0]],
-                 parameters.embedding(tokens=step.rows, vocabulary=config.vocabulary, width=width))
-
-        def add_normed(outputs, weight, offset, branch_norms=None):
-            nonlocal current
-            pair = len(outputs) == 2
-            left, right = branch_norms if pair else (weight, weight)
-            step.run(step.element("residual_norm"),
-                     [residuals[current], outputs[0], weight, outputs[-1], left, right, residuals[1 - current],
-                      copies[1 - current]],
-                     parameters.residual_norm(rows=step.rows, width=width, epsilon=config.epsilon, weight_offset=offset,
-                                              pair=pair))
-            current = 1 - current
-
-        y = self.work32("sublayer_0", width)
+        step.stream = stream = self.residual.open(step)
         for layer in self.layers:
-            outputs = layer.mixer.record(step, copies[current])
-            add_normed(outputs, layer.norm1, config.norm_offset, layer.mixer.branch_norms)
+            layer.mixer.record(step)
+            stream.close(branch_norms=layer.mixer.branch_norms)
             if layer.feed_forward:
-                inner = layer.feed_forward.width
-                hidden = self.work("feed_forward", inner)
-                self.record_linear(step, copies[current], layer.up, hidden, m=step.rows, n=inner, k=width, split=inner,
-                                   epilogue=layer.feed_forward.activation)
-                self.record_linear(step, hidden, layer.down, None, m=step.rows, n=width, k=inner, split=0, out32=y)
-                add_normed([y], layer.norm2, config.norm_offset)
+                layer.feed_forward.record(step)
+                stream.close()
             if config.token_side:
                 dim = config.token_side.dim
                 gated = self.work("token_side", dim)
-                self.record_linear(step, copies[current], layer.side_gate, gated, m=step.rows, n=dim, k=width, split=dim,
+                self.record_linear(step, stream.x, layer.side_gate, gated, m=step.rows, n=dim, k=width, split=dim,
                                    epilogue="token_gate", table=self.token_side, table_stride=dim * len(self.layers),
                                    table_offset=layer.index * dim)
-                self.record_linear(step, gated, layer.side_proj, None, m=step.rows, n=width, k=dim, split=0, out32=y)
-                add_normed([y], layer.side_norm, 0.0)
-        return residuals[current]
+                stream.product(gated, layer.side_proj, k=dim)
+                stream.close(norm=layer.side_norm)
 
-    def _record_logits(self, step: Step, residual: Buffer, chosen: Buffer, count: int, logits: Buffer) -> None:
+    def _record_logits(self, step: Step, chosen: Buffer, count: int, logits: Buffer, every: bool = False) -> None:
+        """``every``: the chosen rows are all rows in order."""
         config = self.config
-        normed = self.work("final_normed", config.width)
-        step.run(step.element("gather_norm"), [residual, chosen, self.final_norm, normed],
-                 parameters.gather_norm(count=count, source_rows=step.rows, width=config.width, epsilon=config.epsilon,
-                                        weight_offset=config.norm_offset))
-        self.record_linear(step, normed, self.head, None, m=count, n=config.vocabulary, k=config.width, split=0,
-                           out32=logits)
+        rows = step.stream.chosen_rows(chosen, count, every)
+        self.record_linear(step, rows, self.head, None, m=count, n=config.vocabulary, k=config.width, split=0, out32=logits,
+                           scale=config.logit_scale)
 
     def _decode_plan(self, sequences: int):
         """(plan, graph, logits, picked tokens) of a step of one token for each of ``sequences`` sequences."""
@@ -229,24 +226,23 @@ class MixerEngine:
             chosen = Buffer.of_array(self.runtime, np.arange(sequences, dtype=np.uint32))
             candidates = self.empty_bytes(sequences * ARGMAX_PARTS * 8)
             picked = self.empty_bytes(max(sequences * 4, 16))
-            residual = self._record_layers(plan.step)
-            self._record_logits(plan.step, residual, chosen, sequences, logits)
+            self._record_layers(plan.step)
+            self._record_logits(plan.step, chosen, sequences, logits, every=True)
             plan.step.run("llmopt_argmax_f32", [logits, candidates], parameters.u32s([sequences, vocabulary, ARGMAX_PARTS]))
             plan.step.run("llmopt_advance_tokens", [candidates, picked, plan.ids, plan.past],
                           parameters.u32s([sequences, ARGMAX_PARTS, 1]))
-            plan.residual = residual
             graph = Prebaked(self.runtime, plan.items, plan.ids, picked)
             self._decode_plans[sequences] = (plan, graph, logits, picked)
         return self._decode_plans[sequences]
 
     def _prompt_plan(self, tokens: int):
-        """(plan, packed dispatch list, residual) of ``tokens`` rows of one sequence."""
+        """(plan, packed dispatch list) of ``tokens`` rows of one sequence."""
         if tokens not in self._prompt_plans:
             plan = _Plan(self, 1, tokens)
-            residual = self._record_layers(plan.step)
+            self._record_layers(plan.step)
             while len(self._prompt_plans) >= 32:
                 self._prompt_plans.popitem(last=False)
-            self._prompt_plans[tokens] = (plan, pack_records(plan.items), residual)
+            self._prompt_plans[tokens] = (plan, pack_records(plan.items))
         self._prompt_plans.move_to_end(tokens)
         return self._prompt_plans[tokens]
 
@@ -313,7 +309,7 @@ class MixerEngine:
         return out
 
     def _run_portion(self, sequence: int, tokens: Sequence[int], want: np.ndarray) -> Optional[np.ndarray]:
-        plan, records, residual = self._prompt_plan(len(tokens))
+        plan, records = self._prompt_plan(len(tokens))
         self._reserve(sequence, len(tokens))
         plan.write(tokens, [self.sequences.lengths[sequence]], [sequence])
         commands = Batch(self.runtime)
@@ -323,7 +319,7 @@ class MixerEngine:
             logits = self.empty_bytes(len(want) * self.config.vocabulary * 4)
             chosen = Buffer.of_array(self.runtime, np.ascontiguousarray(want, np.uint32))
             kept, plan.items = plan.items, []
-            self._record_logits(plan.step, residual, chosen, len(want), logits)
+            self._record_logits(plan.step, chosen, len(want), logits)
             for item in plan.items:
                 commands.dispatch_item(item)
             plan.items = kept

@@ -2,8 +2,8 @@
 
 A mixer declares the projections of its input that it reads (the engine computes all of a layer's in one
 product), owns its weights and its per-sequence state on the device, and records the kernels from the
-projected rows to its output, one fp32 row of the model's width per token.  ``ParallelMixer`` runs
-two of them side by side.
+projected rows to the product that ends the sublayer (``residual``).  ``LayerMixer`` runs one, or two of them
+side by side.
 
 The engine (``mixer_engine.MixerEngine``) hands a ``Step`` to the builders: the shape of the step and the
 device buffers every kernel of it reads."""
@@ -32,6 +32,7 @@ class Step:
     past: Buffer           # u32 [sequences]: tokens behind the step
     sequence_rows: Buffer  # u32 [sequences]: row of the slot table and of the state pools
     run: object            # run(name, buffers, parameters) records a dispatch
+    stream: object = None  # residual stream of the step (``residual``), once its layers are recorded
 
     @property
     def rows(self) -> int:
@@ -43,23 +44,28 @@ class Step:
 
 class Projection:
     """All projections of a layer's mixer input as one weight matrix: parts read in the model's element
-    type first, then the parts that feed fp32 arithmetic."""
+    type first, then keys and values that go straight into the cache, then the parts that feed fp32 arithmetic."""
+
+    ORDER = ("element", "cache", "fp32")
 
     def __init__(self):
-        self.parts: List[Tuple[str, np.ndarray, object, bool]] = []
+        self.parts: List[Tuple[str, np.ndarray, object, str]] = []
+        self.region = None  # cache region of the "cache" parts
 
-    def add(self, key: str, weight: np.ndarray, bias=None, fp32: bool = False) -> None:
-        self.parts.append((key, weight, bias, fp32))
+    def add(self, key: str, weight: np.ndarray, bias=None, fp32: bool = False, cache: bool = False) -> None:
+        self.parts.append((key, weight, bias, "cache" if cache else "fp32" if fp32 else "element"))
 
     def upload(self, engine) -> None:
-        ordered = [p for p in self.parts if not p[3]] + [p for p in self.parts if p[3]]
+        ordered = sorted(self.parts, key=lambda part: self.ORDER.index(part[3]))
         self.columns: Dict[str, int] = {}
-        self.split = sum(weight.shape[0] for _, weight, _, fp32 in ordered if not fp32)
+        rows = {kind: [weight.shape[0] for _, weight, _, k in ordered if k == kind] for kind in self.ORDER}
+        self.split, self.scalars, self.cached = sum(rows["element"]), sum(rows["fp32"]), rows["cache"]
+        self.total = self.split + sum(self.cached) + self.scalars
+        start = dict(zip(self.ORDER, (0, self.split, self.split + sum(self.cached))))
         total = 0
-        for key, weight, _, fp32 in ordered:
-            self.columns[key] = total - (self.split if fp32 else 0)
+        for key, weight, _, kind in ordered:
+            self.columns[key] = total - start[kind]
             total += weight.shape[0]
-        self.total, self.scalars = total, total - self.split
         self.weight = engine.upload_matrix(np.concatenate([np.ascontiguousarray(w) for _, w, _, _ in ordered]))
         self.bias = None
         if any(bias is not None for _, _, bias, _ in ordered):
@@ -73,8 +79,17 @@ class Projection:
         """(rows in the element type, fp32 rows)."""
         engine = step.engine
         projected, scalars = engine.work("projected", self.split), engine.work32("scalars", max(self.scalars, 1))
-        engine.record_linear(step, x, self.weight, projected, m=step.rows, n=self.total, k=engine.config.width,
-                             split=self.split, out32=scalars, bias=self.bias)
+        if self.cached:
+            keys, values = self.cached
+            step.run(step.element("dense_cached"),
+                     [x, self.weight, self.bias or self.weight, projected, scalars, engine.token_pool, engine.slot_table, step.past,
+                      step.sequence_rows],
+                     parameters.dense_cached(m=step.rows, n=self.total, k=engine.config.width, split=self.split, tokens=step.tokens,
+                                             key_columns=keys, value_columns=values, has_bias=self.bias is not None,
+                                             **engine.cache_rows(self.region)))
+        else:
+            engine.record_linear(step, x, self.weight, projected, m=step.rows, n=self.total, k=engine.config.width,
+                                 split=self.split, out32=scalars, bias=self.bias)
         return projected, scalars
 
 
@@ -87,52 +102,67 @@ def fused_step(step: Step, spec) -> bool:
 
 
 class AttentionMixer:
-    """Causal attention over the unquantised row cache."""
+    """Causal attention over the unquantised row cache.  Where queries and keys are used as they are projected
+    (no head norm, no rotation), the projection writes keys and values into the cache and the scores read the queries
+    from its rows; otherwise a kernel between the two prepares them."""
 
-    def __init__(self, engine, spec: AttentionSpec, weights, prefix: str, projection: Projection):
-        self.spec, self.projection, self.prefix = spec, projection, prefix
-        self.region = engine.next_attention_region()
+    def __init__(self, engine, spec: AttentionSpec, weights, prefix: str, projection: Projection, layer: int, branch: int):
+        self.spec, self.projection, self.prefix, self.branch = spec, projection, prefix, branch
+        self.region = engine.attention_region(layer, spec)
+        self.own_keys = spec.kv_from is None
+        direct = self.own_keys and not spec.prepared and projection.region is None
         bias = (lambda name: weights[f"{prefix}.{name}.b"]) if spec.bias else (lambda name: None)
-        for name in "qkv":
-            projection.add(f"{prefix}.{name}", weights[f"{prefix}.{name}"], bias(name))
+        projection.add(f"{prefix}.q", weights[f"{prefix}.q"], bias("q"))
+        if spec.gate:
+            projection.add(f"{prefix}.g", weights[f"{prefix}.g"])
+        if self.own_keys:
+            for name in "kv":
+                projection.add(f"{prefix}.{name}", weights[f"{prefix}.{name}"], bias(name), cache=direct)
+        if direct:
+            projection.region = self.region
+        self.prepares = not direct and (self.own_keys or spec.prepared)
         self.out = engine.upload_matrix(weights[f"{prefix}.o"])
         self.out_bias = engine.upload_vector(bias("o")) if spec.bias else None
-        self.head_norms = [engine.upload_vector(weights[f"{prefix}.{name}.norm"]) for name in "qk"] if spec.head_norm else None
-        self.trig = engine.rotary_table(spec.rotary)
+        self.head_norms = [engine.upload_vector(weights[f"{prefix}.{name}.norm"]) for name in ("qk" if self.own_keys else "qq")
+                           ] if spec.head_norm else None
+        self.trig = engine.rotary_table(spec.rotary) if spec.rotary else None
 
-    def record(self, step: Step, projected: Buffer, scalars: Buffer, y: Buffer) -> None:
+    def record(self, step: Step, projected: Buffer, scalars: Buffer) -> None:
         engine, spec, columns = step.engine, self.spec, self.projection.columns
-        query = engine.work("query", spec.heads * spec.dim)
         attended = engine.work("mixed", spec.heads * spec.vdim)
         shape = dict(sequences=step.sequences, tokens=step.tokens, heads=spec.heads, kv_heads=spec.kv_heads, dim=spec.dim,
                      vdim=spec.vdim)
-        cache = dict(token_stride=engine.layout.token_elements, key_offset=self.region.key_offset,
-                     value_offset=self.region.value_offset, table_stride=engine.sequences.stride,
-                     table_rows=engine.sequences.rows, pool_rows=engine.token_capacity)
-        q_norm, k_norm = self.head_norms or (self.trig, self.trig)
-        step.run(step.element("row_attention_prepare"),
-                 [projected, q_norm, k_norm, self.trig, query, engine.token_pool, engine.slot_table, step.past,
-                  step.sequence_rows],
-                 parameters.row_attention_prepare(
-                     **shape, stride=self.projection.split, q_column=columns[f"{self.prefix}.q"],
-                     k_column=columns[f"{self.prefix}.k"], v_column=columns[f"{self.prefix}.v"],
-                     rotary_dims=spec.rotary.dims, trig_rows=engine.capacity, **cache, head_norm=spec.head_norm,
-                     epsilon=engine.config.epsilon))
+        cache = engine.cache_rows(self.region)
+        stride, column = self.projection.split, lambda name: columns[f"{self.prefix}.{name}"]
+        query, queries = projected, dict(query_stride=stride, query_column=column("q"))
+        if self.prepares:
+            query, queries = engine.work("query", spec.heads * spec.dim), {}
+            trig = self.trig or projected
+            q_norm, k_norm = self.head_norms or (trig, trig)
+            step.run(step.element("row_attention_prepare"),
+                     [projected, q_norm, k_norm, trig, query, engine.token_pool, engine.slot_table, step.past, step.sequence_rows],
+                     parameters.row_attention_prepare(
+                         **shape, stride=stride, q_column=column("q"), k_column=column("k") if self.own_keys else 0,
+                         v_column=column("v") if self.own_keys else 0, rotary_dims=spec.rotary.dims if spec.rotary else 0,
+                         trig_rows=engine.capacity, **cache, head_norm=spec.head_norm, epsilon=engine.config.epsilon,
+                         own_keys=self.own_keys))
+        gate = dict(gate_stride=stride, gate_column=column("g")) if spec.gate else {}
+        window = dict(window=spec.window.size, keep_first=spec.window.keep_first) if spec.window else {}
         splits, scratch = engine.attention_splits(step, spec)
         step.run(step.element("row_attention"),
-                 [query, engine.token_pool, engine.slot_table, step.past, step.sequence_rows, attended, scratch],
-                 parameters.row_attention(**shape, **cache, sink=spec.sink, splits=splits, scale=spec.scale))
-        engine.record_linear(step, attended, self.out, None, m=step.rows, n=engine.config.width,
-                             k=spec.heads * spec.vdim, split=0, out32=y, bias=self.out_bias)
+                 [query, engine.token_pool, engine.slot_table, step.past, step.sequence_rows, attended, scratch, projected],
+                 parameters.row_attention(**shape, **cache, sink=spec.sink, splits=splits, scale=spec.scale,
+                                          softcap=spec.softcap or 0.0, weights32=spec.weights32, **queries, **gate, **window))
+        step.stream.product(attended, self.out, k=spec.heads * spec.vdim, bias=self.out_bias, branch=self.branch)
 
 
 class DeltaMixer:
     """Gated delta rule over short-convolved, unit-length q and k."""
 
-    def __init__(self, engine, spec: DeltaSpec, weights, prefix: str, projection: Projection):
+    def __init__(self, engine, spec: DeltaSpec, weights, prefix: str, projection: Projection, layer: int, branch: int):
         from .safetensors_archive import as_float32
 
-        self.spec, self.projection, self.prefix = spec, projection, prefix
+        self.spec, self.projection, self.prefix, self.branch = spec, projection, prefix, branch
         for name in "qkvg":
             projection.add(f"{prefix}.{name}", weights[f"{prefix}.{name}"])
         for name in "ba":
@@ -147,7 +177,7 @@ class DeltaMixer:
         self.state = engine.empty_bytes(rows * self.state_stride * 4)
         self.conv_state = engine.empty_bytes(rows * self.channels * spec.taps * engine.itemsize)
 
-    def record(self, step: Step, projected: Buffer, scalars: Buffer, y: Buffer) -> None:
+    def record(self, step: Step, projected: Buffer, scalars: Buffer) -> None:
         engine, spec, columns = step.engine, self.spec, self.projection.columns
         qk, vs = spec.kv_heads * spec.dim, spec.heads * spec.vdim
         q, k, v = engine.work32("delta_q", qk), engine.work32("delta_k", qk), engine.work32("delta_v", vs)
@@ -167,7 +197,7 @@ class DeltaMixer:
                          gate_column=columns[f"{self.prefix}.g"], scalar_stride=self.projection.scalars,
                          first_column=columns[f"{self.prefix}.b"], second_column=columns[f"{self.prefix}.a"], state_rows=rows,
                          state_stride=self.state_stride, gate_cap=0.0, epsilon=engine.config.epsilon))
-            engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+            step.stream.product(mixed, self.out, k=vs, branch=self.branch)
             return
         prepare = parameters.delta_prepare(
             **shape, taps=spec.taps, stride=self.projection.split, q_column=columns[f"{self.prefix}.q"],
@@ -186,14 +216,14 @@ class DeltaMixer:
                  parameters.head_norm_gate(rows=step.rows, heads=spec.heads, dim=spec.vdim,
                                            gate_stride=self.projection.split, gate_column=columns[f"{self.prefix}.g"],
                                            weight_per_head=False, gate_sigmoid=False, epsilon=engine.config.epsilon))
-        engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+        step.stream.product(mixed, self.out, k=vs, branch=self.branch)
 
 
 class MatrixMemoryMixer:
     """Matrix memory with stabilised exponential input and forget gates."""
 
-    def __init__(self, engine, spec: MatrixMemorySpec, weights, prefix: str, projection: Projection):
-        self.spec, self.projection, self.prefix = spec, projection, prefix
+    def __init__(self, engine, spec: MatrixMemorySpec, weights, prefix: str, projection: Projection, layer: int, branch: int):
+        self.spec, self.projection, self.prefix, self.branch = spec, projection, prefix, branch
         for name in "qkvg":
             projection.add(f"{prefix}.{name}", weights[f"{prefix}.{name}"])
         for name in "if":
@@ -203,7 +233,7 @@ class MatrixMemoryMixer:
         self.state_stride = matrix_state_elements(spec.heads, spec.dim, spec.vdim, normalized=True)
         self.state = engine.empty_bytes(engine.sequences.rows * self.state_stride * 4)
 
-    def record(self, step: Step, projected: Buffer, scalars: Buffer, y: Buffer) -> None:
+    def record(self, step: Step, projected: Buffer, scalars: Buffer) -> None:
         engine, spec, columns = step.engine, self.spec, self.projection.columns
         vs, stride = spec.heads * spec.vdim, self.projection.split
         read_out, mixed = engine.work32("read_out", vs), engine.work("mixed", vs)
@@ -217,7 +247,7 @@ class MatrixMemoryMixer:
                          scalar_stride=self.projection.scalars, first_column=columns[f"{self.prefix}.i"],
                          second_column=columns[f"{self.prefix}.f"], state_rows=engine.sequences.rows,
                          state_stride=self.state_stride, gate_cap=spec.gate_cap, epsilon=engine.config.epsilon))
-            engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+            step.stream.product(mixed, self.out, k=vs, branch=self.branch)
             return
         step.run(step.element("memory_scan"),
                  [projected, projected, projected, scalars, scalars, self.state, step.past, step.sequence_rows, read_out],
@@ -232,7 +262,7 @@ class MatrixMemoryMixer:
                  parameters.head_norm_gate(rows=step.rows, heads=spec.heads, dim=spec.vdim, gate_stride=stride,
                                            gate_column=columns[f"{self.prefix}.g"], weight_per_head=True,
                                            gate_sigmoid=True, epsilon=engine.config.epsilon))
-        engine.record_linear(step, mixed, self.out, None, m=step.rows, n=engine.config.width, k=vs, split=0, out32=y)
+        step.stream.product(mixed, self.out, k=vs, branch=self.branch)
 
 
 SINGLE_MIXERS = {AttentionSpec: AttentionMixer, DeltaSpec: DeltaMixer, MatrixMemorySpec: MatrixMemoryMixer}
@@ -241,30 +271,24 @@ SINGLE_MIXERS = {AttentionSpec: AttentionMixer, DeltaSpec: DeltaMixer, MatrixMem
 class LayerMixer:
     """A layer's mixer: one, or two side by side whose normed outputs the residual norm averages."""
 
-    def __init__(self, engine, spec, weights, prefix: str):
+    def __init__(self, engine, spec, weights, prefix: str, layer: int):
         self.projection = Projection()
         self.branch_norms = None
         if isinstance(spec, ParallelSpec):
-            self.branches = [SINGLE_MIXERS[type(one)](engine, one, weights, f"{prefix}.{side}", self.projection)
-                             for side, one in (("left", spec.left), ("right", spec.right))]
+            self.branches = [SINGLE_MIXERS[type(one)](engine, one, weights, f"{prefix}.{side}", self.projection, layer, branch)
+                             for branch, (side, one) in enumerate((("left", spec.left), ("right", spec.right)))]
             self.branch_norms = [engine.upload_vector(weights[f"{prefix}.{side}.out"]) for side in ("left", "right")]
         else:
-            self.branches = [SINGLE_MIXERS[type(spec)](engine, spec, weights, prefix, self.projection)]
+            self.branches = [SINGLE_MIXERS[type(spec)](engine, spec, weights, prefix, self.projection, layer, 0)]
         self.projection.upload(engine)
 
-    def record(self, step: Step, x: Buffer) -> List[Buffer]:
-        """Outputs of the branches."""
-        projected, scalars = self.projection.record(step, x)
-        outputs = [step.engine.work32(f"sublayer_{index}", step.engine.config.width) for index in range(len(self.branches))]
-        for branch, y in zip(self.branches, outputs):
-            branch.record(step, projected, scalars, y)
-        return outputs
+    def record(self, step: Step) -> None:
+        projected, scalars = self.projection.record(step, step.stream.x)
+        for branch in self.branches:
+            branch.record(step, projected, scalars)
 
 
 def attention_specs(config) -> list:
-    """Attention mixers of a model in the order their layers claim cache regions."""
-    found = []
-    for layer in config.layers:
-        branches = (layer.mixer.left, layer.mixer.right) if isinstance(layer.mixer, ParallelSpec) else (layer.mixer,)
-        found += [spec for spec in branches if isinstance(spec, AttentionSpec)]
-    return found
+    """(layer, attention mixer) of every cache region of a model: one per mixer with keys and values of its own."""
+    return [(index, spec) for index, layer in enumerate(config.layers) for spec in layer.mixers
+            if isinstance(spec, AttentionSpec) and spec.kv_from is None]

@@ -5,8 +5,8 @@ weights are random-init and quantised W4A16 group-64; there is no checkpoint
 loader for them here — a compiled package brings its own tensors.
 
 The second part describes decoders composed of sequence mixers (attention over
-unquantised cache rows, gated delta rule, matrix memory, two of them side by side)
-with dense bfloat16 weights, which are read from a folder with a config.json and a
+unquantised cache rows, gated delta rule, matrix memory, two of them side by side) and
+dense or routed feed-forward layers with bfloat16 weights, which are read from a folder with a config.json and a
 safetensors checkpoint: ``ARCHITECTURES`` maps the config's architecture name to the
 function that reads it."""
 
@@ -146,16 +146,34 @@ class RotarySpec:
 
 
 @dataclass(frozen=True)
+class WindowSpec:
+    """A token sees the last ``size`` tokens (itself included) and the first ``keep_first`` of the sequence."""
+
+    size: int
+    keep_first: int = 0
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     scale: float
-    rotary: RotarySpec
+    rotary: Optional[RotarySpec] = None
     bias: bool = False       # on q, k, v and the output projection
     head_norm: bool = False  # RMS norm of every query and key head before rotation
     sink: bool = False       # one more term exp(0) in the softmax denominator
+    window: Optional[WindowSpec] = None
+    softcap: Optional[float] = None  # score <- softcap * tanh(score / softcap)
+    gate: bool = False               # read-outs times the sigmoid of a projection of the mixer's input
+    kv_from: Optional[int] = None    # no keys and values of its own: those of that (earlier) layer
+    weights32: bool = False          # softmax weights are not rounded to bfloat16 before they meet the values
+
+    @property
+    def prepared(self) -> bool:
+        """Whether queries and keys change between projection and scores."""
+        return self.head_norm or self.rotary is not None
 
 
 @dataclass(frozen=True)
@@ -185,8 +203,21 @@ class ParallelSpec:
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
+    """down(activation(up x)), or, with ``gated``, down(silu(gate x) * up x)."""
+
     width: int
     activation: str = "gelu"
+    gated: bool = False
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Routed gated feed-forward layers: a token goes through the ``top`` of ``experts`` with the largest scores (sigmoid of
+    the router's logits); a score, not renormalised, multiplies its expert's input, and the outputs are added."""
+
+    experts: int
+    top: int
+    width: int
 
 
 @dataclass(frozen=True)
@@ -199,13 +230,20 @@ class TokenSideSpec:
 @dataclass(frozen=True)
 class MixerLayer:
     mixer: Union[AttentionSpec, DeltaSpec, MatrixMemorySpec, ParallelSpec]
-    feed_forward: Optional[FeedForwardSpec]
+    feed_forward: Union[None, FeedForwardSpec, ExpertsSpec]
+
+    @property
+    def mixers(self) -> tuple:
+        return (self.mixer.left, self.mixer.right) if isinstance(self.mixer, ParallelSpec) else (self.mixer,)
 
 
 @dataclass(frozen=True)
 class MixerConfig:
-    """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), x <- x + norm(token side(x)) per layer; the sublayer
-    norms multiply by ``norm_offset`` + weight."""
+    """With ``norm`` "rms": x <- x + norm(mixer(x)), x <- x + norm(ff(x)), x <- x + norm(token side(x)) per layer; the
+    sublayer norms are RMS norms that multiply by ``norm_offset`` + weight.
+
+    With ``norm`` "tanh" every sublayer has a norm before and one after it, x <- x + post(sublayer(pre(x))), and a norm is
+    tanh(alpha x) weight + bias."""
 
     name: str
     width: int
@@ -214,23 +252,48 @@ class MixerConfig:
     epsilon: float
     norm_offset: float = 0.0
     token_side: Optional[TokenSideSpec] = None
+    norm: str = "rms"
+    sinusoid: bool = False      # sinusoidal positions are added to the embedding
+    tied_head: bool = False     # the embedding table is the output projection too
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         if self.width <= 0 or self.vocabulary <= 0 or not self.layers:
             raise ValueError("a model needs a width, a vocabulary and layers")
-        for layer in self.layers:
-            mixers = (layer.mixer.left, layer.mixer.right) if isinstance(layer.mixer, ParallelSpec) else (layer.mixer,)
-            for mixer in mixers:
+        if self.norm not in ("rms", "tanh"):
+            raise ValueError(f"unsupported norm: {self.norm}")
+        if self.sinusoid != (self.norm == "tanh"):
+            raise ValueError("sinusoidal positions come with tanh norms, and those with sinusoidal positions")
+        for index, layer in enumerate(self.layers):
+            feed_forward = layer.feed_forward
+            if self.norm == "tanh" and (self.token_side or isinstance(layer.mixer, ParallelSpec)):
+                raise ValueError("tanh norms take single mixers and no token side input")
+            if isinstance(feed_forward, ExpertsSpec):
+                if self.norm != "tanh":
+                    raise ValueError("routed experts come with tanh norms")
+                if not 0 < feed_forward.top <= feed_forward.experts or feed_forward.width <= 0:
+                    raise ValueError("a token needs at least one expert and at most all of them")
+            for mixer in layer.mixers:
                 kv_heads = getattr(mixer, "kv_heads", mixer.heads)
                 if min(mixer.heads, kv_heads, mixer.dim, mixer.vdim) <= 0 or mixer.heads % kv_heads:
                     raise ValueError("query heads must come in whole groups per key/value head")
-                if isinstance(mixer, AttentionSpec) and (mixer.rotary.dims % 2 or mixer.rotary.dims > mixer.dim):
+                if not isinstance(mixer, AttentionSpec):
+                    continue
+                if mixer.rotary and (mixer.rotary.dims % 2 or mixer.rotary.dims > mixer.dim):
                     raise ValueError("rotated dimensions come in pairs inside the head")
+                if mixer.window and (mixer.window.size <= 0 or mixer.window.keep_first < 0):
+                    raise ValueError("a window sees at least the token itself")
+                if mixer.kv_from is not None:
+                    source = self.layers[mixer.kv_from].mixer if 0 <= mixer.kv_from < index else None
+                    if not isinstance(source, AttentionSpec) or source.kv_from is not None:
+                        raise ValueError("keys and values can be shared with an earlier attention layer that has its own")
+                    if (source.kv_heads, source.dim, source.vdim) != (mixer.kv_heads, mixer.dim, mixer.vdim):
+                        raise ValueError("layers that share keys and values need equal key and value heads")
 
 
 ARCHITECTURES: Dict[str, Callable[[dict], MixerConfig]] = {}
 # the module that registers each architecture, imported when it is first asked for
-ARCHITECTURE_MODULES = {"Bizodra": "bizodra"}
+ARCHITECTURE_MODULES = {"Bizodra": "bizodra", "Dalorax": "dalorax"}
 
 
 def register_architecture(name: str):
@@ -258,6 +321,22 @@ def load_model(folder: str):
     return config, Archive(os.path.join(folder, "model.safetensors"))
 
 
+def kernel_family(config: MixerConfig) -> str:
+    """The smallest family of kernels (``_build.FAMILIES``) that serves a model."""
+    attention = all(isinstance(mixer, AttentionSpec) for layer in config.layers for mixer in layer.mixers)
+    return "attention" if attention else "mixers"
+
+
+def sublayer_norms(config: MixerConfig) -> list:
+    """Tensor names of the norms of every sublayer in order: (before, after) with tanh norms, (after,) with RMS norms."""
+    names = []
+    for index, layer in enumerate(config.layers):
+        for place in (1, 2) if layer.feed_forward else (1,):
+            name = f"l{index}.norm{place}"
+            names.append((name, f"{name}b") if config.norm == "tanh" else (name,))
+    return names
+
+
 def mixer_tensors(config: MixerConfig) -> Dict[str, tuple]:
     """Name and shape of every tensor of a checkpoint."""
     width, shapes = config.width, {}
@@ -274,17 +353,21 @@ def mixer_tensors(config: MixerConfig) -> Dict[str, tuple]:
         heads, kv_heads = spec.heads, getattr(spec, "kv_heads", spec.heads)
         query_heads = kv_heads if isinstance(spec, DeltaSpec) else heads
         value_heads = heads if isinstance(spec, DeltaSpec) else kv_heads
+        shared = isinstance(spec, AttentionSpec) and spec.kv_from is not None
         for name, rows in (("q", query_heads * spec.dim), ("k", kv_heads * spec.dim), ("v", value_heads * spec.vdim)):
-            shapes[f"{prefix}.{name}"] = (rows, width)
+            if name == "q" or not shared:
+                shapes[f"{prefix}.{name}"] = (rows, width)
         shapes[f"{prefix}.o"] = (width, heads * spec.vdim)
+        if not isinstance(spec, AttentionSpec) or spec.gate:
+            shapes[f"{prefix}.g"] = (heads * spec.vdim, width)
         if isinstance(spec, AttentionSpec):
             if spec.bias:
-                for name in "qkvo":
+                for name in "qo" if shared else "qkvo":
                     shapes[f"{prefix}.{name}.b"] = shapes[f"{prefix}.{name}"][:1]
             if spec.head_norm:
-                shapes[f"{prefix}.q.norm"] = shapes[f"{prefix}.k.norm"] = (spec.dim,)
+                for name in "q" if shared else "qk":
+                    shapes[f"{prefix}.{name}.norm"] = (spec.dim,)
             return
-        shapes[f"{prefix}.g"] = (heads * spec.vdim, width)
         if isinstance(spec, DeltaSpec):
             for name in "qkv":
                 shapes[f"{prefix}.{name}.conv"] = (shapes[f"{prefix}.{name}"][0], spec.taps)
@@ -297,19 +380,39 @@ def mixer_tensors(config: MixerConfig) -> Dict[str, tuple]:
                 shapes[f"{prefix}.{name}"] = (heads, width)
                 shapes[f"{prefix}.{name}.b"] = (heads,)
 
+    def gated(prefix, inner):
+        shapes[f"{prefix}.gate"] = shapes[f"{prefix}.up"] = (inner, width)
+        shapes[f"{prefix}.down"] = (width, inner)
+
+    def norm(*names):
+        for name in names:
+            shapes[name] = (width,)
+            if config.norm == "tanh":
+                shapes[f"{name}.b"], shapes[f"{name}.alpha"] = (width,), ()
+
+    around = iter(sublayer_norms(config))
     for index, layer in enumerate(config.layers):
-        shapes[f"l{index}.norm1"] = (width,)
+        norm(*next(around))
         mixer(f"l{index}.mix", layer.mixer)
-        if layer.feed_forward:
-            shapes[f"l{index}.norm2"] = (width,)
-            shapes[f"l{index}.mlp.up"] = (layer.feed_forward.width, width)
-            shapes[f"l{index}.mlp.down"] = (width, layer.feed_forward.width)
+        feed_forward, prefix = layer.feed_forward, f"l{index}.mlp"
+        if feed_forward:
+            norm(*next(around))
+        if isinstance(feed_forward, ExpertsSpec):
+            shapes[f"{prefix}.router"] = (feed_forward.experts, width)
+            for expert in range(feed_forward.experts):
+                gated(f"{prefix}.e{expert}", feed_forward.width)
+        elif feed_forward and feed_forward.gated:
+            gated(prefix, feed_forward.width)
+        elif feed_forward:
+            shapes[f"{prefix}.up"] = (feed_forward.width, width)
+            shapes[f"{prefix}.down"] = (width, feed_forward.width)
         if config.token_side:
             shapes[f"l{index}.side.gate"] = (config.token_side.dim, width)
             shapes[f"l{index}.side.proj"] = (width, config.token_side.dim)
             shapes[f"l{index}.side.norm"] = (width,)
-    shapes["final.norm"] = (width,)
-    shapes["head"] = (config.vocabulary, width)
+    norm("final.norm")
+    if not config.tied_head:
+        shapes["head"] = (config.vocabulary, width)
     return shapes
 
 
@@ -324,7 +427,9 @@ def random_mixer_weights(config: MixerConfig, seed: int = 0, std: float = 0.02, 
     for name, shape in mixer_tensors(config).items():
         leaf = name.rsplit(".", 1)[-1]
         offset = config.norm_offset if leaf in ("norm1", "norm2") or name == "final.norm" else 0.0
-        if leaf in ("norm1", "norm2", "norm", "out"):
+        if leaf == "alpha":
+            value = rng.uniform(0.4, 0.8, size=shape)
+        elif leaf in ("norm1", "norm2", "norm1b", "norm2b", "norm", "out"):
             value = rng.uniform(0.8, 1.2, size=shape) - offset
         elif leaf == "A_log":
             value = np.log(rng.uniform(1.0, 8.0, size=shape))

@@ -165,13 +165,50 @@ def pointwise(*, output_shape, left_shape=None, right_shape=None, left_scalar=No
 
 
 # ---- sequence-mixer kernels (no reference counterpart; layouts of csrc/dense_linear.cu, sequence_glue.cu,
-# ---- row_attention.cu and matrix_state.cu) ---------------------------------------------------------------
+# ---- row_attention.cu, experts.cu and matrix_state.cu) ---------------------------------------------------------------
 
-DENSE_EPILOGUES = {None: 0, "gelu": 1, "token_gate": 2}
+DENSE_EPILOGUES = {None: 0, "gelu": 1, "token_gate": 2, "silu_pair": 3}
 
 
-def dense_linear(*, m, n, k, split, has_bias=False, epilogue=None, table_rows=0, table_stride=0, table_offset=0) -> bytes:
-    return u32s([m, n, k, split, 1 if has_bias else 0, DENSE_EPILOGUES[epilogue], table_rows, table_stride, table_offset])
+def dense_linear(*, m, n, k, split, has_bias=False, epilogue=None, table_rows=0, table_stride=0, table_offset=0,
+                 scale=1.0) -> bytes:
+    return u32s([m, n, k, split, 1 if has_bias else 0, DENSE_EPILOGUES[epilogue], table_rows, table_stride,
+                 table_offset]) + struct.pack("<f", scale)
+
+
+def dense_cached(*, m, n, k, split, tokens, key_columns, value_columns, token_stride, key_offset, value_offset, table_stride,
+                 table_rows, pool_rows, has_bias=False) -> bytes:
+    return u32s([m, n, k, split, 1 if has_bias else 0, tokens, key_columns, value_columns, token_stride, key_offset,
+                 value_offset, table_stride, table_rows, pool_rows])
+
+
+def dense_residual(*, m, n, k, has_bias=False) -> bytes:
+    return u32s([m, n, k, 1 if has_bias else 0])
+
+
+def embedding_sinusoid(*, rows, tokens, vocabulary, width) -> bytes:
+    return u32s([rows, tokens, vocabulary, width])
+
+
+def gather_rows(*, count, source_rows, width) -> bytes:
+    return u32s([count, source_rows, width])
+
+
+def route(*, rows, experts, top) -> bytes:
+    """Of route_step, route_rows and route_plan."""
+    return u32s([rows, experts, top])
+
+
+def expert_step(*, rows, n, k, experts, top) -> bytes:
+    return u32s([rows, n, k, experts, top])
+
+
+def expert_rows(*, pairs, n, k, experts, paired) -> bytes:
+    return u32s([pairs, n, k, experts, 1 if paired else 0])
+
+
+def expert_combine(*, rows, width, top) -> bytes:
+    return u32s([rows, width, top])
 
 
 def residual_norm(*, rows, width, epsilon, weight_offset, pair=False) -> bytes:
@@ -184,16 +221,21 @@ def gather_norm(*, count, source_rows, width, epsilon, weight_offset) -> bytes:
 
 def row_attention_prepare(*, sequences, tokens, heads, kv_heads, dim, vdim, stride, q_column, k_column, v_column,
                           rotary_dims, trig_rows, token_stride, key_offset, value_offset, table_stride, table_rows,
-                          pool_rows, head_norm, epsilon) -> bytes:
+                          pool_rows, head_norm, epsilon, own_keys=True) -> bytes:
     return u32s([sequences, tokens, heads, kv_heads, dim, vdim, stride, q_column, k_column, v_column, rotary_dims,
                  trig_rows, token_stride, key_offset, value_offset, table_stride, table_rows, pool_rows,
-                 1 if head_norm else 0]) + struct.pack("<f", epsilon)
+                 1 if head_norm else 0]) + struct.pack("<fI", epsilon, 1 if own_keys else 0)
 
 
 def row_attention(*, sequences, tokens, heads, kv_heads, dim, vdim, token_stride, key_offset, value_offset, table_stride,
-                  table_rows, pool_rows, sink, splits, scale) -> bytes:
+                  table_rows, pool_rows, sink, splits, scale, softcap=0.0, window=0, keep_first=0, query_stride=None,
+                  query_column=0, gate_stride=0, gate_column=0, weights32=False) -> bytes:
+    """``query_stride``: by default the queries are packed; ``window`` 0: every earlier key is visible; ``gate_stride`` 0:
+    the read-outs are not gated."""
     return u32s([sequences, tokens, heads, kv_heads, dim, vdim, token_stride, key_offset, value_offset, table_stride,
-                 table_rows, pool_rows, 1 if sink else 0, splits]) + struct.pack("<f", scale)
+                 table_rows, pool_rows, 1 if sink else 0, splits]) + struct.pack("<ff", scale, softcap) + u32s(
+                     [window, keep_first, heads * dim if query_stride is None else query_stride, query_column, gate_stride,
+                      gate_column, 1 if weights32 else 0])
 
 
 def head_norm_gate(*, rows, heads, dim, gate_stride, gate_column, weight_per_head, gate_sigmoid, epsilon) -> bytes:

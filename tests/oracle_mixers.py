@@ -210,6 +210,10 @@ def token_side(x, ids, index, w, prefix, dim, eps):
 
 def forward(config, w, tokens, per_layer=None):
     """Logits [tokens, vocab]; ``per_layer`` (a list) collects the residual after every layer."""
+    return FORWARD[config["architecture"]](config, w, tokens, per_layer)
+
+
+def forward_post_norm(config, w, tokens, per_layer=None):
     ids, eps = np.asarray(tokens), config["norm"]["eps"]
     x = f64(w["embed"])[ids]
     for index, layer in enumerate(config["layers"]):
@@ -225,11 +229,116 @@ def forward(config, w, tokens, per_layer=None):
     return linear(rms(x, eps) * (1.0 + f64(w["final.norm"])), w["head"])
 
 
+# ---- tanh norms before and after each sublayer, windowed attention, routed experts -----------
+def tanh_norm(x, w, name):
+    return np.tanh(f64(w[f"{name}.alpha"]).reshape(()) * x) * f64(w[name]) + f64(w[f"{name}.b"])
+
+
+def sinusoids(positions, width):
+    """Neighbouring entries 2i, 2i + 1: sine and cosine of position * 10000^(-2i / width)."""
+    column = np.arange(width)
+    angle = f64(positions)[:, None] * 10000.0 ** (-2.0 * (column // 2) / width)
+    return np.where(column % 2 == 0, np.sin(angle), np.cos(angle))
+
+
+def visible_keys(queries, keys, mask):
+    """[queries, keys] positions: not in the future, and near enough or among the first."""
+    distance = queries[:, None] - keys[None, :]
+    seen = distance >= 0
+    if mask:
+        seen &= (distance < mask["size"]) | (keys[None, :] < mask.get("keep_first", 0))
+    return seen
+
+
+def capped(score, cap):
+    return cap * np.tanh(score / cap) if cap else score
+
+
+def masked_attention(q, k, v, seen, scale, cap=None):
+    """q [T, H, dim], k [S, G, dim], v [S, G, vdim], seen [T, S]."""
+    group = q.shape[1] // k.shape[1]
+    out = np.zeros((*q.shape[:2], v.shape[2]))
+    for h in range(q.shape[1]):
+        score = np.where(seen, capped((q[:, h] @ k[:, h // group].T) * scale, cap), -np.inf)
+        weight = np.exp(score - score.max(axis=1, keepdims=True))
+        out[:, h] = weight / weight.sum(axis=1, keepdims=True) @ v[:, h // group]
+    return out
+
+
+def windowed_mixer(h, w, prefix, size, kept):
+    """``kept``: the keys and values of earlier layers by index; returns (output, own keys and values)."""
+    tokens = h.shape[0]
+    q = linear(h, w[f"{prefix}.q"]).reshape(tokens, size["heads"], size["dim"])
+    if size.get("kv_from") is not None:
+        k, v = kept[size["kv_from"]]
+    else:
+        k = linear(h, w[f"{prefix}.k"]).reshape(tokens, size["kv_heads"], size["dim"])
+        v = linear(h, w[f"{prefix}.v"]).reshape(tokens, size["kv_heads"], size["vdim"])
+    places = np.arange(tokens)
+    out = masked_attention(q, k, v, visible_keys(places, places, size.get("mask")), size["scale"], size.get("softcap"))
+    out = out.reshape(tokens, -1) * sigmoid(linear(h, w[f"{prefix}.g"]))
+    return linear(out, w[f"{prefix}.o"]), (k, v)
+
+
+def gated_feed_forward(x, w, prefix):
+    return linear(silu(linear(x, w[f"{prefix}.gate"])) * linear(x, w[f"{prefix}.up"]), w[f"{prefix}.down"])
+
+
+def chosen_experts(scores, top):
+    """[tokens, top] indices of the largest scores, the lower index first among equals."""
+    return np.argsort(-scores, axis=1, kind="stable")[:, :top]
+
+
+# (layer prefix -> choices) while ``rounding_error`` runs: its disturbed passes keep the undisturbed choices.
+_choices = None
+
+
+def routed_experts(h, w, prefix, router, margins=None):
+    z = linear(h, w[f"{prefix}.router"])
+    scores = sigmoid(z)
+    chosen = chosen_experts(z, router["top"])
+    if _choices is not None:
+        chosen = _choices.setdefault(prefix, chosen)
+    if margins is not None and router["top"] < router["experts"]:
+        ranked = -np.sort(-z, axis=1)
+        margins.append((ranked[:, router["top"] - 1] - ranked[:, router["top"]]) / z.std())
+    out = np.zeros_like(h)
+    for expert in range(router["experts"]):
+        for place in range(router["top"]):
+            rows = np.nonzero(chosen[:, place] == expert)[0]
+            if len(rows):
+                out[rows] += gated_feed_forward(scores[rows, expert][:, None] * h[rows], w, f"{prefix}.e{expert}")
+    return out
+
+
+def forward_sandwich(config, w, tokens, per_layer=None, margins=None):
+    """``margins`` (a list) collects, per routed layer, how far each token's last chosen expert is ahead of the next."""
+    ids, kept = np.asarray(tokens), {}
+    x = f64(w["embed"])[ids] + sinusoids(np.arange(len(ids)), config["width"])
+    for index, layer in enumerate(config["layers"]):
+        p = f"l{index}"
+        y, kept[index] = windowed_mixer(tanh_norm(x, w, f"{p}.norm1"), w, f"{p}.mix", layer["mixer"], kept)
+        x = x + tanh_norm(y, w, f"{p}.norm1b")
+        mlp = layer.get("mlp")
+        if mlp:
+            h = tanh_norm(x, w, f"{p}.norm2")
+            y = gated_feed_forward(h, w, f"{p}.mlp") if mlp["kind"] == "dense" else routed_experts(
+                h, w, f"{p}.mlp", mlp["router"], margins)
+            x = x + tanh_norm(y, w, f"{p}.norm2b")
+        if per_layer is not None:
+            per_layer.append(x.copy())
+    return linear(tanh_norm(x, w, "final.norm"), w["embed"]) * config["logit_scale"]
+
+
+FORWARD = {"Bizodra": forward_post_norm, "Dalorax": forward_sandwich}
+
+
 def rounding_error(config, w, tokens, relative, draws=4):
     """Per position, the largest root-mean-square change of the centred logits over some draws of relative
     errors of size ``relative`` in every matrix product (and of that size times the row's scale): how much
     of a difference rounding alone explains.  Positions where a read-out nearly cancels stand out."""
-    global _disturb
+    global _disturb, _choices
+    _choices = {}
     base, worst = forward(config, w, tokens), None
     for draw in range(draws):
         rng = np.random.default_rng(draw)
@@ -246,4 +355,5 @@ def rounding_error(config, w, tokens, relative, draws=4):
         change -= change.mean(axis=-1, keepdims=True)
         error = np.sqrt((change ** 2).mean(axis=-1))
         worst = error if worst is None else np.maximum(worst, error)
+    _choices = None
     return worst / np.sqrt(((base - base.mean(axis=-1, keepdims=True)) ** 2).mean())

@@ -168,7 +168,7 @@ class AttentionBench:
         for _ in range(2):  # the arrival counters return to zero
             self.runtime.dispatch(
                 "llmopt_row_attention_" + suffix(self.dtype),
-                buffers=[query, self.pool, self.table, past, self.row, out, scratch],
+                buffers=[query, self.pool, self.table, past, self.row, out, scratch, query],
                 parameters=parameters.row_attention(sequences=1, tokens=tokens, **size, **cache, sink=self.sink, splits=splits, scale=self.scale))
         self.past += tokens
         return download(out, (tokens, size["heads"], size["vdim"]), self.dtype)

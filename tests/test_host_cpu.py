@@ -99,7 +99,7 @@ def test_kernel_abi_surface():
     # families that keep their own name table are registered from it
     csrc = os.path.join(ROOT, "llmopt_b200", "csrc")
     sources = [os.path.join(csrc, name + ".cu") for name in ("runtime", "norm_family", "dense_linear", "sequence_glue",
-                                                             "row_attention", "matrix_state")]
+                                                             "row_attention", "matrix_state", "experts")]
     registered = set(re.findall(r'"(llmopt_[a-z0-9_]+)"', "".join(open(path).read() for path in sources)))
     assert {e.name for e in kernel_abi.ENTRIES} <= registered
 
