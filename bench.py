@@ -929,9 +929,10 @@ def main() -> None:
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--no-extra-legs", action="store_true",
                         help="only the headline batch: no batch-32, small-model, prefill-sweep or input-mode legs")
-    parser.add_argument("--mixers", action="store_true",
+    parser.add_argument("--mixers", nargs="?", const="bizodra", default=None, choices=["bizodra", "dalorax"],
                         help="instead: prefill and decode throughput and per-kernel rooflines of decoders composed of sequence "
-                             "mixers (random weights), beside the W4A16 decoder of equal size; one GPU")
+                             "mixers (random weights): bizodra beside the W4A16 decoder of equal size, dalorax beside "
+                             "bizodra; one GPU")
     parser.add_argument("--parallel", default="tp", choices=["tp", "replicas"],
                         help="with --gpus N > 1: tensor parallel (when the model splits over N) or N replicas")
     args = parser.parse_args()
@@ -940,8 +941,8 @@ def main() -> None:
         from llmopt_b200.cuda_native import Runtime
 
         runtime, sampler = Runtime(), ClockSampler(0)
-        sizes = mixer_bench.measure(runtime, measured_peaks())
-        print(json.dumps({"workload": "mixers", "data": "synthetic", "dtype": "bf16", "clocks": sampler.stop(), "sizes": sizes}),
+        sizes = mixer_bench.measure(runtime, measured_peaks(), design=args.mixers)
+        print(json.dumps({"workload": "mixers", "design": args.mixers, "data": "synthetic", "dtype": "bf16", "clocks": sampler.stop(), "sizes": sizes}),
               flush=True)
         return
     from llmopt_b200 import model

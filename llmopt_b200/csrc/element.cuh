@@ -60,7 +60,7 @@ __device__ __forceinline__ void store_four(bf16* target, const float4& v) {
 
 // Larger values first, then smaller columns, as one unsigned integer.
 __device__ __forceinline__ unsigned long long ranked(float value, uint32_t column) {
-  uint32_t bits = __float_as_uint(value);
+  uint32_t bits = __float_as_uint(value + 0.0f);  // both zeros are equal
   bits = (bits & 0x80000000u) ? ~bits : bits | 0x80000000u;
   return ((unsigned long long)bits << 32) | (0xffffffffu - column);
 }

@@ -1,8 +1,9 @@
 """Prefill and decode throughput of decoders composed of sequence mixers, and the roofline share of every
-kernel of their steps, beside the W4A16 decoder of the same width, depth, heads and vocabulary and the
-like kernels of that path.  Used by ``bench.py --mixers``; random weights.
+kernel of their steps: the recurrent design beside the W4A16 decoder of the same width, depth, heads and vocabulary
+and the like kernels of that path, the windowed design with routed experts beside the recurrent one.  Used by
+``bench.py --mixers``; random weights.
 
-  python -m llmopt_b200.mixer_bench [--size 2048|4096|all] [--tokens 2048] [--context 2048]"""
+  python -m llmopt_b200.mixer_bench [--design bizodra|dalorax] [--size 2048|4096|all] [--tokens 2048] [--context 2048]"""
 
 from __future__ import annotations
 
@@ -15,9 +16,11 @@ from types import SimpleNamespace
 
 import numpy as np
 
+from . import parameters
 from .cuda_native import Batch, Runtime
-from .model import (AttentionSpec, DeltaSpec, FeedForwardSpec, MatrixMemorySpec, MixerConfig, MixerLayer, ModelConfig,
-                    ParallelSpec, RotarySpec, TokenSideSpec, YarnSpec, random_mixer_weights, random_weights)
+from .model import (AttentionSpec, DeltaSpec, ExpertsSpec, FeedForwardSpec, MatrixMemorySpec, MixerConfig, MixerLayer,
+                    ModelConfig, ParallelSpec, RotarySpec, TokenSideSpec, WindowSpec, YarnSpec, random_mixer_weights,
+                    random_weights)
 
 
 def sized_config(width: int) -> MixerConfig:
@@ -36,6 +39,23 @@ def sized_config(width: int) -> MixerConfig:
                        token_side=TokenSideSpec(dim=256))
 
 
+def windowed_config(width: int) -> MixerConfig:
+    """The same width, depth, heads, feed-forward width and vocabulary with windowed attention; half of the layers read
+    another's keys and values, half have sixteen experts of a quarter of the feed-forward width, two per token."""
+    heads = width // 128
+
+    def layer(index):
+        attention = AttentionSpec(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, gate=True,
+                                  weights32=True, window=WindowSpec(size=1024, keep_first=4),
+                                  kv_from=index // 4 * 4 + 1 if index % 4 >= 2 else None)
+        routed = ExpertsSpec(experts=16, top=2, width=7 * width // 8)
+        return MixerLayer(mixer=attention, feed_forward=routed if index % 2 else FeedForwardSpec(
+            width=7 * width // 2, activation="silu", gated=True))
+
+    return MixerConfig(name=f"windows-{width}", width=width, vocabulary=32768, layers=tuple(layer(index) for index in range(8)),
+                       epsilon=1e-5, norm="tanh", sinusoid=True, tied_head=True)
+
+
 def like_config(config: MixerConfig) -> ModelConfig:
     """The W4A16 decoder of the same size."""
     heads = config.width // 128
@@ -45,6 +65,14 @@ def like_config(config: MixerConfig) -> ModelConfig:
 
 # ---- algorithmic work of a dispatch ------------------------------------------------------------------------
 
+def experts_in_use(item) -> int:
+    """Experts that some row of an expert kernel's step chose, from its device-side route or plan."""
+    words = item.buffers[2].to_numpy(np.uint32)
+    if "expert_step" in item.name:
+        return int(words[0])
+    return len(set(words[4:4 + 4 * int(words[0])].reshape(-1, 4)[:, 0].tolist()))
+
+
 def work_of(item, past: int, itemsize: int):
     """(label, bytes, flops) of a recorded dispatch; every operand once."""
     stem = item.name.removeprefix("llmopt_").removesuffix("_bf16").removesuffix("_f32")
@@ -52,7 +80,34 @@ def work_of(item, past: int, itemsize: int):
     e = itemsize
     if stem == "dense_linear":
         m, n, k, split = u[:4]
+        if u[5] == parameters.DENSE_EPILOGUES["silu_pair"]:
+            return f"dense_linear (pairs) n{n} k{k}", n * k * e + m * k * e + m * n // 2 * e, 2 * m * n * k
         return f"dense_linear n{n} k{k}", n * k * e + m * k * e + m * split * e + m * (n - split) * 4, 2 * m * n * k
+    if stem == "dense_cached":
+        m, n, k = u[:3]
+        return f"dense_cached n{n} k{k}", (n * k + m * k + m * n) * e, 2 * m * n * k
+    if stem == "dense_residual":
+        m, n, k = u[:3]
+        return f"dense_residual n{n} k{k}", (n * k + m * k + m * n) * e + m * n * 8, 2 * m * n * k
+    if stem in ("expert_step", "expert_step_residual"):
+        rows, n, k, experts, top = u
+        used = experts_in_use(item)
+        edges = rows * k + used * rows * n // 2 if stem == "expert_step" else used * rows * k + rows * n
+        return f"{stem} n{n} k{k}", (used * n * k + edges) * e + (rows * n * 8 if "residual" in stem else 0), 2 * rows * top * n * k
+    if stem == "expert_rows":
+        pairs, n, k, experts, paired = u
+        return (f"expert_rows n{n} k{k}", (experts_in_use(item) * n * k + pairs * k) * e + pairs * n * (e // 2 if paired else 4),
+                2 * pairs * n * k)
+    if stem in ("route_step", "route_rows", "route_plan"):
+        rows, experts, top = u
+        return stem, rows * (experts * 4 if stem != "route_plan" else top * 8) + rows * top * (8 if stem != "route_plan" else 12), 0
+    if stem == "expert_combine":
+        rows, width, top = u
+        return stem, rows * width * (4 * top + 8 + e), 0
+    if stem == "embedding_sinusoid":
+        return stem, u[0] * u[3] * (2 * e + 4), 0
+    if stem == "gather_rows":
+        return stem, u[0] * u[2] * 2 * e, 0
     if stem == "embedding_residual":
         return stem, u[0] * u[2] * (2 * e + 4), 0
     if stem == "residual_norm":
@@ -65,9 +120,14 @@ def work_of(item, past: int, itemsize: int):
         return stem, sequences * tokens * 2 * e * (heads * dim + kv_heads * (dim + vdim)), 0
     if stem == "row_attention":
         sequences, tokens, heads, kv_heads, dim, vdim = u[:6]
-        keys = past + tokens
-        pairs = tokens * past + tokens * (tokens + 1) // 2
-        return (stem, sequences * (keys * kv_heads * (dim + vdim) * e + tokens * heads * (dim + vdim) * e),
+        window, keep_first, gated = u[16], u[17], u[20] > 0
+        keys, pairs = past + tokens, tokens * past + tokens * (tokens + 1) // 2
+        if window:
+            seen = [min(past + t + 1, window + min(keep_first, max(0, past + t + 1 - window))) for t in range(tokens)]
+            pairs, keys = sum(seen), min(keys, window + tokens - 1 + keep_first)
+        if gated:
+            stem += " (windowed, gated)"
+        return (stem, sequences * (keys * kv_heads * (dim + vdim) * e + tokens * heads * (dim + vdim + (vdim if gated else 0)) * e),
                 2 * sequences * heads * pairs * (dim + vdim))
     if stem == "head_norm_gate":
         return stem, u[0] * u[1] * u[2] * (4 + 2 * e), 0
@@ -148,15 +208,17 @@ def measure_mixers(runtime, peaks: dict, config: MixerConfig, tokens: int, conte
         result["decode"].append(decode_rate(engine, batch, context))
         plan = engine._decode_plan(batch)[0]
         engine.rewind(context)
-        plan.write([1] * batch, [context] * batch, [engine._row(index) for index in range(batch)])
+        plan.write(list(range(1, batch + 1)), [context] * batch, [engine._row(index) for index in range(batch)])
         items = [item for item in plan.items if item.name != "llmopt_advance_tokens"]
+        runtime.time_dispatches(items, warmup=0, iterations=1)  # every kernel's own inputs, the routes among them
         result["kernels"][f"decode, {batch} sequences, {context} tokens behind"] = time_items(
             runtime, items, context, engine.itemsize, peaks)
         result["decode"][-1]["kernels_per_step"] = engine._decode_plan(batch)[1].kernel_count()
         if batch == 1:
             result["prefill"] = prefill_rate(engine, tokens)
             plan = engine._prompt_plan(tokens)[0]
-            plan.write([1] * tokens, [0], [engine._row(0)])
+            plan.write(np.random.default_rng(0).integers(0, config.vocabulary, size=tokens), [0], [engine._row(0)])
+            runtime.time_dispatches(plan.items, warmup=0, iterations=1)  # every kernel's own inputs, the routes among them
             result["kernels"][f"prompt of {tokens} tokens"] = time_items(runtime, plan.items, 0, engine.itemsize, peaks)
     return result
 
@@ -179,7 +241,7 @@ def measure_like(runtime, peaks: dict, config: MixerConfig, tokens: int, context
 
 def like_kernels(runtime, peaks: dict, config: MixerConfig, tokens: int, context: int) -> dict:
     """The like kernels of the W4A16 path at the same sizes: share of the roofline of each."""
-    from . import dispatch, kernel_bench, parameters
+    from . import dispatch, kernel_bench
     from .cuda_native import Buffer, DispatchItem
 
     width, heads = config.width, config.width // 128
@@ -240,28 +302,35 @@ def like_kernels(runtime, peaks: dict, config: MixerConfig, tokens: int, context
     return table
 
 
-def measure(runtime, peaks: dict, widths=(2048, 4096), tokens: int = 2048, context: int = 2048, like: bool = True) -> list:
+def measure(runtime, peaks: dict, widths=(2048, 4096), tokens: int = 2048, context: int = 2048, like: bool = True,
+            design: str = "bizodra") -> list:
     results = []
     for width in widths:
         config = sized_config(width)
-        entry = {"mixers": measure_mixers(runtime, peaks, config, tokens, context)}
-        if like:
-            entry["w4a16"] = measure_like(runtime, peaks, config, tokens, context)
-            entry["w4a16_kernels"] = like_kernels(runtime, peaks, config, tokens, context)
+        if design == "dalorax":
+            entry = {"windows": measure_mixers(runtime, peaks, windowed_config(width), tokens, context)}
+            if like:
+                entry["mixers"] = measure_mixers(runtime, peaks, config, tokens, context)
+        else:
+            entry = {"mixers": measure_mixers(runtime, peaks, config, tokens, context)}
+            if like:
+                entry["w4a16"] = measure_like(runtime, peaks, config, tokens, context)
+                entry["w4a16_kernels"] = like_kernels(runtime, peaks, config, tokens, context)
         results.append(entry)
     return results
 
 
 def main() -> None:
     parser = argparse.ArgumentParser()
+    parser.add_argument("--design", default="bizodra", choices=["bizodra", "dalorax"])
     parser.add_argument("--size", default="all", choices=["2048", "4096", "all"])
     parser.add_argument("--tokens", type=int, default=2048)
     parser.add_argument("--context", type=int, default=2048)
-    parser.add_argument("--no-like", action="store_true", help="only the mixer models")
+    parser.add_argument("--no-like", action="store_true", help="only the design itself")
     args = parser.parse_args()
     peaks = {"hbm_gbs": 6531.6, "bf16_tflops": 1657.8}
     widths = (2048, 4096) if args.size == "all" else (int(args.size),)
-    for entry in measure(Runtime(), peaks, widths, args.tokens, args.context, not args.no_like):
+    for entry in measure(Runtime(), peaks, widths, args.tokens, args.context, not args.no_like, args.design):
         print(json.dumps(entry, indent=1))
 
 
