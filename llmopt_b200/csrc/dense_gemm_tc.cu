@@ -48,10 +48,136 @@ __host__ __device__ constexpr uint32_t bf16_instruction(uint32_t m, uint32_t n) 
   return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((m >> 4) << 24);
 }
 
-template <uint32_t BN>
+// 32 neighbouring sums of an output row on their way out, and what they need besides, requested ahead of them.
+template <DenseStore STORE>
+struct Piece {
+  __device__ __forceinline__ void fetch(const DenseTask<STORE>&, uint32_t, uint32_t, uint32_t) {}
+  __device__ __forceinline__ void store(const DenseTask<STORE>& p, uint32_t row, uint32_t column, const uint32_t (&raw)[32]) const {
+    const uint32_t kept = dense_kept(p);
+    const size_t at = (size_t)row * p.split + column;
+    const size_t at32 = (size_t)row * (p.n - p.split - kept) + (column - p.split - kept);
+    auto value = [&](int i) {
+      return STORE == kStoreCached ? dense_biased(p, column + i, __uint_as_float(raw[i]))
+                                   : dense_finish<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+    };
+    if (column + 32u <= p.split && (at & 7u) == 0) {
+      uint4* target = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + at);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        uint32_t packed[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const __nv_bfloat162 pair = __floats2bfloat162_rn(value(i * 8 + j * 2), value(i * 8 + j * 2 + 1));
+          packed[j] = *reinterpret_cast<const uint32_t*>(&pair);
+        }
+        target[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+      }
+      return;
+    }
+    if (column >= p.split + kept && column + 32u <= p.n && (at32 & 3u) == 0) {
+      float4* target = reinterpret_cast<float4*>(p.out32 + at32);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) target[i] = make_float4(value(i * 4), value(i * 4 + 1), value(i * 4 + 2), value(i * 4 + 3));
+      return;
+    }
+    if constexpr (STORE == kStoreCached) {
+      if (column >= p.split && column + 32u <= p.split + kept) {
+        // one head may end and the next begin inside the piece, and keys may end and values begin
+        bf16* const cached = dense_cache_row<bf16>(p, row);
+        if (!cached) return;
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          const uint32_t first = dense_cache_offset(p, column - p.split + i), second = dense_cache_offset(p, column - p.split + i + 1);
+          if (second == first + 1u && ((uintptr_t)(cached + first) & 3u) == 0) {
+            *reinterpret_cast<__nv_bfloat162*>(cached + first) = __floats2bfloat162_rn(value(i), value(i + 1));
+          } else {
+            cached[first] = __float2bfloat16_rn(value(i));
+            cached[second] = __float2bfloat16_rn(value(i + 1));
+          }
+        }
+        return;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+  }
+};
+
+template <>
+struct Piece<kStorePair> {
+  __device__ __forceinline__ void fetch(const DenseTask<kStorePair>&, uint32_t, uint32_t, uint32_t) {}
+  __device__ __forceinline__ void store(const DenseTask<kStorePair>& p, uint32_t row, uint32_t column, const uint32_t (&raw)[32]) const {
+    bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * (p.n / 2u) + column / 2u;
+    const bool whole = column + 32u <= p.n && ((uintptr_t)target & 15u) == 0;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      uint32_t packed[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int e = i * 16 + j * 4;
+        float pair[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          pair[h] = column + e + 2 * h < p.n ? dense_pair(p, row, column + e + 2 * h, __uint_as_float(raw[e + 2 * h]),
+                                                          __uint_as_float(raw[e + 2 * h + 1]))
+                                             : 0.0f;
+        const __nv_bfloat162 both = __floats2bfloat162_rn(pair[0], pair[1]);
+        packed[j] = *reinterpret_cast<const uint32_t*>(&both);
+        if (!whole) {
+          if (column + e < p.n) target[i * 8 + j * 2] = both.x;
+          if (column + e + 2 < p.n) target[i * 8 + j * 2 + 1] = both.y;
+        }
+      }
+      if (whole) reinterpret_cast<uint4*>(target)[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+    }
+  }
+};
+
+template <>
+struct Piece<kStoreResidual> {
+  float4 x[8];
+  static __device__ __forceinline__ bool vectors(const DenseTask<kStoreResidual>& p, uint32_t column) {
+    return p.n % 4u == 0 && column + 32u <= p.n;
+  }
+  __device__ __forceinline__ void fetch(const DenseTask<kStoreResidual>& p, uint32_t row, uint32_t row_end, uint32_t column) {
+    if (row >= row_end || !vectors(p, column)) return;
+    const float4* source = reinterpret_cast<const float4*>(p.residual + (size_t)row * p.n + column);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = source[i];
+  }
+  __device__ __forceinline__ void store(const DenseTask<kStoreResidual>& p, uint32_t row, uint32_t column,
+                                        const uint32_t (&raw)[32]) const {
+    if (!vectors(p, column)) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+      return;
+    }
+    const TanhNorm post(p.post_norm, p.n), next(p.next_norm, p.n);
+    float4* residual = reinterpret_cast<float4*>(p.residual + (size_t)row * p.n + column);
+    bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * p.n + column;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float4 v = make_float4(__uint_as_float(raw[i * 4]), __uint_as_float(raw[i * 4 + 1]), __uint_as_float(raw[i * 4 + 2]),
+                             __uint_as_float(raw[i * 4 + 3]));
+      if (p.has_bias) {
+        const float* bias = p.bias + column + i * 4;
+        v.x += __ldg(bias), v.y += __ldg(bias + 1), v.z += __ldg(bias + 2), v.w += __ldg(bias + 3);
+      }
+      const float4 y = post.four_short(v, column + i * 4);
+      const float4 sum = make_float4(x[i].x + y.x, x[i].y + y.y, x[i].z + y.z, x[i].w + y.w);
+      residual[i] = sum;
+      store_four(target + i * 4, next.four_short(sum, column + i * 4));
+    }
+  }
+};
+
+template <uint32_t BN, DenseStore STORE>
 __global__ void __launch_bounds__(kThreads, 1)
 dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                     const DenseProblem p, uint32_t most_tiles, uint32_t* error_word) {
+                     const __grid_constant__ DenseTask<STORE> p, const DensePlan plan, uint32_t most_tiles,
+                     uint32_t* error_word) {
   using S = Shape<BN>;
   extern __shared__ unsigned char shared_raw[];
   grid_chain_prologue();
@@ -62,13 +188,13 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
   volatile uint32_t* holder = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kHolder);
   volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(base_pointer + S::kAbort);
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
-  const uint32_t m_tiles = p.plan ? min(p.plan[0], most_tiles) : (p.m + kRows - 1u) / kRows;
+  const uint32_t m_tiles = plan.tiles ? min(plan.tiles[0], most_tiles) : (p.m + kRows - 1u) / kRows;
   const uint32_t n_tiles = (p.n + BN - 1u) / BN, tiles = m_tiles * n_tiles;
   // first row, row end, and first row of the weights (column of the output) of a tile
   auto place = [&](uint32_t tile) -> DenseTile {
     const uint32_t m_tile = tile % m_tiles, n0 = tile / m_tiles * BN;
-    if (!p.plan) return {n0, m_tile * kRows, p.m};
-    const DenseTile rows = dense_tile(p, m_tile);
+    if (!plan.tiles) return {n0, m_tile * kRows, p.m};
+    const DenseTile rows = dense_tile(plan, m_tile);
     return {rows.expert * p.n + n0, rows.first, min(rows.end, p.m)};
   };
   const uint32_t k_stages = (p.k + kDepth * S::kBlocks - 1u) / (kDepth * S::kBlocks);
@@ -161,6 +287,10 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
     bool ok = true;
     for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++turn) {
       const uint32_t half = turn & 1u;
+      const DenseTile rows = place(tile);
+      const uint32_t row = rows.first + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
+      Piece<STORE> ahead;
+      ahead.fetch(p, row, rows.end, n0 + side * 32u);
       ok = !*abort_flag && barrier_wait(sums_full + half * 8, (turn >> 1) & 1u);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) {
@@ -168,106 +298,16 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
         break;
       }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const DenseTile rows = place(tile);
-      const uint32_t row = rows.first + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
-      bf16* const cached = p.cache.pool && row < p.m ? dense_cache_row<bf16>(p, row) : nullptr;
-      const uint32_t kept = dense_cache_columns(p);
       const uint32_t address = tmem_base + half * BN + ((quarter * 32u) << 16);
 #pragma unroll 1
       for (uint32_t piece = side; piece < BN / 32u; piece += kEpilogueWarps / 4u) {
         uint32_t raw[32];
         tmem_load_32(address + piece * 32u, raw);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-        const uint32_t column = n0 + piece * 32u;
-        const size_t at = (size_t)row * p.split + column;
-        const size_t at32 = (size_t)row * (p.n - p.split - kept) + (column - p.split - kept);
-        if (row >= rows.end || column >= p.n) {
-          // absent
-        } else if (p.epilogue == kDenseSiluPair) {
-          bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * (p.n / 2u) + column / 2u;
-          const bool whole = column + 32u <= p.n && ((uintptr_t)target & 15u) == 0;
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            uint32_t packed[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const int e = i * 16 + j * 4;
-              float pair[2];
-#pragma unroll
-              for (int h = 0; h < 2; ++h)
-                pair[h] = column + e + 2 * h < p.n ? dense_pair(p, row, column + e + 2 * h, __uint_as_float(raw[e + 2 * h]),
-                                                                __uint_as_float(raw[e + 2 * h + 1]))
-                                                   : 0.0f;
-              const __nv_bfloat162 both = __floats2bfloat162_rn(pair[0], pair[1]);
-              packed[j] = *reinterpret_cast<const uint32_t*>(&both);
-              if (!whole) {
-                if (column + e < p.n) target[i * 8 + j * 2] = both.x;
-                if (column + e + 2 < p.n) target[i * 8 + j * 2 + 1] = both.y;
-              }
-            }
-            if (whole) reinterpret_cast<uint4*>(target)[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
-          }
-        } else if (p.epilogue == kDenseResidualTanh && column + 32u <= p.n && p.n % 4u == 0) {
-          const TanhNorm post(p.post_norm, p.n), next(p.next_norm, p.n);
-          float* residual = p.residual + (size_t)row * p.n + column;
-          bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * p.n + column;
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            float v[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) v[j] = dense_finish<bf16>(p, row, column + i * 4 + j, __uint_as_float(raw[i * 4 + j]));
-            float4 x = reinterpret_cast<const float4*>(residual)[i];
-            const float4 y = post.four(make_float4(v[0], v[1], v[2], v[3]), column + i * 4);
-            x.x += y.x, x.y += y.y, x.z += y.z, x.w += y.w;
-            reinterpret_cast<float4*>(residual)[i] = x;
-            store_four(target + i * 4, next.four(x, column + i * 4));
-          }
-        } else if (p.epilogue != kDenseResidualTanh && column >= p.split && column + 32u <= p.split + kept) {
-          // one head may end and the next begin inside the piece, and keys may end and values begin
-#pragma unroll
-          for (int i = 0; i < 32; i += 2) {
-            const uint32_t at_cache = column - p.split + i;
-            if (!cached) continue;
-            const float low = dense_finish<bf16>(p, row, column + i, __uint_as_float(raw[i]));
-            const float high = dense_finish<bf16>(p, row, column + i + 1, __uint_as_float(raw[i + 1]));
-            const uint32_t first = dense_cache_offset(p.cache, at_cache), second = dense_cache_offset(p.cache, at_cache + 1u);
-            if (second == first + 1u && (((uintptr_t)(cached + first)) & 3u) == 0) {
-              *reinterpret_cast<__nv_bfloat162*>(cached + first) = __floats2bfloat162_rn(low, high);
-            } else {
-              cached[first] = __float2bfloat16_rn(low);
-              cached[second] = __float2bfloat16_rn(high);
-            }
-          }
-        } else if (p.epilogue != kDenseResidualTanh && column + 32u <= p.split && (at & 7u) == 0) {
-          uint4* target = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + at);
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            uint32_t packed[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const int e = i * 8 + j * 2;
-              const __nv_bfloat162 pair =
-                  __floats2bfloat162_rn(dense_finish<bf16>(p, row, column + e, __uint_as_float(raw[e])),
-                                        dense_finish<bf16>(p, row, column + e + 1, __uint_as_float(raw[e + 1])));
-              packed[j] = *reinterpret_cast<const uint32_t*>(&pair);
-            }
-            target[i] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
-          }
-        } else if (p.epilogue != kDenseResidualTanh && column >= p.split + kept && column + 32u <= p.n && (at32 & 3u) == 0) {
-          float4* target = reinterpret_cast<float4*>(p.out32 + at32);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            float v[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-              v[j] = dense_finish<bf16>(p, row, column + i * 4 + j, __uint_as_float(raw[i * 4 + j]));
-            target[i] = make_float4(v[0], v[1], v[2], v[3]);
-          }
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i)
-            if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
-        }
+        const uint32_t column = n0 + piece * 32u, following = piece + kEpilogueWarps / 4u;
+        Piece<STORE> held = ahead;
+        if (following < BN / 32u) ahead.fetch(p, row, rows.end, n0 + following * 32u);
+        if (row < rows.end && column < p.n) held.store(p, row, column, raw);
         __syncwarp();  // tcgen05.ld needs the whole warp
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -309,31 +349,30 @@ bool make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer
 
 // Row tiles; of rows sorted by expert, the most there can be.
 uint32_t most_tiles(const DenseProblem& p) {
-  if (!p.plan) return (p.m + kRows - 1u) / kRows;
-  return p.m / kRows + (p.experts < p.m ? p.experts : p.m);
+  if (!p.plan.tiles) return (p.m + kRows - 1u) / kRows;
+  return p.m / kRows + (p.plan.experts < p.m ? p.plan.experts : p.m);
 }
 
-template <uint32_t BN>
+template <uint32_t BN, DenseStore STORE>
 int run(const KernelArgs& args, const DenseProblem& p, uint32_t sms) {
   using S = Shape<BN>;
   CUtensorMap map_x, map_w;
   if (!make_map(&map_x, p.x, p.k, p.m, kRows) ||
-      !make_map(&map_w, p.w, p.k, (uint64_t)p.n * (p.plan ? p.experts : 1u), BN))
+      !make_map(&map_w, p.w, p.k, (uint64_t)p.n * (p.plan.tiles ? p.plan.experts : 1u), BN))
     return -1;
-  auto kernel = dense_gemm_tc_kernel<BN>;
+  auto kernel = dense_gemm_tc_kernel<BN, STORE>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSharedBytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
   }
   const uint32_t most = most_tiles(p), tiles = most * ((p.n + BN - 1u) / BN);
-  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, p, most,
+  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, DenseTask<STORE>(p), p.plan, most,
                 context_device_error(args.ctx));
   return check_launch(args);
 }
 
-}  // namespace
-
-int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& p) {
+template <DenseStore STORE>
+int run_tiles(const KernelArgs& args, const DenseProblem& p) {
   if (args.ctx == nullptr || p.k % 8u != 0 || ((uintptr_t)p.x & 15u) != 0 || ((uintptr_t)p.w & 15u) != 0) return -1;
   const uint32_t sms = (uint32_t)context_sm_count(args.ctx);
   // waves times the cost of one MMA (an MMA of up to 128 columns costs about two thirds of one of 256)
@@ -343,9 +382,20 @@ int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& p) {
     return (tiles + sms - 1u) / sms * mma;
   };
   const uint32_t wide = cost(256, 128), middle = cost(128, 85), narrow = cost(64, 80);
-  if (narrow < middle && narrow < wide) return run<64>(args, p, sms);
-  if (middle < wide) return run<128>(args, p, sms);
-  return run<256>(args, p, sms);
+  if (narrow < middle && narrow < wide) return run<64, STORE>(args, p, sms);
+  if (middle < wide) return run<128, STORE>(args, p, sms);
+  return run<256, STORE>(args, p, sms);
+}
+
+}  // namespace
+
+int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& p, DenseStore store) {
+  switch (store) {
+    case kStoreCached: return run_tiles<kStoreCached>(args, p);
+    case kStorePair: return run_tiles<kStorePair>(args, p);
+    case kStoreResidual: return run_tiles<kStoreResidual>(args, p);
+    default: return run_tiles<kStorePlain>(args, p);
+  }
 }
 
 }  // namespace llmopt

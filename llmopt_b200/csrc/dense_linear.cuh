@@ -12,59 +12,91 @@ enum DenseEpilogue : uint32_t {
   kDenseResidualTanh = 4,  // residual += tanh norm of the sum; out = the next sublayer's tanh norm of the new residual
 };
 
-// Where the key and value columns of a product go: into the cache row of their token.
-struct DenseCacheRows {
+// What a kernel does with its sums, fixed at compile time (the code of the others would cost every launch).
+enum DenseStore : uint32_t {
+  kStorePlain = 0,     // rows in T and in fp32: kDenseNone, kDenseGeluErf, kDenseTokenGate
+  kStoreCached = 1,    // the same, and key and value columns in the cache
+  kStorePair = 2,      // kDenseSiluPair
+  kStoreResidual = 3,  // kDenseResidualTanh
+};
+
+// y = scale * x . w^T (+ bias), x [m, k], w [n, k].  Columns below `split` go to `out` (T, row stride split), the next
+// cache columns (if any) to the cache, the others to `out32` (fp32): one product serves projections that are read
+// in T, that are kept, and that feed fp32 arithmetic.
+struct DenseCore {
+  const void* x;
+  const void* w;
+  uint32_t m, n, k, cluster;  // cluster: CTAs that share a tile's k-blocks, in the kernels that stream the weights
+  uint32_t split, has_bias, epilogue;
+  float scale;
+  const float* bias;  // [n], read when has_bias
+  void* out;
+  float* out32;
+  const long long* ids;  // kDenseTokenGate: token of every row
+  const void* table;     // kDenseTokenGate: T [table_rows, table_stride]
+  uint32_t table_rows, table_stride, table_offset;
+};
+
+// What only one kind of store reads.  A kernel gets no more than its own: a launch that streams few weights feels the
+// size of its parameters.
+struct DenseCacheRows {  // where the key and value columns go: the cache row of their token
   void* pool;
-  const uint32_t* slots;  // [table_rows, table_stride]
+  const uint32_t* slots;  // [slots_rows, slots_stride]
   const uint32_t* past;
   const uint32_t* sequence_rows;
   uint32_t* error_word;
   uint32_t tokens;  // rows per sequence
   uint32_t key_columns, value_columns;
   uint32_t token_stride, key_offset, value_offset;  // in elements
-  uint32_t table_stride, table_rows, pool_rows;
+  uint32_t slots_stride, slots_rows, pool_rows;
+};
+struct DenseRowScale {
+  const float* row_scale;  // per row, multiplies the input; null: none
+};
+struct DenseResidual {
+  const float* post_norm;  // norm of the sum, and of the sublayer that follows
+  const float* next_norm;
+  float* residual;  // [m, n], updated in place
 };
 
 // Rows sorted by expert, every expert with its own n rows of the weight matrix.  The plan holds the number of tiles,
 // three unused words, and {expert, first row, row end, unused} per tile of at most kExpertTile rows.
 constexpr uint32_t kExpertTile = 128;
+struct DensePlan {
+  const uint32_t* tiles;  // null: one matrix for all rows
+  uint32_t experts;
+};
 struct DenseTile {
   uint32_t expert, first, end;
 };
-
-// y = scale * x . w^T (+ bias), x [m, k], w [n, k].  Columns below `split` go to `out` (T, row stride split), the next
-// cache columns (if any) to the cache, the others to `out32` (fp32): one product serves projections that are read
-// in T, that are kept, and that feed fp32 arithmetic.
-struct DenseProblem {
-  const void* x;
-  const void* w;
-  const float* bias;  // [n], read when has_bias
-  void* out;
-  float* out32;
-  const long long* ids;  // kDenseTokenGate: token of every row
-  const void* table;     // kDenseTokenGate: T [table_rows, table_stride]
-  uint32_t m, n, k, split, has_bias, epilogue, table_rows, table_stride, table_offset;
-  float scale;
-  const float* post_norm;  // kDenseResidualTanh: norm of the sum, and of the sublayer that follows
-  const float* next_norm;
-  float* residual;  // kDenseResidualTanh: [m, n], updated in place
-  DenseCacheRows cache;
-  const uint32_t* plan;    // rows sorted by expert; null: one matrix for all rows
-  const float* row_scale;  // per row, multiplies the input; null: none
-  uint32_t experts;
-};
-
-__host__ __device__ __forceinline__ uint32_t dense_cache_columns(const DenseProblem& p) {
-  return p.cache.key_columns + p.cache.value_columns;
-}
-
-__device__ __forceinline__ DenseTile dense_tile(const DenseProblem& p, uint32_t index) {
-  const uint4 entry = reinterpret_cast<const uint4*>(p.plan)[1 + index];
+__device__ __forceinline__ DenseTile dense_tile(const DensePlan& plan, uint32_t index) {
+  const uint4 entry = reinterpret_cast<const uint4*>(plan.tiles)[1 + index];
   return {entry.x, entry.y, entry.z};
 }
 
+// What a launch is described by, and what its kernel takes of that.
+struct DenseProblem : DenseCore, DenseCacheRows, DenseRowScale, DenseResidual {
+  DensePlan plan;
+};
+template <DenseStore STORE>
+struct DenseTask : DenseCore {
+  explicit DenseTask(const DenseProblem& p) : DenseCore(p) {}
+};
+template <>
+struct DenseTask<kStoreCached> : DenseCore, DenseCacheRows {
+  explicit DenseTask(const DenseProblem& p) : DenseCore(p), DenseCacheRows(p) {}
+};
+template <>
+struct DenseTask<kStorePair> : DenseCore, DenseRowScale {
+  explicit DenseTask(const DenseProblem& p) : DenseCore(p), DenseRowScale(p) {}
+};
+template <>
+struct DenseTask<kStoreResidual> : DenseCore, DenseResidual {
+  explicit DenseTask(const DenseProblem& p) : DenseCore(p), DenseResidual(p) {}
+};
+
 template <typename T>
-__device__ __forceinline__ float dense_finish(const DenseProblem& p, uint32_t row, uint32_t column, float value) {
+__device__ __forceinline__ float dense_finish(const DenseCore& p, uint32_t row, uint32_t column, float value) {
   value *= p.scale;
   if (p.has_bias) value += __ldg(p.bias + column);
   if (p.epilogue == kDenseGeluErf) {
@@ -76,14 +108,16 @@ __device__ __forceinline__ float dense_finish(const DenseProblem& p, uint32_t ro
   }
   return value;
 }
+__device__ __forceinline__ float dense_biased(const DenseCore& p, uint32_t column, float value) {
+  return p.has_bias ? value + __ldg(p.bias + column) : value;
+}
 
 // Cache row of the row's token; null (and the error word raised) when there is none.
 template <typename T>
-__device__ __forceinline__ T* dense_cache_row(const DenseProblem& p, uint32_t row) {
-  const DenseCacheRows& c = p.cache;
+__device__ __forceinline__ T* dense_cache_row(const DenseCacheRows& c, uint32_t row) {
   const uint32_t sequence = row / c.tokens, position = c.past[sequence] + row % c.tokens, table_row = c.sequence_rows[sequence];
   uint32_t slot = c.pool_rows;
-  if (table_row < c.table_rows && position < c.table_stride) slot = c.slots[(size_t)table_row * c.table_stride + position];
+  if (table_row < c.slots_rows && position < c.slots_stride) slot = c.slots[(size_t)table_row * c.slots_stride + position];
   if (slot < c.pool_rows) return reinterpret_cast<T*>(c.pool) + (size_t)slot * c.token_stride;
   if (c.error_word) atomicExch(c.error_word, 1u);
   return nullptr;
@@ -92,45 +126,56 @@ __device__ __forceinline__ T* dense_cache_row(const DenseProblem& p, uint32_t ro
 __device__ __forceinline__ uint32_t dense_cache_offset(const DenseCacheRows& c, uint32_t at) {
   return at < c.key_columns ? c.key_offset + at : c.value_offset + at - c.key_columns;
 }
+// Columns that go to the cache.
+template <DenseStore STORE>
+__device__ __forceinline__ uint32_t dense_kept(const DenseTask<STORE>& p) {
+  if constexpr (STORE == kStoreCached) return p.key_columns + p.value_columns;
+  else return 0u;
+}
 
-template <typename T>
-__device__ __forceinline__ void dense_store(const DenseProblem& p, uint32_t row, uint32_t column, float value) {
-  value = dense_finish<T>(p, row, column, value);
-  if (p.epilogue == kDenseResidualTanh) {
+template <typename T, DenseStore STORE>
+__device__ __forceinline__ void dense_store(const DenseTask<STORE>& p, uint32_t row, uint32_t column, float value) {
+  if constexpr (STORE == kStoreResidual) {
     const size_t at = (size_t)row * p.n + column;
-    const float x = p.residual[at] + TanhNorm(p.post_norm, p.n)(value, column);
+    const float x = p.residual[at] + TanhNorm(p.post_norm, p.n)(dense_biased(p, column, value), column);
     p.residual[at] = x;
     reinterpret_cast<T*>(p.out)[at] = from_float<T>(TanhNorm(p.next_norm, p.n)(x, column));
-    return;
-  }
-  const uint32_t kept = dense_cache_columns(p);
-  if (column < p.split) {
-    reinterpret_cast<T*>(p.out)[(size_t)row * p.split + column] = from_float<T>(value);
-  } else if (column < p.split + kept) {
-    T* const cached = dense_cache_row<T>(p, row);
-    if (cached) cached[dense_cache_offset(p.cache, column - p.split)] = from_float<T>(value);
   } else {
+    value = STORE == kStoreCached ? dense_biased(p, column, value) : dense_finish<T>(p, row, column, value);
+    const uint32_t kept = dense_kept(p);
+    if (column < p.split) {
+      reinterpret_cast<T*>(p.out)[(size_t)row * p.split + column] = from_float<T>(value);
+      return;
+    }
+    if constexpr (STORE == kStoreCached) {
+      if (column < p.split + kept) {
+        T* const cached = dense_cache_row<T>(p, row);
+        if (cached) cached[dense_cache_offset(p, column - p.split)] = from_float<T>(value);
+        return;
+      }
+    }
     p.out32[(size_t)row * (p.n - p.split - kept) + (column - p.split - kept)] = value;
   }
 }
 
 // kDenseSiluPair: `column` is even; the row's scale (of its input) is linear in both sums.
-__device__ __forceinline__ float dense_pair(const DenseProblem& p, uint32_t row, uint32_t column, float gate, float value) {
+__device__ __forceinline__ float dense_pair(const DenseTask<kStorePair>& p, uint32_t row, uint32_t column, float gate, float value) {
   const float scale = p.row_scale ? p.scale * p.row_scale[row] : p.scale;
   gate *= scale, value *= scale;
   if (p.has_bias) gate += __ldg(p.bias + column), value += __ldg(p.bias + column + 1u);
   return silu_f32(gate) * value;
 }
 template <typename T>
-__device__ __forceinline__ void dense_store_pair(const DenseProblem& p, uint32_t row, uint32_t column, float gate, float value) {
+__device__ __forceinline__ void dense_store_pair(const DenseTask<kStorePair>& p, uint32_t row, uint32_t column, float gate,
+                                                 float value) {
   reinterpret_cast<T*>(p.out)[(size_t)row * (p.n / 2u) + column / 2u] = from_float<T>(dense_pair(p, row, column, gate, value));
 }
 
 // Prompt rows on tcgen05 (bf16); -1 when the shape or the pointers are outside its domain.
-int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& problem);
+int launch_dense_gemm_tc(const KernelArgs& args, const DenseProblem& problem, DenseStore store);
 
 // Rows of at most `tiles` tiles of a plan, each with its expert's matrix.
 template <typename T>
-int run_expert_rows(const KernelArgs& args, const DenseProblem& problem, uint32_t tiles);
+int run_expert_rows(const KernelArgs& args, const DenseProblem& problem, DenseStore store, uint32_t tiles);
 
 }  // namespace llmopt

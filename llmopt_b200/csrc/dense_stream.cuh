@@ -37,65 +37,61 @@ __device__ __forceinline__ void stream_fetch(uint4 (&stage)[4], const bf16* w_lo
   }
 }
 
-// sum += the k-block of the weights times the same k of the first `rows` rows of x [rows, width].
-template <int NT>
-__device__ __forceinline__ void stream_block(float (&sum)[NT][4], const uint4 (&stage)[4], const bf16* x, uint32_t rows,
-                                             uint32_t width, uint32_t block) {
-  const uint32_t lane = threadIdx.x & 31u, g = lane >> 2, t = lane & 3u;
-#pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const uint32_t k = block * 64u + half * 32u + t * 8u;
-    const uint4 low = stage[half], high = stage[2 + half];
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const uint32_t row = nt * 8u + g;
-      const uint4 b = (row < rows && k < width) ? *reinterpret_cast<const uint4*>(x + (size_t)row * width + k)
-                                                : make_uint4(0u, 0u, 0u, 0u);
-      mma_bf16(sum[nt], low.x, high.x, low.y, high.y, b.x, b.y);
-      mma_bf16(sum[nt], low.z, high.z, low.w, high.w, b.z, b.w);
-    }
-  }
+// sum += a half (32 k) of a k-block of the weights times the same k of a tile's rows.
+__device__ __forceinline__ void stream_multiply(float (&sum)[4], const uint4& low, const uint4& high, const uint4& x) {
+  mma_bf16(sum, low.x, high.x, low.y, high.y, x.x, x.y);
+  mma_bf16(sum, low.z, high.z, low.w, high.w, x.z, x.w);
 }
 
-// Adds the warps' sums of the 16 columns from n0 on (and those of the cluster's CTAs) and stores them.
+// A warp's sums, [activation row][weight row].
 template <int NT>
-__device__ __forceinline__ void stream_finish(const DenseProblem& p, const float (&sum)[NT][4],
-                                              float (&partial)[kGemvWarps][NT * 8][17], uint32_t n0, uint32_t rank,
-                                              uint32_t cluster) {
-  const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, g = lane >> 2, t = lane & 3u;
-  const uint32_t stride = kGemvWarps * cluster;
+__device__ __forceinline__ void stream_collect(const float (&sum)[NT][4], float (&mine)[NT * 8][17]) {
+  const uint32_t lane = threadIdx.x & 31u, g = lane >> 2, t = lane & 3u;
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) partial[warp][nt * 8 + 2 * t + (i & 1)][g + (i >> 1) * 8] = sum[nt][i];
+    for (int i = 0; i < 4; ++i) mine[nt * 8 + 2 * t + (i & 1)][g + (i >> 1) * 8] = sum[nt][i];
+}
+
+template <DenseStore STORE, int N>
+__device__ __forceinline__ void stream_store(const DenseTask<STORE>& p, uint32_t row, uint32_t column, const float (&value)[N]) {
+  if constexpr (STORE == kStorePair) dense_store_pair<bf16>(p, row, column, value[0], value[N - 1]);
+  else dense_store<bf16>(p, row, column, value[0]);
+}
+
+// Adds the warps' sums of the 16 columns from n0 on (and those of the cluster's CTAs) and stores them.
+template <int NT, DenseStore STORE>
+__device__ __forceinline__ void stream_finish(const DenseTask<STORE>& p, float (&partial)[kGemvWarps][NT * 8][17], uint32_t n0,
+                                              uint32_t rank, uint32_t cluster) {
+  const uint32_t stride = kGemvWarps * cluster;
   __syncthreads();
-  const bool pairs = p.epilogue == kDenseSiluPair;  // the even column of a pair stores for both
-  auto own_total = [&](uint32_t row, uint32_t column) {
-    float value = 0.0f;
-#pragma unroll
-    for (int part = 0; part < kGemvWarps; ++part) value += partial[part][row][column];
-    return value;
-  };
-  for (uint32_t index = threadIdx.x; index < NT * 8u * 16u; index += kGemvWarps * 32) {
+  constexpr uint32_t kStep = STORE == kStorePair ? 2u : 1u;  // columns a thread stores together
+  for (uint32_t index = threadIdx.x * kStep; index < NT * 8u * 16u; index += kGemvWarps * 32 * kStep) {
     const uint32_t column = index & 15u, row = index >> 4;
     if (row >= p.m || n0 + column >= p.n) continue;
-    if (cluster > 1u) partial[0][row][column] = own_total(row, column);  // read and written by this thread only
-    else if (!pairs) dense_store<bf16>(p, row, n0 + column, own_total(row, column));
-    else if ((column & 1u) == 0u) dense_store_pair<bf16>(p, row, n0 + column, own_total(row, column), own_total(row, column + 1u));
+    float value[kStep];
+#pragma unroll
+    for (uint32_t i = 0; i < kStep; ++i) {
+      value[i] = 0.0f;
+#pragma unroll
+      for (int part = 0; part < kGemvWarps; ++part) value[i] += partial[part][row][column + i];
+      if (cluster > 1u) partial[0][row][column + i] = value[i];  // read and written by this thread only
+    }
+    if (cluster == 1u) stream_store(p, row, n0 + column, value);
   }
   if (cluster == 1u) return;
   cluster_sync();
   // the cluster's CTAs share out the outputs; sums in rank order
-  auto total = [&](uint32_t row, uint32_t column) {
-    float value = 0.0f;
-    for (uint32_t other = 0; other < cluster; ++other) value += cluster_load(&partial[0][row][column], other);
-    return value;
-  };
-  for (uint32_t index = rank * kGemvWarps * 32 + threadIdx.x; index < NT * 8u * 16u; index += stride * 32u) {
+  for (uint32_t index = (rank * kGemvWarps * 32 + threadIdx.x) * kStep; index < NT * 8u * 16u; index += stride * 32u * kStep) {
     const uint32_t column = index & 15u, row = index >> 4;
     if (row >= p.m || n0 + column >= p.n) continue;
-    if (!pairs) dense_store<bf16>(p, row, n0 + column, total(row, column));
-    else if ((column & 1u) == 0u) dense_store_pair<bf16>(p, row, n0 + column, total(row, column), total(row, column + 1u));
+    float value[kStep];
+#pragma unroll
+    for (uint32_t i = 0; i < kStep; ++i) {
+      value[i] = 0.0f;
+      for (uint32_t other = 0; other < cluster; ++other) value[i] += cluster_load(&partial[0][row][column + i], other);
+    }
+    stream_store(p, row, n0 + column, value);
   }
   cluster_sync();  // nobody leaves while its sums may be read
 }

@@ -33,10 +33,12 @@ struct RowAttentionParams {
   uint32_t window, keep_first; // 0: no window
   uint32_t query_stride, query_column, gate_stride, gate_column;  // in elements; gate_stride 0: no gate
   uint32_t weights32;  // softmax weights meet the values in 32 bits (two bfloat16 parts), not rounded to bfloat16
+  bool extended() const { return weights32 || window || softcap > 0.0f || gate_stride; }
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kLowest = -1.0e30f;
+constexpr float kBoundedCap = 40.0f;  // e^40 and e^-40, and sums of many of them, are ordinary fp32 numbers
 
 struct KeyRows {  // rows of one sequence
   const uint32_t* slots;
@@ -54,25 +56,29 @@ __device__ __forceinline__ KeyRows key_rows(const RowAttentionParams& p, const u
   return {table + (present ? (size_t)row * p.table_stride : 0u), present ? p.table_stride : 0u, p.pool_rows};
 }
 
+// EXTENDED kernels know windows, caps and gates, and keep the softmax weights in 32 bits; the others compile without.
+
 // The keys a run of rows sees, positions first .. last of them: the kept ones, then those from `begin` on.
+template <bool EXTENDED>
 struct Visible {
   uint32_t kept, begin, end;
   __device__ __forceinline__ Visible(const RowAttentionParams& p, uint32_t first, uint32_t last) {
     end = last + 1u;
-    begin = p.window && first + 1u > p.window ? first + 1u - p.window : 0u;
-    kept = p.window ? min(p.keep_first, begin) : 0u;
+    begin = EXTENDED && p.window && first + 1u > p.window ? first + 1u - p.window : 0u;
+    kept = EXTENDED && p.window ? min(p.keep_first, begin) : 0u;
   }
   __device__ __forceinline__ uint32_t count() const { return kept + end - begin; }
   __device__ __forceinline__ uint32_t position(uint32_t index) const { return index < kept ? index : index - kept + begin; }
 };
+template <bool EXTENDED>
 __device__ __forceinline__ bool sees(const RowAttentionParams& p, uint32_t position, uint32_t key) {
-  return key <= position && (!p.window || position - key < p.window || key < p.keep_first);
+  return key <= position && (!EXTENDED || !p.window || position - key < p.window || key < p.keep_first);
 }
 
 // Factor of a read-out.
-template <typename T>
+template <bool EXTENDED, typename T>
 __device__ __forceinline__ float gate_of(const RowAttentionParams& p, const T* gate, size_t row, uint32_t head, uint32_t column) {
-  return p.gate_stride ? sigmoid_f32(as_float(gate[row * p.gate_stride + p.gate_column + head * p.vdim + column])) : 1.0f;
+  return EXTENDED && p.gate_stride ? sigmoid_f32(as_float(gate[row * p.gate_stride + p.gate_column + head * p.vdim + column])) : 1.0f;
 }
 
 // ---- one warp per (row, head) --------------------------------------------------------------------
@@ -86,7 +92,7 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(const T* query, con
   const uint32_t row = item / p.heads, head = item % p.heads, sequence = row / p.tokens;
   const uint32_t kv_head = head / (p.heads / p.kv_heads);
   const uint32_t position = past[sequence] + row % p.tokens;
-  const Visible visible(p, position, position);
+  const Visible<true> visible(p, position, position);
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
   float q[SEGMENTS], o[SEGMENTS];
 #pragma unroll
@@ -120,7 +126,7 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(const T* query, con
 #pragma unroll
   for (int s = 0; s < SEGMENTS; ++s) {
     const uint32_t c = lane + s * 32u;
-    if (c < p.vdim) out[(size_t)item * p.vdim + c] = from_float<T>(o[s] / total * gate_of(p, gate, row, head, c));
+    if (c < p.vdim) out[(size_t)item * p.vdim + c] = from_float<T>(o[s] / total * gate_of<true>(p, gate, row, head, c));
   }
 }
 
@@ -157,19 +163,21 @@ __host__ __device__ constexpr uint32_t round16(uint32_t v) { return (v + 15u) & 
 
 // Online softmax of one warp's 16 rows (this lane: rows r and r + 8) over KEYS keys, scores already in units
 // of log2 e with invisible ones at -inf; then O += P V from the value tile at `v_tile` (row stride v_stride).
-// FINE: P enters the product as its bfloat16 rounding plus the bfloat16 rounding of what that leaves.
-template <int KEYS, int DV, bool FINE>
+// EXTENDED: P enters the product as its bfloat16 rounding plus the bfloat16 rounding of what that leaves.
+template <int KEYS, int DV, bool EXTENDED>
 struct Softmax {
   float top[2], total[2], out[DV / 8][4];
-  __device__ __forceinline__ void reset() {
-    top[0] = top[1] = kLowest;
+  bool bounded;  // capped scores: no maximum has to be taken off
+  __device__ __forceinline__ explicit Softmax(const RowAttentionParams& p)
+      : bounded(EXTENDED && p.softcap > 0.0f && p.softcap <= kBoundedCap) {
+    top[0] = top[1] = bounded ? 0.0f : kLowest;
     total[0] = total[1] = 0.0f;
 #pragma unroll
     for (int t = 0; t < DV / 8; ++t)
 #pragma unroll
       for (int i = 0; i < 4; ++i) out[t][i] = 0.0f;
   }
-  __device__ __forceinline__ void absorb(float (&score)[KEYS / 8][4], const bf16* v_tile, uint32_t v_stride, uint32_t lane) {
+  __device__ __forceinline__ void raise_maximum(const float (&score)[KEYS / 8][4]) {
     float next[2] = {top[0], top[1]};
 #pragma unroll
     for (int j = 0; j < KEYS / 8; ++j)
@@ -188,7 +196,10 @@ struct Softmax {
         out[t][2 * h + 1] *= keep;
       }
     }
-    uint32_t weights[KEYS / 16][4], rests[FINE ? KEYS / 16 : 1][4];
+  }
+  __device__ __forceinline__ void absorb(float (&score)[KEYS / 8][4], const bf16* v_tile, uint32_t v_stride, uint32_t lane) {
+    if (!bounded) raise_maximum(score);
+    uint32_t weights[KEYS / 16][4], rests[EXTENDED ? KEYS / 16 : 1][4];
 #pragma unroll
     for (int j = 0; j < KEYS / 8; ++j) {
       float e[4];
@@ -199,11 +210,11 @@ struct Softmax {
       const __nv_bfloat162 low = __floats2bfloat162_rn(e[0], e[1]), high = __floats2bfloat162_rn(e[2], e[3]);
       weights[j >> 1][(j & 1) * 2] = *reinterpret_cast<const uint32_t*>(&low);
       weights[j >> 1][(j & 1) * 2 + 1] = *reinterpret_cast<const uint32_t*>(&high);
-      if (FINE) {
+      if (EXTENDED) {
         const __nv_bfloat162 low_rest = __floats2bfloat162_rn(e[0] - __low2float(low), e[1] - __high2float(low));
         const __nv_bfloat162 high_rest = __floats2bfloat162_rn(e[2] - __low2float(high), e[3] - __high2float(high));
-        rests[FINE ? j >> 1 : 0][(j & 1) * 2] = *reinterpret_cast<const uint32_t*>(&low_rest);
-        rests[FINE ? j >> 1 : 0][(j & 1) * 2 + 1] = *reinterpret_cast<const uint32_t*>(&high_rest);
+        rests[EXTENDED ? j >> 1 : 0][(j & 1) * 2] = *reinterpret_cast<const uint32_t*>(&low_rest);
+        rests[EXTENDED ? j >> 1 : 0][(j & 1) * 2 + 1] = *reinterpret_cast<const uint32_t*>(&high_rest);
       }
     }
 #pragma unroll
@@ -214,22 +225,23 @@ struct Softmax {
         ldmatrix_x4_trans(b, v_tile + (16 * s + (lane & 7u) + ((lane >> 3) & 1u) * 8u) * v_stride + 16 * t + (lane >> 4) * 8u);
         mma_bf16(out[2 * t], weights[s], b[0], b[1]);
         mma_bf16(out[2 * t + 1], weights[s], b[2], b[3]);
-        if (FINE) {
-          mma_bf16(out[2 * t], rests[FINE ? s : 0], b[0], b[1]);
-          mma_bf16(out[2 * t + 1], rests[FINE ? s : 0], b[2], b[3]);
+        if (EXTENDED) {
+          mma_bf16(out[2 * t], rests[EXTENDED ? s : 0], b[0], b[1]);
+          mma_bf16(out[2 * t + 1], rests[EXTENDED ? s : 0], b[2], b[3]);
         }
       }
   }
 };
 
-// A raw score in units of log2 e.
+// A raw score in units of log2 e; with a cap c, c tanh(s / c) = c - 2 c / (e^(2 s / c) + 1).
+template <bool EXTENDED>
 struct ScoreScale {
   float scale, cap;  // cap 0: none
   __device__ __forceinline__ explicit ScoreScale(const RowAttentionParams& p)
-      : scale(p.softcap > 0.0f ? p.scale / p.softcap : p.scale * kLog2e), cap(p.softcap * kLog2e) {}
+      : scale((EXTENDED && p.softcap > 0.0f ? p.scale / p.softcap * 2.0f : p.scale) * kLog2e), cap(p.softcap * kLog2e) {}
   __device__ __forceinline__ float operator()(float raw) const {
     const float score = raw * scale;
-    return cap > 0.0f ? cap * tanh_f32(score) : score;
+    return EXTENDED && cap > 0.0f ? fmaf(-2.0f * cap, __fdividef(1.0f, exp2_approx(score) + 1.0f), cap) : score;
   }
 };
 
@@ -266,7 +278,7 @@ __device__ __forceinline__ void scores(float (&score)[KEYS / 8][4], const uint32
 // ---- prompts -------------------------------------------------------------------------------------
 constexpr uint32_t kQueryTile = 64, kKeyTile = 64;
 
-template <int DK, int DV, bool FINE>
+template <int DK, int DV, bool EXTENDED>
 __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
                                                                const uint32_t* past_lengths, const uint32_t* sequence_rows,
                                                                bf16* out, const bf16* gate, RowAttentionParams p, uint32_t* error_word) {
@@ -284,7 +296,7 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
   const uint32_t key_end = past + min(q0 + kQueryTile, p.tokens);
   // whole key tiles: those with kept keys, then from the first row's window on
-  const Visible visible(p, past + q0, key_end - 1u);
+  const Visible<EXTENDED> visible(p, past + q0, key_end - 1u);
   const uint32_t kept_tiles = (visible.kept + kKeyTile - 1u) / kKeyTile;
   const uint32_t skipped = max(visible.begin / kKeyTile, kept_tiles) - kept_tiles;
   const uint32_t tiles = (key_end + kKeyTile - 1u) / kKeyTile - skipped;
@@ -330,9 +342,8 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
       ldmatrix_x4(q_frag[s], q_rows + ((lane & 7u) + ((lane >> 3) & 1u) * 8u) * k_stride + 16 * s + (lane >> 4) * 8u);
   }
   const uint32_t row_low = q0 + warp * 16u + r;  // and row_low + 8
-  const ScoreScale score_of(p);
-  Softmax<kKeyTile, DV, FINE> state;
-  state.reset();
+  const ScoreScale<EXTENDED> score_of(p);
+  Softmax<kKeyTile, DV, EXTENDED> state(p);
 
   for (uint32_t tile = 0; tile < tiles; ++tile) {
     const uint32_t k0 = first_key(tile);
@@ -343,13 +354,13 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
     scores<kKeyTile, DK>(score, q_frag, q_rows, k_tiles + (tile & 1u) * kKeyTile * k_stride, k_stride, padded / 16u, lane);
     const uint32_t first_row = past + q0 + warp * 16u;  // of this warp
     const bool all_visible = k0 + kKeyTile - 1u <= first_row &&
-                             (!p.window || first_row + 15u - k0 < p.window || k0 + kKeyTile <= p.keep_first);
+                             (!EXTENDED || !p.window || first_row + 15u - k0 < p.window || k0 + kKeyTile <= p.keep_first);
 #pragma unroll
     for (int j = 0; j < (int)kKeyTile / 8; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const uint32_t token = row_low + ((i & 2) ? 8u : 0u), key = k0 + 8u * j + 2u * c + (i & 1);
-        score[j][i] = all_visible || sees(p, past + token, key) ? score_of(score[j][i]) : -INFINITY;
+        score[j][i] = all_visible || sees<EXTENDED>(p, past + token, key) ? score_of(score[j][i]) : -INFINITY;
       }
     state.absorb(score, v_tiles + (tile & 1u) * kKeyTile * v_stride, v_stride, lane);
     __syncthreads();  // every warp is done with this buffer before the next iteration's fetch refills it
@@ -376,8 +387,8 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
       const uint32_t column = 8u * t + 2u * c;
       if (column < p.vdim)  // vdim is a multiple of eight
         *reinterpret_cast<__nv_bfloat162*>(target + column) =
-            __floats2bfloat162_rn(state.out[t][2 * h] * scale * gate_of(p, gate, row, head, column),
-                                  state.out[t][2 * h + 1] * scale * gate_of(p, gate, row, head, column + 1u));
+            __floats2bfloat162_rn(state.out[t][2 * h] * scale * gate_of<EXTENDED>(p, gate, row, head, column),
+                                  state.out[t][2 * h + 1] * scale * gate_of<EXTENDED>(p, gate, row, head, column + 1u));
     }
   }
 }
@@ -389,7 +400,7 @@ constexpr uint32_t kWarpKeys = 16, kDecodeWarps = 4, kDecodeStages = 3, kMostSpl
 template <int DV>
 __host__ __device__ constexpr uint32_t record_floats() { return 32u + 16u * DV; }
 
-template <int DK, int DV, bool FINE>
+template <int DK, int DV, bool EXTENDED>
 __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
                                                                const uint32_t* past_lengths, const uint32_t* sequence_rows,
                                                                bf16* out, const bf16* gate, uint32_t* counters, float* records,
@@ -404,7 +415,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
   const uint32_t split = blockIdx.x, kv_head = blockIdx.y, sequence = blockIdx.z;
   const uint32_t group = p.heads / p.kv_heads, query_rows = p.tokens * group;
   const uint32_t past = past_lengths[sequence];
-  const Visible visible(p, past, past + p.tokens - 1u);
+  const Visible<EXTENDED> visible(p, past, past + p.tokens - 1u);
   const uint32_t keys = visible.count();
   const KeyRows rows = key_rows(p, table, sequence_rows[sequence]);
   // whole 64-key stretches per split
@@ -452,9 +463,8 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
       ldmatrix_x4(q_frag[s], q_tile + ((lane & 7u) + ((lane >> 3) & 1u) * 8u) * k_stride + 16 * s + (lane >> 4) * 8u);
   }
   const uint32_t token_low = r / group, token_high = (r + 8u) / group;
-  const ScoreScale score_of(p);
-  Softmax<kWarpKeys, DV, FINE> state;
-  state.reset();
+  const ScoreScale<EXTENDED> score_of(p);
+  Softmax<kWarpKeys, DV, EXTENDED> state(p);
   for (uint32_t tile = 0; tile < tiles; ++tile) {
     fetch_tile(tile + kDecodeStages - 1u);
     asm volatile("cp.async.wait_group %0;" ::"n"(kDecodeStages - 1) : "memory");
@@ -468,7 +478,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const uint32_t index = k0 + 8u * j + 2u * c + (i & 1);
-        const bool seen = index < end && sees(p, past + ((i & 2) ? token_high : token_low), visible.position(index));
+        const bool seen = index < end && sees<EXTENDED>(p, past + ((i & 2) ? token_high : token_low), visible.position(index));
         score[j][i] = seen ? score_of(score[j][i]) : -INFINITY;
       }
     state.absorb(score, k_tile + kWarpKeys * k_stride, v_stride, lane);
@@ -523,7 +533,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
       const uint32_t head = kv_head * group + row % group;
       if (column < p.vdim)
         out[(token * p.heads + head) * p.vdim + column] =
-            __float2bfloat16_rn(sum / total * gate_of(p, gate, token, head, column));
+            __float2bfloat16_rn(sum / total * gate_of<EXTENDED>(p, gate, token, head, column));
     } else {
       record[32 + row * DV + column] = sum;
       if (column == 0) {
@@ -595,10 +605,10 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const bf16* query
     if (column < p.vdim) {  // vdim is a multiple of eight
       const size_t token = (size_t)sequence * p.tokens + row / group;
       const uint32_t head = kv_head * group + row % group;
-      sum.x *= gate_of(p, gate, token, head, column);
-      sum.y *= gate_of(p, gate, token, head, column + 1u);
-      sum.z *= gate_of(p, gate, token, head, column + 2u);
-      sum.w *= gate_of(p, gate, token, head, column + 3u);
+      sum.x *= gate_of<EXTENDED>(p, gate, token, head, column);
+      sum.y *= gate_of<EXTENDED>(p, gate, token, head, column + 1u);
+      sum.z *= gate_of<EXTENDED>(p, gate, token, head, column + 2u);
+      sum.w *= gate_of<EXTENDED>(p, gate, token, head, column + 3u);
       store_four(out + (token * p.heads + head) * p.vdim + column, sum);
     }
   }
@@ -622,11 +632,11 @@ int run_rows(const KernelArgs& args, const RowAttentionParams& p) {
   return check_launch(args);
 }
 
-template <int DK, int DV, bool FINE>
+template <int DK, int DV, bool EXTENDED>
 int run_prompt(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t padded = DK > 0 ? DK : round16(p.dim);
   const uint32_t bytes = ((kQueryTile + 2u * kKeyTile) * (padded + 8u) + 2u * kKeyTile * (DV + 8u)) * 2u;
-  auto kernel = attention_prompt_kernel<DK, DV, FINE>;
+  auto kernel = attention_prompt_kernel<DK, DV, EXTENDED>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
@@ -639,7 +649,7 @@ int run_prompt(const KernelArgs& args, const RowAttentionParams& p) {
   return check_launch(args);
 }
 
-template <int DK, int DV, bool FINE>
+template <int DK, int DV, bool EXTENDED>
 int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t padded = DK > 0 ? DK : round16(p.dim);
   uint32_t bytes = (16u * (padded + 8u) + kDecodeWarps * kDecodeStages * kWarpKeys * (padded + 8u + DV + 8u)) * 2u;
@@ -649,7 +659,7 @@ int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
   LLMOPT_REQUIRE(p.splits <= kMostSplits, "at most 64 splits");
   LLMOPT_REQUIRE(p.splits == 1u || args.lengths[6] >= counters + heads * p.splits * record_floats<DV>() * 4,
                  "split scratch is too short");
-  auto kernel = attention_decode_kernel<DK, DV, FINE>;
+  auto kernel = attention_decode_kernel<DK, DV, EXTENDED>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
     cudaGetLastError();
     return -1;
@@ -665,8 +675,8 @@ int run_decode(const KernelArgs& args, const RowAttentionParams& p) {
 template <int DK, int DV>
 int run_tensor(const KernelArgs& args, const RowAttentionParams& p) {
   if (p.tokens * (p.heads / p.kv_heads) <= 16u)
-    return p.weights32 ? run_decode<DK, DV, true>(args, p) : run_decode<DK, DV, false>(args, p);
-  return p.weights32 ? run_prompt<DK, DV, true>(args, p) : run_prompt<DK, DV, false>(args, p);
+    return p.extended() ? run_decode<DK, DV, true>(args, p) : run_decode<DK, DV, false>(args, p);
+  return p.extended() ? run_prompt<DK, DV, true>(args, p) : run_prompt<DK, DV, false>(args, p);
 }
 
 int run_tensor_shapes(const KernelArgs& args, const RowAttentionParams& p) {

@@ -29,9 +29,13 @@ class DenseFeedForward:
         step.stream.product(hidden, self.down, k=inner)
 
 
-# rows of a step whose experts' weights are streamed, every row riding along with every chosen expert
-STREAMED_ROWS = 64
+STREAMED_ROWS = 64  # most rows of a step whose experts' weights are streamed
 EXPERT_TILE = 128  # rows of a tile of sorted rows
+
+
+def route_words(rows: int, experts: int, top: int) -> int:
+    """Words of a step's route (csrc/experts.cu, ``Route``): experts, their first slots, row and score per slot."""
+    return 4 + (experts + 3) // 4 * 4 + (experts + 4) // 4 * 4 + 2 * rows * top
 
 
 class RoutedExperts:
@@ -48,7 +52,7 @@ class RoutedExperts:
     def _streams(self, step) -> bool:
         spec, engine = self.spec, step.engine
         return (engine.itemsize == 2 and step.rows <= STREAMED_ROWS and engine.config.width % 8 == 0 and spec.width % 8 == 0 and
-                spec.experts <= 1024 and (spec.experts + 2 * step.rows * spec.top) * 4 <= 48 * 1024)
+                spec.experts <= 1024 and step.rows * spec.top <= 4096 and (3 * spec.experts + 1 + 2 * step.rows * spec.top) * 4 <= 48 * 1024)
 
     def record(self, step) -> None:
         engine, spec = step.engine, self.spec
@@ -60,9 +64,8 @@ class RoutedExperts:
     def _record_streamed(self, step, logits) -> None:
         engine, spec, width = step.engine, self.spec, step.engine.config.width
         rows = min(STREAMED_ROWS, engine.max_rows)
-        most = min(spec.experts, rows * spec.top)
-        route = engine.scratch("route", (4 + (spec.experts + 3) // 4 * 4 + most * rows) * 4)
-        hidden = engine.scratch("experts_hidden", most * rows * spec.width * engine.itemsize)
+        route = engine.scratch("route", route_words(rows, spec.experts, spec.top) * 4)
+        hidden = engine.scratch("experts_hidden", rows * spec.top * spec.width * engine.itemsize)
         size = dict(rows=step.rows, experts=spec.experts, top=spec.top)
         step.run("llmopt_route_step_f32", [logits, route], parameters.route(**size))
         step.run("llmopt_expert_step_bf16", [step.stream.x, self.up, route, hidden],

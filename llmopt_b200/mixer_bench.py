@@ -154,16 +154,19 @@ def time_items(runtime, items, past: int, itemsize: int, peaks: dict) -> dict:
     """Per kernel: all its launches of the step back to back (every layer's own operands)."""
     groups = {}
     for item in items:
-        label, nbytes, flops = work_of(item, past, itemsize)
-        groups.setdefault(label, {"items": [], "bytes": nbytes, "flops": flops})["items"].append(item)
+        groups.setdefault(work_of(item, past, itemsize)[0], []).append(item)
     table = {}
     for label, group in groups.items():
-        launches = len(group["items"])
-        repeated = group["items"] * max(1, min(16, 64 // launches))
-        ms = runtime.time_dispatches(repeated, warmup=2, iterations=5)
-        floor = max(group["bytes"] / peaks["hbm_gbs"] / 1e6, group["flops"] / peaks["bf16_tflops"] / 1e9)
+        if label.startswith(("route", "expert")):
+            runtime.time_dispatches(items, warmup=0, iterations=1)  # routes of a whole step, not of what was timed before
+        launches = len(group)
+        ms = runtime.time_dispatches(group * max(1, min(16, 64 // launches)), warmup=2, iterations=5)
+        _, nbytes, flops = work_of(group[0], past, itemsize)
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e6, flops / peaks["bf16_tflops"] / 1e9)
         table[label] = {"launches": launches, "us": round(ms * 1e3, 2), "floor_us": round(floor * 1e3, 2),
                         "frac": round(floor / ms, 3) if ms else None, "share_us": round(ms * 1e3 * launches, 1)}
+        if label.startswith("expert") and "combine" not in label:
+            table[label]["experts_in_use"] = experts_in_use(group[0])
     return table
 
 
@@ -210,7 +213,6 @@ def measure_mixers(runtime, peaks: dict, config: MixerConfig, tokens: int, conte
         engine.rewind(context)
         plan.write(list(range(1, batch + 1)), [context] * batch, [engine._row(index) for index in range(batch)])
         items = [item for item in plan.items if item.name != "llmopt_advance_tokens"]
-        runtime.time_dispatches(items, warmup=0, iterations=1)  # every kernel's own inputs, the routes among them
         result["kernels"][f"decode, {batch} sequences, {context} tokens behind"] = time_items(
             runtime, items, context, engine.itemsize, peaks)
         result["decode"][-1]["kernels_per_step"] = engine._decode_plan(batch)[1].kernel_count()
@@ -218,7 +220,6 @@ def measure_mixers(runtime, peaks: dict, config: MixerConfig, tokens: int, conte
             result["prefill"] = prefill_rate(engine, tokens)
             plan = engine._prompt_plan(tokens)[0]
             plan.write(np.random.default_rng(0).integers(0, config.vocabulary, size=tokens), [0], [engine._row(0)])
-            runtime.time_dispatches(plan.items, warmup=0, iterations=1)  # every kernel's own inputs, the routes among them
             result["kernels"][f"prompt of {tokens} tokens"] = time_items(runtime, plan.items, 0, engine.itemsize, peaks)
     return result
 

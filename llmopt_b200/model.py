@@ -419,7 +419,8 @@ def mixer_tensors(config: MixerConfig) -> Dict[str, tuple]:
 def random_mixer_weights(config: MixerConfig, seed: int = 0, std: float = 0.02, fast: bool = False) -> Dict[str, np.ndarray]:
     """Random-init weights under the checkpoint's names, as bfloat16 bits; matrices N(0, std), norm weights
     near the value that leaves a vector as it is, decays of a few to a few hundred tokens.  ``fast`` draws
-    the bits of matrices directly (magnitudes 1/64 .. 1/32, for multi-GB models)."""
+    the bits of matrices directly (magnitudes 1/64 .. 1/32, for multi-GB models).  An embedding that positions are added
+    to has their magnitude, so that tokens differ and take different experts."""
     from .safetensors_archive import as_bfloat16_bits
 
     rng = np.random.default_rng(seed)
@@ -441,6 +442,8 @@ def random_mixer_weights(config: MixerConfig, seed: int = 0, std: float = 0.02, 
             value = rng.standard_normal(shape) * 0.5
         elif leaf == "b" and len(shape) == 1:
             value = rng.standard_normal(shape) * 0.1
+        elif name == "embed" and config.sinusoid:
+            value = rng.standard_normal(shape, dtype=np.float32)
         elif fast:
             bits = np.frombuffer(rng.bytes(2 * int(np.prod(shape))), np.uint16)
             weights[name] = ((bits & 0x807F) | 0x3C80).reshape(shape)

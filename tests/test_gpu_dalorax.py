@@ -405,14 +405,18 @@ def test_routes(runtime, rows, experts, top, width, inner):
     assert entries[0, 0] == len(tiles) <= most and np.array_equal(entries[1:1 + len(tiles), :3], np.array(tiles, np.uint32))
     if rows > 64:
         return
-    start = 4 + (experts + 3) // 4 * 4
-    route = upload(runtime, np.full(start + min(experts, pairs) * rows, 0x7FC00000, np.uint32))
+    from llmopt_b200.feed_forward import route_words
+
+    route = upload(runtime, np.full(route_words(rows, experts, top), 0x7FC00000, np.uint32))
     run(runtime, "llmopt_route_step_f32", [z, route], parameters.route(**size))
     words, used = route.to_numpy(np.uint32), np.nonzero(counts)[0]
+    first_at = 4 + (experts + 3) // 4 * 4
+    row_at = first_at + (experts + 4) // 4 * 4
+    score_at = row_at + pairs
     assert words[0] == len(used) and np.array_equal(words[4:4 + len(used)], used)
-    table = np.zeros((rows, experts))
-    np.put_along_axis(table, want, scores, 1)
-    close(words[start:start + len(used) * rows].view(np.float32).reshape(len(used), rows), table[:, used].T, 1e-6)
+    assert np.array_equal(words[first_at:first_at + len(used) + 1], np.concatenate([[0], np.cumsum(counts[used])]))
+    assert np.array_equal(words[row_at:row_at + pairs], order // top)
+    close(words[score_at:score_at + pairs].view(np.float32), scores.reshape(-1)[order], 1e-6)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
