@@ -276,12 +276,17 @@ __device__ __forceinline__ void scores(float (&score)[KEYS / 8][4], const uint32
 }
 
 // ---- prompts -------------------------------------------------------------------------------------
-constexpr uint32_t kQueryTile = 64, kKeyTile = 64;
+constexpr uint32_t kQueryTile = 64;
+// Keys per tile, and CTAs per SM to compile for (0: no bound): with smaller tiles a third CTA fits, which hides more of the
+// longer way from a score to its weight.
+__host__ __device__ constexpr uint32_t key_tile(int DK, bool EXTENDED) { return EXTENDED && DK == 128 ? 32u : 64u; }
+constexpr int prompt_ctas(int DK, bool EXTENDED) { return DK != 128 ? 0 : EXTENDED ? 3 : 2; }
 
 template <int DK, int DV, bool EXTENDED>
-__global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
+__global__ void __launch_bounds__(128, prompt_ctas(DK, EXTENDED)) attention_prompt_kernel(const bf16* query, const bf16* pool, const uint32_t* table,
                                                                const uint32_t* past_lengths, const uint32_t* sequence_rows,
                                                                bf16* out, const bf16* gate, RowAttentionParams p, uint32_t* error_word) {
+  constexpr uint32_t kKeyTile = key_tile(DK, EXTENDED), kPerKey = 128u / kKeyTile;  // threads that fetch a key
   grid_chain_prologue();
   extern __shared__ __align__(16) unsigned char attention_shared[];
   const uint32_t padded = DK > 0 ? DK : round16(p.dim), k_stride = padded + 8u, v_stride = DV + 8u;
@@ -307,17 +312,17 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const bf16* query
     if (tile < tiles) {
       bf16* k_tile = k_tiles + (tile & 1u) * kKeyTile * k_stride;
       bf16* v_tile = v_tiles + (tile & 1u) * kKeyTile * v_stride;
-      // two threads per key row: one slot look-up, half of the chunks each
-      const uint32_t key = threadIdx.x >> 1, half = threadIdx.x & 1u, position = first_key(tile) + key;
+      // a few threads per key row: one slot look-up, a share of the chunks each
+      const uint32_t key = threadIdx.x / kPerKey, share = threadIdx.x % kPerKey, position = first_key(tile) + key;
       const bool present = position < key_end;
       const bf16* cached = pool + (size_t)(present ? rows(position, error_word) : 0u) * p.token_stride;
       const bf16* k = cached + p.key_offset + kv_head * p.dim;
       const bf16* v = cached + p.value_offset + kv_head * p.vdim;
-      for (uint32_t chunk = half; chunk < k_chunks; chunk += 2u) {
+      for (uint32_t chunk = share; chunk < k_chunks; chunk += kPerKey) {
         const bool there = present && chunk * 8u < p.dim;
         copy_async_16(k_tile + key * k_stride + chunk * 8u, there ? k + chunk * 8u : pool, there ? 16u : 0u);
       }
-      for (uint32_t chunk = half; chunk < v_chunks; chunk += 2u) {
+      for (uint32_t chunk = share; chunk < v_chunks; chunk += kPerKey) {
         const bool there = present && chunk * 8u < p.vdim;
         copy_async_16(v_tile + key * v_stride + chunk * 8u, there ? v + chunk * 8u : pool, there ? 16u : 0u);
       }
@@ -635,6 +640,7 @@ int run_rows(const KernelArgs& args, const RowAttentionParams& p) {
 template <int DK, int DV, bool EXTENDED>
 int run_prompt(const KernelArgs& args, const RowAttentionParams& p) {
   const uint32_t padded = DK > 0 ? DK : round16(p.dim);
+  constexpr uint32_t kKeyTile = key_tile(DK, EXTENDED);
   const uint32_t bytes = ((kQueryTile + 2u * kKeyTile) * (padded + 8u) + 2u * kKeyTile * (DV + 8u)) * 2u;
   auto kernel = attention_prompt_kernel<DK, DV, EXTENDED>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
