@@ -59,36 +59,56 @@ int launch_embedding_residual(const KernelArgs& args) {
 }
 
 // ---- embedding with absolute positions -----------------------------------------------------------
-// Columns 2i, 2i + 1 take sine and cosine of position * frequency[i].  The angle is formed and reduced to one turn in
-// double precision, so that late positions lose nothing.
+// Columns 2i, 2i + 1 take sine and cosine of a full turn times position * turns[i].  The turns are formed and reduced to
+// less than one in double precision, so that late positions lose nothing.
+__device__ __forceinline__ float2 sinusoid(double position, double turns) {
+  const double angle = position * turns;
+  float2 value;
+  sincospif(2.0f * (float)(angle - rint(angle)), &value.x, &value.y);
+  return value;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) embedding_sinusoid_kernel(const long long* ids, const T* __restrict__ table,
-                                                                 const uint32_t* past, const double* __restrict__ frequency,
+                                                                 const uint32_t* past, const double* __restrict__ turns,
                                                                  const float* __restrict__ norm, float* x, T* normed,
-                                                                 uint32_t tokens, uint32_t vocabulary, uint32_t width) {
+                                                                 uint32_t tokens, uint32_t vocabulary, uint32_t width,
+                                                                 uint32_t vectors) {
   grid_chain_prologue();
   const uint32_t row = blockIdx.y;
   const size_t token = min((unsigned long long)ids[row], (unsigned long long)(vocabulary - 1u));
   const double position = (double)(past[row / tokens] + row % tokens);
   const TanhNorm next(norm, width);
-  constexpr double kTurn = 6.283185307179586476925;
-  const uint32_t pair = blockIdx.x * 256u + threadIdx.x, column = pair * 2u;
+  const uint32_t thread = blockIdx.x * 256u + threadIdx.x;
+  if (vectors) {  // two pairs together
+    const uint32_t column = thread * 4u;
+    if (column >= width) return;
+    struct alignas(4 * sizeof(T)) Four {
+      T v[4];
+    };
+    const size_t at = (size_t)row * width + column;
+    const Four e = *reinterpret_cast<const Four*>(table + token * width + column);
+    const float2 low = sinusoid(position, turns[column / 2u]), high = sinusoid(position, turns[column / 2u + 1u]);
+    const float4 sum = make_float4(as_float(e.v[0]) + low.x, as_float(e.v[1]) + low.y, as_float(e.v[2]) + high.x, as_float(e.v[3]) + high.y);
+    *reinterpret_cast<float4*>(x + at) = sum;
+    store_four(normed + at, next.four(sum, column));
+    return;
+  }
+  const uint32_t column = thread * 2u;
   if (column >= width) return;
-  const double angle = position * frequency[pair];
-  float sine, cosine;
-  sincosf((float)(angle - kTurn * rint(angle / kTurn)), &sine, &cosine);
   const size_t at = (size_t)row * width + column;
-  const float first = as_float(table[token * width + column]) + sine;
+  const float2 pair = sinusoid(position, turns[thread]);
+  const float first = as_float(table[token * width + column]) + pair.x;
   x[at] = first;
   normed[at] = from_float<T>(next(first, column));
   if (column + 1u < width) {
-    const float second = as_float(table[token * width + column + 1u]) + cosine;
+    const float second = as_float(table[token * width + column + 1u]) + pair.y;
     x[at + 1] = second;
     normed[at + 1] = from_float<T>(next(second, column + 1u));
   }
 }
 
-// Buffers [ids, table, past, frequencies f64, following norm, x, normed]; params {rows, tokens per sequence, vocabulary, width}.
+// Buffers [ids, table, past, turns per position f64, following norm, x, normed]; params {rows, tokens per sequence, vocabulary, width}.
 template <typename T>
 int launch_embedding_sinusoid(const KernelArgs& args) {
   LLMOPT_REQUIRE(args.buffer_count == 7 && args.param_bytes == 16, "expects 7 buffers and 16 parameter bytes");
@@ -102,10 +122,14 @@ int launch_embedding_sinusoid(const KernelArgs& args) {
                      args.lengths[6] >= (size_t)rows * width * sizeof(T),
                  "buffer is too short");
   if (rows == 0) return 0;
-  launch_kernel(args, embedding_sinusoid_kernel<T>, dim3((pairs + 255u) / 256u, rows), dim3(256), 0,
+  uint32_t vectors = width % 4u == 0;
+  for (int i : {1, 4, 5, 6})
+    if ((uintptr_t)args.buffers[i] & 15u) vectors = 0;
+  const uint32_t threads = vectors ? width / 4u : pairs;
+  launch_kernel(args, embedding_sinusoid_kernel<T>, dim3((threads + 255u) / 256u, rows), dim3(256), 0,
                 (const long long*)args.buffers[0], (const T*)args.buffers[1], (const uint32_t*)args.buffers[2],
                 (const double*)args.buffers[3], (const float*)args.buffers[4], (float*)args.buffers[5], (T*)args.buffers[6],
-                tokens, vocabulary, width);
+                tokens, vocabulary, width, vectors);
   return check_launch(args);
 }
 

@@ -96,7 +96,7 @@ class TanhResidual:
         self.before = [before for before, _ in around] + [upload("final.norm")]
         self.after = [after for _, after in around]
         pairs = np.arange((config.width + 1) // 2, dtype=np.float64)
-        self.frequencies = Buffer.of_array(engine.runtime, 10000.0 ** (-2.0 * pairs / config.width))
+        self.turns = Buffer.of_array(engine.runtime, 10000.0 ** (-2.0 * pairs / config.width) / (2.0 * np.pi))  # per position
 
     def open(self, step):
         return _TanhStream(self, step)
@@ -108,7 +108,7 @@ class _TanhStream:
         self.residual, self.step, self.sublayer = residual, step, 0
         self.rows, self.x = engine.work32("residual", config.width), engine.work("normed", config.width)
         step.run(step.element("embedding_sinusoid"),
-                 [step.ids, residual.embedding, step.past, residual.frequencies, residual.before[0], self.rows, self.x],
+                 [step.ids, residual.embedding, step.past, residual.turns, residual.before[0], self.rows, self.x],
                  parameters.embedding_sinusoid(rows=step.rows, tokens=step.tokens, vocabulary=config.vocabulary,
                                                width=config.width))
 

@@ -162,7 +162,7 @@ def test_embedding_with_sinusoidal_positions(runtime, dtype, width):
     rng = np.random.default_rng(width)
     table = bf16_round(rng.standard_normal((30, width)))
     norm, next_norm = norm_vector(rng, width)
-    frequencies = 10000.0 ** (-2.0 * np.arange((width + 1) // 2) / width)
+    turns = 10000.0 ** (-2.0 * np.arange((width + 1) // 2) / width) / (2.0 * np.pi)
     for sequences, tokens in ((1, 1), (3, 1), (1, 70), (2, 5)):
         past = rng.integers(0, 300000, size=sequences).astype(np.uint32)
         past[0] = 0 if tokens == 70 else 262143
@@ -170,7 +170,7 @@ def test_embedding_with_sinusoidal_positions(runtime, dtype, width):
         x, normed = empty(runtime, sequences * tokens * width), empty(runtime, sequences * tokens * width, dtype)
         run(runtime, "llmopt_embedding_sinusoid_" + suffix(dtype),
             [upload(runtime, ids.astype(np.int64)), upload(runtime, table, dtype), upload(runtime, past),
-             upload_f64(runtime, frequencies), upload(runtime, norm), x, normed],
+             upload_f64(runtime, turns), upload(runtime, norm), x, normed],
             parameters.embedding_sinusoid(rows=sequences * tokens, tokens=tokens, vocabulary=30, width=width))
         places = (past[:, None].astype(np.int64) + np.arange(tokens)[None, :]).reshape(-1)
         want = table[ids] + plain.sinusoids(places, width)
