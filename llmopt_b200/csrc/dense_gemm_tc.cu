@@ -14,6 +14,8 @@
 // and the CTA lets its copies land, frees its tensor memory and returns.
 #include <cuda.h>
 
+#include <initializer_list>
+
 #include "dense_linear.cuh"
 #include "w4a16_tc_device.cuh"
 
@@ -27,6 +29,10 @@ namespace {
 constexpr uint32_t kRows = kExpertTile, kDepth = 64;
 constexpr uint32_t kEpilogueWarps = 8;
 constexpr uint32_t kThreads = (2 + kEpilogueWarps) * 32;  // TMA, MMA, epilogue
+constexpr uint32_t kStagingRow = 20;  // words of a lane's values on their way out: sixteen and four of padding
+// per epilogue warp; the others keep the shared memory as cache for what their writeback reads
+template <DenseStore STORE>
+constexpr uint32_t kStagingBytes = STORE == kStoreResidual || STORE == kStoreCached ? 32u * kStagingRow * 4u : 0u;
 constexpr uint32_t kXTileBytes = kRows * kDepth * 2;
 
 template <uint32_t BN>
@@ -40,7 +46,8 @@ struct Shape {
   static constexpr uint32_t kBarriers = kStages * kStageBytes;
   static constexpr uint32_t kHolder = kBarriers + (2 * kStages + 4) * 8;
   static constexpr uint32_t kAbort = kHolder + 4;
-  static constexpr uint32_t kSharedBytes = kAbort + 4 + 1024;  // slack: 1024-byte alignment of the tiles
+  static constexpr uint32_t kStaging = (kAbort + 4 + 15) / 16 * 16;
+  static constexpr uint32_t kSharedBytes = kStaging + 1024;  // without the staging; slack: 1024-byte alignment of the tiles
 };
 
 // kind::f16 with bfloat16 A and B (format 1), fp32 accumulator, both K-major.
@@ -48,12 +55,63 @@ __host__ __device__ constexpr uint32_t bf16_instruction(uint32_t m, uint32_t n) 
   return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((m >> 4) << 24);
 }
 
-// 32 neighbouring sums of an output row on their way out, and what they need besides, requested ahead of them.
+// 32 neighbouring sums of each of a warp's 32 rows on their way out, and what they need besides, requested ahead of them.
+// The sums lie a row per lane.  Plain rows leave in that order; where as much is read as written (the residual) or the target
+// rows lie apart (the cache) values change places through shared memory first, so that four lanes share 64 bytes of a row.
+
+// Sixteen words per lane -> what lane / 4 of eight rows at a time stores: take(row of the warp, four words, their place).
+template <typename Take>
+__device__ __forceinline__ void exchange(float* staging, const uint4 (&words)[4], Take take) {
+  const uint32_t lane = threadIdx.x & 31u;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) *reinterpret_cast<uint4*>(staging + lane * kStagingRow + j * 4) = words[j];
+  __syncwarp();
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const uint32_t row = i * 8u + (lane >> 2);
+    take(i, row, *reinterpret_cast<const uint4*>(staging + row * kStagingRow + (lane & 3u) * 4u), lane & 3u);
+  }
+  __syncwarp();  // read before the next exchange
+}
+
 template <DenseStore STORE>
 struct Piece {
   __device__ __forceinline__ void fetch(const DenseTask<STORE>&, uint32_t, uint32_t, uint32_t) {}
-  __device__ __forceinline__ void store(const DenseTask<STORE>& p, uint32_t row, uint32_t column, const uint32_t (&raw)[32]) const {
-    const uint32_t kept = dense_kept(p);
+  __device__ __forceinline__ void store(const DenseTask<STORE>& p, uint32_t first_row, uint32_t row_end, uint32_t column,
+                                        const uint32_t (&raw)[32], float* staging) const {
+    const uint32_t row = first_row + (threadIdx.x & 31u), kept = dense_kept(p);
+    if constexpr (STORE == kStoreCached) {
+      if (column >= p.split && column + 32u <= p.split + kept) {
+        bf16* const cached = row < row_end ? dense_cache_row<bf16>(p, row) : nullptr;
+        const uint32_t at = column - p.split, offset = dense_cache_offset(p, at);
+        if ((at + 32u <= p.key_columns || at >= p.key_columns) && offset % 8u == 0 && p.token_stride % 8u == 0) {
+          uint4 words[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            uint32_t packed[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int i = j * 8 + e * 2;
+              const __nv_bfloat162 pair = __floats2bfloat162_rn(dense_biased(p, column + i, __uint_as_float(raw[i])),
+                                                                dense_biased(p, column + i + 1, __uint_as_float(raw[i + 1])));
+              packed[e] = *reinterpret_cast<const uint32_t*>(&pair);
+            }
+            words[j] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+          }
+          exchange(staging, words, [&](int, uint32_t r, const uint4& v, uint32_t place) {
+            const unsigned long long target = __shfl_sync(0xffffffffu, (unsigned long long)(uintptr_t)cached, r);
+            if (target) *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>((uintptr_t)target) + offset + place * 8u) = v;
+          });
+          return;
+        }
+        if (!cached) return;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+          cached[dense_cache_offset(p, at + i)] = __float2bfloat16_rn(dense_biased(p, column + i, __uint_as_float(raw[i])));
+        return;
+      }
+    }
+    if (row >= row_end || column >= p.n) return;
     const size_t at = (size_t)row * p.split + column;
     const size_t at32 = (size_t)row * (p.n - p.split - kept) + (column - p.split - kept);
     auto value = [&](int i) {
@@ -80,24 +138,6 @@ struct Piece {
       for (int i = 0; i < 8; ++i) target[i] = make_float4(value(i * 4), value(i * 4 + 1), value(i * 4 + 2), value(i * 4 + 3));
       return;
     }
-    if constexpr (STORE == kStoreCached) {
-      if (column >= p.split && column + 32u <= p.split + kept) {
-        // one head may end and the next begin inside the piece, and keys may end and values begin
-        bf16* const cached = dense_cache_row<bf16>(p, row);
-        if (!cached) return;
-#pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-          const uint32_t first = dense_cache_offset(p, column - p.split + i), second = dense_cache_offset(p, column - p.split + i + 1);
-          if (second == first + 1u && ((uintptr_t)(cached + first) & 3u) == 0) {
-            *reinterpret_cast<__nv_bfloat162*>(cached + first) = __floats2bfloat162_rn(value(i), value(i + 1));
-          } else {
-            cached[first] = __float2bfloat16_rn(value(i));
-            cached[second] = __float2bfloat16_rn(value(i + 1));
-          }
-        }
-        return;
-      }
-    }
 #pragma unroll
     for (int i = 0; i < 32; ++i)
       if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
@@ -107,7 +147,10 @@ struct Piece {
 template <>
 struct Piece<kStorePair> {
   __device__ __forceinline__ void fetch(const DenseTask<kStorePair>&, uint32_t, uint32_t, uint32_t) {}
-  __device__ __forceinline__ void store(const DenseTask<kStorePair>& p, uint32_t row, uint32_t column, const uint32_t (&raw)[32]) const {
+  __device__ __forceinline__ void store(const DenseTask<kStorePair>& p, uint32_t first_row, uint32_t row_end, uint32_t column,
+                                        const uint32_t (&raw)[32], float*) const {
+    const uint32_t row = first_row + (threadIdx.x & 31u);
+    if (row >= row_end || column >= p.n) return;
     bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * (p.n / 2u) + column / 2u;
     const bool whole = column + 32u <= p.n && ((uintptr_t)target & 15u) == 0;
 #pragma unroll
@@ -136,39 +179,46 @@ struct Piece<kStorePair> {
 
 template <>
 struct Piece<kStoreResidual> {
-  float4 x[8];
-  static __device__ __forceinline__ bool vectors(const DenseTask<kStoreResidual>& p, uint32_t column) {
-    return p.n % 4u == 0 && column + 32u <= p.n;
-  }
-  __device__ __forceinline__ void fetch(const DenseTask<kStoreResidual>& p, uint32_t row, uint32_t row_end, uint32_t column) {
-    if (row >= row_end || !vectors(p, column)) return;
-    const float4* source = reinterpret_cast<const float4*>(p.residual + (size_t)row * p.n + column);
+  float4 x[8];  // in the order of the exchange
+  static __device__ __forceinline__ uint32_t row_of(uint32_t first_row, int i) { return first_row + (i & 3) * 8u + ((threadIdx.x & 31u) >> 2); }
+  static __device__ __forceinline__ uint32_t column_of(uint32_t column, int i) { return column + (i >> 2) * 16u + (threadIdx.x & 3u) * 4u; }
+  __device__ __forceinline__ void fetch(const DenseTask<kStoreResidual>& p, uint32_t first_row, uint32_t row_end, uint32_t column) {
+    if (p.n % 4u != 0) return;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) x[i] = source[i];
+    for (int i = 0; i < 8; ++i) {
+      const uint32_t row = row_of(first_row, i), c = column_of(column, i);
+      if (row < row_end && c < p.n) x[i] = *reinterpret_cast<const float4*>(p.residual + (size_t)row * p.n + c);
+    }
   }
-  __device__ __forceinline__ void store(const DenseTask<kStoreResidual>& p, uint32_t row, uint32_t column,
-                                        const uint32_t (&raw)[32]) const {
-    if (!vectors(p, column)) {
+  __device__ __forceinline__ void store(const DenseTask<kStoreResidual>& p, uint32_t first_row, uint32_t row_end, uint32_t column,
+                                        const uint32_t (&raw)[32], float* staging) const {
+    const uint32_t lane = threadIdx.x & 31u;
+    if (p.n % 4u != 0) {
 #pragma unroll
       for (int i = 0; i < 32; ++i)
-        if (column + i < p.n) dense_store<bf16>(p, row, column + i, __uint_as_float(raw[i]));
+        if (first_row + lane < row_end && column + i < p.n) dense_store<bf16>(p, first_row + lane, column + i, __uint_as_float(raw[i]));
       return;
     }
     const TanhNorm post(p.post_norm, p.n), next(p.next_norm, p.n);
-    float4* residual = reinterpret_cast<float4*>(p.residual + (size_t)row * p.n + column);
-    bf16* target = reinterpret_cast<bf16*>(p.out) + (size_t)row * p.n + column;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      float4 v = make_float4(__uint_as_float(raw[i * 4]), __uint_as_float(raw[i * 4 + 1]), __uint_as_float(raw[i * 4 + 2]),
-                             __uint_as_float(raw[i * 4 + 3]));
-      if (p.has_bias) {
-        const float* bias = p.bias + column + i * 4;
-        v.x += __ldg(bias), v.y += __ldg(bias + 1), v.z += __ldg(bias + 2), v.w += __ldg(bias + 3);
-      }
-      const float4 y = post.four_short(v, column + i * 4);
-      const float4 sum = make_float4(x[i].x + y.x, x[i].y + y.y, x[i].z + y.z, x[i].w + y.w);
-      residual[i] = sum;
-      store_four(target + i * 4, next.four_short(sum, column + i * 4));
+    for (int half = 0; half < 2; ++half) {
+      uint4 words[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        words[j] = make_uint4(raw[half * 16 + j * 4], raw[half * 16 + j * 4 + 1], raw[half * 16 + j * 4 + 2], raw[half * 16 + j * 4 + 3]);
+      exchange(staging, words, [&](int i, uint32_t r, const uint4& sums, uint32_t place) {
+        const uint32_t row = first_row + r, c = column + half * 16 + place * 4u;
+        if (row >= row_end || c >= p.n) return;
+        float4 v = make_float4(__uint_as_float(sums.x), __uint_as_float(sums.y), __uint_as_float(sums.z), __uint_as_float(sums.w));
+        if (p.has_bias) {
+          const float4 bias = __ldg(reinterpret_cast<const float4*>(p.bias + c));
+          v.x += bias.x, v.y += bias.y, v.z += bias.z, v.w += bias.w;
+        }
+        const float4 y = post.four_short(v, c), &held = x[half * 4 + i];
+        const float4 sum = make_float4(held.x + y.x, held.y + y.y, held.z + y.z, held.w + y.w);
+        *reinterpret_cast<float4*>(p.residual + (size_t)row * p.n + c) = sum;
+        store_four(reinterpret_cast<bf16*>(p.out) + (size_t)row * p.n + c, next.four_short(sum, c));
+      });
     }
   }
 };
@@ -283,14 +333,15 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
     }
   } else {
     const uint32_t quarter = warp & 3u, side = (warp - 2u) >> 2;  // lanes of tensor memory; every other piece of the columns
+    float* staging = reinterpret_cast<float*>(base_pointer + S::kStaging) + (warp - 2u) * (kStagingBytes<STORE> / 4u);
     uint32_t turn = 0;
     bool ok = true;
     for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++turn) {
       const uint32_t half = turn & 1u;
       const DenseTile rows = place(tile);
-      const uint32_t row = rows.first + quarter * 32u + lane, n0 = (tile / m_tiles) * BN;
+      const uint32_t first_row = rows.first + quarter * 32u, n0 = (tile / m_tiles) * BN;  // of this warp
       Piece<STORE> ahead;
-      ahead.fetch(p, row, rows.end, n0 + side * 32u);
+      ahead.fetch(p, first_row, rows.end, n0 + side * 32u);
       ok = !*abort_flag && barrier_wait(sums_full + half * 8, (turn >> 1) & 1u);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) {
@@ -306,8 +357,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_con
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         const uint32_t column = n0 + piece * 32u, following = piece + kEpilogueWarps / 4u;
         Piece<STORE> held = ahead;
-        if (following < BN / 32u) ahead.fetch(p, row, rows.end, n0 + following * 32u);
-        if (row < rows.end && column < p.n) held.store(p, row, column, raw);
+        if (following < BN / 32u) ahead.fetch(p, first_row, rows.end, n0 + following * 32u);
+        held.store(p, first_row, rows.end, column, raw, staging);
         __syncwarp();  // tcgen05.ld needs the whole warp
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -361,19 +412,22 @@ int run(const KernelArgs& args, const DenseProblem& p, uint32_t sms) {
       !make_map(&map_w, p.w, p.k, (uint64_t)p.n * (p.plan.tiles ? p.plan.experts : 1u), BN))
     return -1;
   auto kernel = dense_gemm_tc_kernel<BN, STORE>;
-  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSharedBytes) != cudaSuccess) {
+  constexpr uint32_t shared = S::kSharedBytes + kEpilogueWarps * kStagingBytes<STORE>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared) != cudaSuccess) {
     cudaGetLastError();
     return -1;
   }
   const uint32_t most = most_tiles(p), tiles = most * ((p.n + BN - 1u) / BN);
-  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), S::kSharedBytes, map_x, map_w, DenseTask<STORE>(p), p.plan, most,
+  launch_kernel(args, kernel, dim3(tiles < sms ? tiles : sms), dim3(kThreads), shared, map_x, map_w, DenseTask<STORE>(p), p.plan, most,
                 context_device_error(args.ctx));
   return check_launch(args);
 }
 
 template <DenseStore STORE>
 int run_tiles(const KernelArgs& args, const DenseProblem& p) {
-  if (args.ctx == nullptr || p.k % 8u != 0 || ((uintptr_t)p.x & 15u) != 0 || ((uintptr_t)p.w & 15u) != 0) return -1;
+  if (args.ctx == nullptr || p.k % 8u != 0) return -1;
+  for (const void* pointer : {p.x, p.w, (const void*)p.out, (const void*)p.out32, (const void*)p.pool})
+    if ((uintptr_t)pointer & 15u) return -1;
   const uint32_t sms = (uint32_t)context_sm_count(args.ctx);
   // waves times the cost of one MMA (an MMA of up to 128 columns costs about two thirds of one of 256)
   const uint32_t m_tiles = most_tiles(p);

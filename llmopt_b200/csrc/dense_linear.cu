@@ -314,7 +314,7 @@ int launch_dense_residual(const KernelArgs& args) {
   LLMOPT_REQUIRE(args.lengths[5] >= (size_t)p.m * p.n * 4 && args.lengths[6] >= (size_t)p.m * p.n * sizeof(T),
                  "output buffer is too short");
   LLMOPT_REQUIRE(p.out != p.x, "the product cannot overwrite its input");
-  for (int i = 3; i < 7; ++i) LLMOPT_REQUIRE(((uintptr_t)args.buffers[i] & 15u) == 0, "buffers must be 16-byte aligned");
+  for (int i = 2; i < 7; ++i) LLMOPT_REQUIRE(((uintptr_t)args.buffers[i] & 15u) == 0, "buffers must be 16-byte aligned");
   return run_dense<T>(args, p, kStoreResidual);
 }
 
